@@ -23,7 +23,7 @@
 
 namespace {
 constexpr int WARPS = 4;
-constexpr int MAX_HD = 512;
+constexpr int MOST_HD = 1024;         // heads of up to 512 entries take a smaller instantiation
 
 // q . k over one key row, accumulated in the order i = 0 .. hd-1.
 __device__ __forceinline__ float dot_row(const float* q, const float* k, int hd) {
@@ -60,7 +60,7 @@ __device__ __forceinline__ float dot_row(const float* q, const __nv_bfloat16* k,
     return dot;
 }
 
-template <typename T>
+template <typename T, int MAX_HD>
 __global__ void __launch_bounds__(WARPS * 32)
 attention_simt_kernel(const T* __restrict__ qkv, T* __restrict__ out,
                       const T* __restrict__ k_pool, const T* __restrict__ v_pool,
@@ -151,20 +151,22 @@ MLS_API int mls_attention_simt(const void* qkv, void* out, int dtype, const void
                                const float* slopes, int keep_first, long long out_stride,
                                cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
-    if (hd > MAX_HD || hd <= 0 || n_heads % n_kv) return MLS_ERR_UNSUPPORTED;
+    if (hd > MOST_HD || hd <= 0 || n_heads % n_kv) return MLS_ERR_UNSUPPORTED;
     if (out_stride <= 0) out_stride = (long long)n_heads * hd;
     const long long units = (long long)n_tokens * n_heads;
     const int blocks = (int)((units + WARPS - 1) / WARPS);
-    if (dtype == MLS_BF16)
-        MLS_LAUNCH((attention_simt_kernel<__nv_bfloat16>), dim3(blocks), dim3(WARPS * 32), 0,
-                   stream, (const __nv_bfloat16*)qkv, (__nv_bfloat16*)out,
-                   (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool, block_table,
-                   max_blocks, positions, req_of_token, n_tokens, n_heads, n_kv, hd, block_size,
-                   scale, window, softcap, n_pages, sink, slopes, keep_first, out_stride);
-    else
-        MLS_LAUNCH((attention_simt_kernel<float>), dim3(blocks), dim3(WARPS * 32), 0, stream,
-                   (const float*)qkv, (float*)out, (const float*)k_pool, (const float*)v_pool,
-                   block_table, max_blocks, positions, req_of_token, n_tokens, n_heads, n_kv, hd,
-                   block_size, scale, window, softcap, n_pages, sink, slopes, keep_first, out_stride);
+#define SIMT_GO(T, HD)                                                                            \
+    MLS_LAUNCH((attention_simt_kernel<T, HD>), dim3(blocks), dim3(WARPS * 32), 0, stream,          \
+               (const T*)qkv, (T*)out, (const T*)k_pool, (const T*)v_pool, block_table, max_blocks, \
+               positions, req_of_token, n_tokens, n_heads, n_kv, hd, block_size, scale, window,    \
+               softcap, n_pages, sink, slopes, keep_first, out_stride)
+    if (dtype == MLS_BF16) {
+        if (hd <= 512) SIMT_GO(__nv_bfloat16, 512);
+        else SIMT_GO(__nv_bfloat16, MOST_HD);
+    } else {
+        if (hd <= 512) SIMT_GO(float, 512);
+        else SIMT_GO(float, MOST_HD);
+    }
+#undef SIMT_GO
     return launch_status();
 }

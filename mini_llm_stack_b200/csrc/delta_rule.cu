@@ -1,0 +1,706 @@
+// The gated delta rule: a matrix state per head that decays, forgets what it holds under the
+// token's key and takes the token's value in, carried from token to token in a float32 state
+// slot per request.
+//
+// Per head, with key size e, value size f, state S [e, f], unit vectors q (times e^-1/2) and k,
+// a decay g in (0, 1) and a step size b in (0, 1) per token:
+//
+//   S <- g S;   u = b (v - S^T k);   S <- S + k u^T;   o = S^T q
+//
+// q, k and v are projections that pass a short causal convolution per channel and silu; several
+// value heads may share a key head.  Written with the state before the token, the token needs
+// two products with it that do not wait for one another, S^T k and S^T q:
+//
+//   u = b (v - g S^T k);   o = g S^T q + (k . q) u;   S <- g S + k u^T
+//
+//   mls_delta_prep   projection rows (float32) -> convolution, silu, unit vectors, k . q, decay
+//                    and step size, as the rows the scan reads
+//   mls_delta_scan   walks the tokens of every request through the state; also stores the
+//                    convolution's last inputs
+//   mls_delta_step   one token a request: all of the above and what follows (norm over the
+//                    head's values, weight, silu gate) in one kernel
+//
+// Layout of a request's state slot: S of every head transposed and padded, [H][fr][er] with
+// er = e rounded up to 32 and fr = f rounded up to 16 (the padding stays zero), then the
+// convolution's inputs as a ring [taps][channels]: position p lies in row p mod taps, so a
+// token's row never falls on a row that its own convolution reads.  Rows of positions before
+// the sequence's start are never read.
+//
+// A warp owns four columns of S with eight lanes a column; a lane keeps er / 8 rows of its
+// column in registers, four neighbouring rows at a time (16-byte accesses of the state and of
+// k and q), and multiplies them two at a time (fma.rn.f32x2).  The sum over the rows is the
+// lane's own in a fixed order and three shuffles: a token's bits depend neither on the batch
+// nor on how the tokens were cut into steps (in steps that run the same kernel).
+// Everything is float32.
+#include "common.cuh"
+
+namespace {
+constexpr float DR_UNIT_EPS = 1e-6f;     // inside the root of the unit vectors
+
+__device__ __forceinline__ float silu1(float z) { return z / (1.0f + expf(-z)); }
+__device__ __forceinline__ float sigmoid1(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float softplus1(float z) {
+    return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
+}
+
+// Two float32 operations in one instruction on register pairs.
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pack2(float a, float b) {
+    f32x2 r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+    return r;
+}
+__device__ __forceinline__ float sum2(f32x2 v) {
+    float a, b;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v));
+    return a + b;
+}
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+    f32x2 d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+    f32x2 d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ f32x2 add2(f32x2 a, f32x2 b) {
+    f32x2 d;
+    asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+// the sum over the eight lanes that share a column
+__device__ __forceinline__ float column_sum(float v) {
+    v += __shfl_xor_sync(0xffffffffu, v, 1);
+    v += __shfl_xor_sync(0xffffffffu, v, 2);
+    v += __shfl_xor_sync(0xffffffffu, v, 4);
+    return v;
+}
+__device__ __forceinline__ void copy16(void* dst, const void* src) {
+    const unsigned d = (unsigned)__cvta_generic_to_shared(dst);
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(d), "l"(src) : "memory");
+}
+
+// Sizes, places and parameters every kernel here needs.
+struct DeltaArgs {
+    const float* proj;                 // [parts][T, width]: q heads | k heads | v heads, gates, ...
+    int n_parts;
+    long long part_stride;
+    int width, qkv_col, a_col, b_col, g_col;
+    const void* conv;                  // [channels, taps], last column meets the current token
+    int conv_dtype, taps, channels;    // channels = 2 G e + H f, in the order of the projection
+    const float* a_exp;                // [H]: exp(A_log)
+    const float* dt_bias;              // [H]
+    const int* state_slot;
+    const int* cu_q;
+    const int* req_of_token;
+    const int* positions;
+    float* state;                      // [slots], state_stride floats apart
+    long long state_stride, ring_at;   // ring_at: the ring's place in a slot
+    int n_tokens, n_requests;
+    int H, G, e, f, er, fr;
+    float q_scale;                     // e^-1/2
+    __device__ __forceinline__ float at(int t, int col) const {
+        const float* p = proj + (size_t)t * width + col;
+        float s = *p;
+        int k = 1;
+        for (; k + 4 <= n_parts; k += 4) {
+            float w[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) w[i] = p[(size_t)(k + i) * part_stride];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) s += w[i];
+        }
+        for (; k < n_parts; ++k) s += p[(size_t)k * part_stride];
+        return s;
+    }
+    __device__ __forceinline__ float* ring(int slot) const {
+        return state + (size_t)slot * state_stride + ring_at;
+    }
+};
+
+// The rows the scan reads, float32: [q: G er | k: G er | v: H fr | (decay, step, k . q, 0): 4 H].
+struct RowLayout {
+    int k_off, v_off, s_off, row;
+};
+__host__ __device__ inline RowLayout row_layout(int H, int G, int er, int fr) {
+    RowLayout l;
+    l.k_off = G * er;
+    l.v_off = 2 * G * er;
+    l.s_off = l.v_off + H * fr;
+    l.row = l.s_off + 4 * H;
+    return l;
+}
+
+// A head's channels spread over a warp (channel lane + 32 i) with the convolution's weights and
+// its last inputs; TT >= taps, the places before the real taps count as zero.
+template <int NI, int TT>
+struct ConvHead {
+    float w[TT][NI], win[TT - 1][NI];
+    int col, first, n;                 // column in a projection row, first channel, channels
+    __device__ __forceinline__ void init(const DeltaArgs& a, int channel0, int count, int lane) {
+        col = a.qkv_col + channel0;
+        first = channel0;
+        n = count;
+#pragma unroll
+        for (int j = 0; j < TT; ++j)
+#pragma unroll
+            for (int i = 0; i < NI; ++i) {
+                const int c = lane + 32 * i, tap = j - (TT - a.taps);
+                w[j][i] = (tap >= 0 && c < n)
+                    ? load_as_float(a.conv, (size_t)(first + c) * a.taps + tap, a.conv_dtype) : 0.f;
+            }
+    }
+    // the inputs before token t (the i_t-th of this step of its request, at position p)
+    __device__ __forceinline__ void fill(const DeltaArgs& a, int t, int i_t, int p,
+                                         const float* ring, int lane) {
+#pragma unroll
+        for (int j = 0; j < TT - 1; ++j) {
+            const int back = TT - 1 - j;
+#pragma unroll
+            for (int i = 0; i < NI; ++i) {
+                const int c = lane + 32 * i;
+                float v = 0.f;
+                if (back < a.taps && back <= p && c < n)
+                    v = back <= i_t ? a.proj[(size_t)(t - back) * a.width + col + c]
+                                    : ring[(size_t)((p - back) % a.taps) * a.channels + first + c];
+                win[j][i] = v;
+            }
+        }
+    }
+    __device__ __forceinline__ void load(const DeltaArgs& a, int t, int lane, float (&x)[NI]) const {
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+            const int c = lane + 32 * i;
+            x[i] = c < n ? a.proj[(size_t)t * a.width + col + c] : 0.f;
+        }
+    }
+    __device__ __forceinline__ void step(const float (&x)[NI], float (&y)[NI]) {
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+            float s = 0.f;
+#pragma unroll
+            for (int j = 0; j < TT - 1; ++j) s = fmaf(w[j][i], win[j][i], s);
+            s = fmaf(w[TT - 1][i], x[i], s);
+            y[i] = silu1(s);
+#pragma unroll
+            for (int j = 0; j + 1 < TT - 1; ++j) win[j][i] = win[j + 1][i];
+            win[TT - 2][i] = x[i];
+        }
+    }
+};
+
+constexpr int DP_RUN = 8;              // consecutive tokens a warp takes
+constexpr int DP_WARPS = 4;
+
+// One warp a (run of tokens, head): a key head's q and k together, or a value head.
+template <int NI, int TT>
+__global__ void __launch_bounds__(DP_WARPS * 32)
+delta_prep_kernel(const DeltaArgs a, float* __restrict__ out) {
+    chain_release();
+    const int lane = threadIdx.x & 31, unit = blockIdx.y * DP_WARPS + (threadIdx.x >> 5);
+    if (unit >= a.G + a.H) return;
+    const RowLayout lay = row_layout(a.H, a.G, a.er, a.fr);
+    const int t_begin = blockIdx.x * DP_RUN, t_end = min(t_begin + DP_RUN, a.n_tokens);
+    int r_now = -1;
+    if (unit < a.G) {
+        const int ratio = a.H / a.G;
+        ConvHead<NI, TT> hq, hk;
+        hq.init(a, unit * a.e, a.e, lane);
+        hk.init(a, (a.G + unit) * a.e, a.e, lane);
+        chain_wait();
+        float xq[NI], xk[NI];
+        hq.load(a, t_begin, lane, xq);
+        hk.load(a, t_begin, lane, xk);
+        for (int t = t_begin; t < t_end; ++t) {
+            const int r = a.req_of_token[t];
+            if (r != r_now) {
+                const float* ring = a.ring(a.state_slot[r]);
+                const int i_t = t - a.cu_q[r], p = a.positions[t];
+                hq.fill(a, t, i_t, p, ring, lane);
+                hk.fill(a, t, i_t, p, ring, lane);
+                r_now = r;
+            }
+            float yq[NI], yk[NI];
+            hq.step(xq, yq);
+            hk.step(xk, yk);
+            if (t + 1 < t_end) {
+                hq.load(a, t + 1, lane, xq);
+                hk.load(a, t + 1, lane, xk);
+            }
+            float sq = 0.f, sk = 0.f, sqk = 0.f;
+#pragma unroll
+            for (int i = 0; i < NI; ++i) {
+                if (lane + 32 * i >= a.e) yq[i] = yk[i] = 0.f;
+                sq = fmaf(yq[i], yq[i], sq);
+                sk = fmaf(yk[i], yk[i], sk);
+                sqk = fmaf(yq[i], yk[i], sqk);
+            }
+            const float iq = 1.0f / sqrtf(warp_sum(sq) + DR_UNIT_EPS) * a.q_scale;
+            const float ik = 1.0f / sqrtf(warp_sum(sk) + DR_UNIT_EPS);
+            const float kq = warp_sum(sqk) * iq * ik;
+            float* row = out + (size_t)t * lay.row;
+#pragma unroll
+            for (int i = 0; i < NI; ++i) {
+                const int c = lane + 32 * i;
+                if (c < a.er) {
+                    row[unit * a.er + c] = yq[i] * iq;
+                    row[lay.k_off + unit * a.er + c] = yk[i] * ik;
+                }
+            }
+            for (int hh = lane; hh < ratio; hh += 32) {
+                const int head = unit * ratio + hh;
+                const float za = a.proj[(size_t)t * a.width + a.a_col + head] + a.dt_bias[head];
+                const float zb = a.proj[(size_t)t * a.width + a.b_col + head];
+                const float g = expf(-a.a_exp[head] * softplus1(za));
+                *reinterpret_cast<float4*>(row + lay.s_off + 4 * head) =
+                    make_float4(g, sigmoid1(zb), kq, 0.f);
+            }
+        }
+    } else {
+        const int head = unit - a.G;
+        ConvHead<NI, TT> hv;
+        hv.init(a, 2 * a.G * a.e + head * a.f, a.f, lane);
+        chain_wait();
+        float x[NI];
+        hv.load(a, t_begin, lane, x);
+        for (int t = t_begin; t < t_end; ++t) {
+            const int r = a.req_of_token[t];
+            if (r != r_now) {
+                hv.fill(a, t, t - a.cu_q[r], a.positions[t], a.ring(a.state_slot[r]), lane);
+                r_now = r;
+            }
+            float y[NI];
+            hv.step(x, y);
+            if (t + 1 < t_end) hv.load(a, t + 1, lane, x);
+            float* row = out + (size_t)t * lay.row + lay.v_off + head * a.fr;
+#pragma unroll
+            for (int i = 0; i < NI; ++i) {
+                const int c = lane + 32 * i;
+                if (c < a.fr) row[c] = c < a.f ? y[i] : 0.f;
+            }
+        }
+    }
+}
+
+constexpr int DS_COLS = 16;            // columns of S a CTA of the scan owns
+constexpr int DS_THREADS = 128;        // four warps, four columns each
+constexpr int DS_TOKENS = 16;          // tokens in one of the two buffers
+
+// R4: groups of four rows a lane keeps, er = 32 R4.
+template <int R4>
+__global__ void __launch_bounds__(DS_THREADS)
+delta_scan_kernel(const DeltaArgs a, const float* __restrict__ rows, float* __restrict__ out) {
+    constexpr int ER = 32 * R4;
+    constexpr int TOK = 2 * ER + DS_COLS + 4;          // floats of a token in shared memory
+    chain_release();
+    extern __shared__ __align__(16) float smem[];      // [2][DS_TOKENS][TOK]
+    const int r = blockIdx.z, head = blockIdx.y, col0 = blockIdx.x * DS_COLS;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, grp = lane & 7;
+    const int my = warp * 4 + (lane >> 3), col = col0 + my;
+    const RowLayout lay = row_layout(a.H, a.G, ER, a.fr);
+    const int t0 = a.cu_q[r], n = a.cu_q[r + 1] - t0;
+    if (n <= 0) return;
+    const int slot = a.state_slot[r];
+    chain_wait();
+    const int kv = head / (a.H / a.G);
+    const float* q_src = rows + kv * ER;
+    const float* k_src = rows + lay.k_off + kv * ER;
+    const float* v_src = rows + lay.v_off + head * a.fr + col0;
+    const float* s_src = rows + lay.s_off + 4 * head;
+    auto fetch = [&](int b0) {                          // the copies of tokens b0 .. into their buffer
+        const int nb = min(DS_TOKENS, n - b0);
+        float* dst = smem + (size_t)((b0 / DS_TOKENS) & 1) * DS_TOKENS * TOK;
+        constexpr int U = ER / 4, PER = 2 * U + DS_COLS / 4 + 1;
+        for (int u = threadIdx.x; u < nb * PER; u += DS_THREADS) {
+            const int tt = u / PER, i = u - tt * PER;
+            const size_t t = (size_t)(t0 + b0 + tt) * lay.row;
+            const float* src = i < U ? q_src + t + 4 * i
+                : i < 2 * U ? k_src + t + 4 * (i - U)
+                : i < 2 * U + DS_COLS / 4 ? v_src + t + 4 * (i - 2 * U) : s_src + t;
+            copy16(dst + (size_t)tt * TOK + 4 * i, src);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    fetch(0);
+    float* S = a.state + (size_t)slot * a.state_stride + ((size_t)head * a.fr + col) * ER + 4 * grp;
+    f32x2 s[R4][2];
+#pragma unroll
+    for (int i = 0; i < R4; ++i) {
+        const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(S + 32 * i);
+        s[i][0] = v.x;
+        s[i][1] = v.y;
+    }
+    // the convolution's last inputs (the preparation has read the older ones)
+    {
+        const int keep = a.taps - 1, i0 = max(0, n - keep);
+        float* ring = a.ring(slot);
+        const int part = (int)(blockIdx.y * gridDim.x + blockIdx.x) * DS_THREADS + threadIdx.x;
+        const int step = (int)(gridDim.x * gridDim.y) * DS_THREADS;
+        for (int i = i0; i < n && keep > 0; ++i) {
+            const size_t row = (size_t)(a.positions[t0 + i] % a.taps) * a.channels;
+            for (int c = part; c < a.channels; c += step)
+                ring[row + c] = a.proj[(size_t)(t0 + i) * a.width + a.qkv_col + c];
+        }
+    }
+    const bool writes = grp == 0 && col < a.f;
+    float* o_col = out + (size_t)t0 * a.H * a.f + (size_t)head * a.f + col;
+    for (int b0 = 0; b0 < n; b0 += DS_TOKENS) {
+        const int nb = min(DS_TOKENS, n - b0);
+        if (b0 + DS_TOKENS < n) {
+            fetch(b0 + DS_TOKENS);
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+        } else {
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+        }
+        __syncthreads();
+        const float* tok = smem + (size_t)((b0 / DS_TOKENS) & 1) * DS_TOKENS * TOK;
+        ulonglong2 k[R4], q[R4];
+#pragma unroll
+        for (int i = 0; i < R4; ++i) {
+            q[i] = *reinterpret_cast<const ulonglong2*>(tok + 32 * i + 4 * grp);
+            k[i] = *reinterpret_cast<const ulonglong2*>(tok + ER + 32 * i + 4 * grp);
+        }
+        for (int tt = 0; tt < nb; ++tt, tok += TOK) {
+            f32x2 dk[2] = {0ull, 0ull}, dq[2] = {0ull, 0ull};
+#pragma unroll
+            for (int i = 0; i < R4; ++i) {
+                dk[0] = fma2(s[i][0], k[i].x, dk[0]);
+                dk[1] = fma2(s[i][1], k[i].y, dk[1]);
+            }
+#pragma unroll
+            for (int i = 0; i < R4; ++i) {
+                dq[0] = fma2(s[i][0], q[i].x, dq[0]);
+                dq[1] = fma2(s[i][1], q[i].y, dq[1]);
+            }
+            const float vj = tok[2 * ER + my];
+            const float4 sc = *reinterpret_cast<const float4*>(tok + 2 * ER + DS_COLS);
+            float sk = column_sum(sum2(add2(dk[0], dk[1])));
+            float sq = column_sum(sum2(add2(dq[0], dq[1])));
+            // the next token's key and query come while the sums cross the lanes
+            ulonglong2 kn[R4];
+            const float* nxt = tt + 1 < nb ? tok + TOK : tok;
+#pragma unroll
+            for (int i = 0; i < R4; ++i) {
+                q[i] = *reinterpret_cast<const ulonglong2*>(nxt + 32 * i + 4 * grp);
+                kn[i] = *reinterpret_cast<const ulonglong2*>(nxt + ER + 32 * i + 4 * grp);
+            }
+            const f32x2 g2 = pack2(sc.x, sc.x);
+#pragma unroll
+            for (int i = 0; i < R4; ++i) {
+                s[i][0] = mul2(g2, s[i][0]);
+                s[i][1] = mul2(g2, s[i][1]);
+            }
+            const float u = sc.y * fmaf(-sc.x, sk, vj);
+            const f32x2 u2 = pack2(u, u);
+#pragma unroll
+            for (int i = 0; i < R4; ++i) {
+                s[i][0] = fma2(k[i].x, u2, s[i][0]);
+                s[i][1] = fma2(k[i].y, u2, s[i][1]);
+                k[i] = kn[i];
+            }
+            if (writes) o_col[(size_t)(b0 + tt) * a.H * a.f] = fmaf(sc.x, sq, sc.z * u);
+        }
+        __syncthreads();                                // before this buffer is fetched into again
+    }
+#pragma unroll
+    for (int i = 0; i < R4; ++i)
+        *reinterpret_cast<ulonglong2*>(S + 32 * i) = make_ulonglong2(s[i][0], s[i][1]);
+}
+
+constexpr int DT_THREADS = 256;        // eight warps of a (request, head)
+
+// One token a request: convolution, unit vectors, the state's step, head norm and gate.  C:
+// columns a lane keeps at a time (a pass of the block takes 32 C columns).
+template <int R4, int C, typename T>
+__global__ void __launch_bounds__(DT_THREADS)
+delta_step_kernel(const DeltaArgs a, const float* __restrict__ norm_w, float eps,
+                  T* __restrict__ out) {
+    constexpr int ER = 32 * R4;
+    chain_release();
+    extern __shared__ __align__(16) float smem[];
+    float* q_s = smem;                                  // [ER]
+    float* k_s = q_s + ER;                              // [ER]
+    float* v_s = k_s + ER;                              // [fr]
+    float* o_s = v_s + a.fr;                            // [fr]
+    float* old_s = o_s + a.fr;                          // [2 e + f]: the older taps' share
+    float* now_s = old_s + 2 * a.e + a.f;               // [2 e + f]: the current token's tap
+    __shared__ float sums[3];
+    __shared__ float gb[2];
+    const int r = blockIdx.y, head = blockIdx.x, t = a.cu_q[r];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, grp = lane & 7;
+    const int ratio = a.H / a.G, kv = head / ratio;
+    const int slot = a.state_slot[r], p = a.positions[t];
+    float* S = a.state + (size_t)slot * a.state_stride + (size_t)head * a.fr * ER + 4 * grp;
+    float* ring = a.ring(slot);
+    // nothing of the state slot is written by this step's earlier kernels, so the state and the
+    // convolution's older inputs are read ahead of the wait
+    f32x2 s[C][R4][2];
+    auto load_columns = [&](int c0) {
+#pragma unroll
+        for (int ci = 0; ci < C; ++ci) {
+            const int col = c0 + (warp * C + ci) * 4 + (lane >> 3);
+#pragma unroll
+            for (int i = 0; i < R4; ++i) {
+                ulonglong2 v = make_ulonglong2(0ull, 0ull);
+                if (col < a.fr)
+                    v = *reinterpret_cast<const ulonglong2*>(S + (size_t)col * ER + 32 * i);
+                s[ci][i][0] = v.x;
+                s[ci][i][1] = v.y;
+            }
+        }
+    };
+    load_columns(0);
+    const int locals = 2 * a.e + a.f;
+    auto channel_of = [&](int u) {                      // a local channel's place among all
+        return u < a.e ? kv * a.e + u
+             : u < 2 * a.e ? (a.G + kv) * a.e + (u - a.e)
+                           : 2 * a.G * a.e + head * a.f + (u - 2 * a.e);
+    };
+    for (int u = threadIdx.x; u < locals; u += DT_THREADS) {
+        const int c = channel_of(u);
+        float acc = 0.f;
+        for (int j = 0; j + 1 < a.taps; ++j) {
+            const int back = a.taps - 1 - j;
+            if (back <= p)
+                acc = fmaf(load_as_float(a.conv, (size_t)c * a.taps + j, a.conv_dtype),
+                           ring[(size_t)((p - back) % a.taps) * a.channels + c], acc);
+        }
+        old_s[u] = acc;
+        now_s[u] = load_as_float(a.conv, (size_t)c * a.taps + a.taps - 1, a.conv_dtype);
+    }
+    for (int i = threadIdx.x; i < ER; i += DT_THREADS)
+        if (i >= a.e) q_s[i] = k_s[i] = 0.f;
+    for (int i = threadIdx.x; i < a.fr; i += DT_THREADS)
+        if (i >= a.f) v_s[i] = 0.f;
+    const float a_exp = a.a_exp[head], dt = a.dt_bias[head];
+    chain_wait();
+    const bool keeps_qk = head % ratio == 0;
+    const size_t ring_row = (size_t)(p % a.taps) * a.channels;
+    for (int u = threadIdx.x; u < locals; u += DT_THREADS) {
+        const int c = channel_of(u);
+        const float x = a.at(t, a.qkv_col + c);
+        const float y = silu1(fmaf(now_s[u], x, old_s[u]));
+        if (u < a.e) q_s[u] = y;
+        else if (u < 2 * a.e) k_s[u - a.e] = y;
+        else v_s[u - 2 * a.e] = y;
+        if (a.taps > 1 && (keeps_qk || u >= 2 * a.e)) ring[ring_row + c] = x;
+    }
+    if (threadIdx.x == DT_THREADS - 1) {
+        gb[0] = expf(-a_exp * softplus1(a.at(t, a.a_col + head) + dt));
+        gb[1] = sigmoid1(a.at(t, a.b_col + head));
+    }
+    __syncthreads();
+    if (warp < 3) {
+        const float* x = warp == 1 ? k_s : q_s;
+        const float* y = warp == 0 ? q_s : k_s;
+        float v = 0.f;
+#pragma unroll
+        for (int i = 0; i < R4; ++i) v = fmaf(x[lane + 32 * i], y[lane + 32 * i], v);
+        v = warp_sum(v);
+        if (lane == 0) sums[warp] = v;
+    }
+    __syncthreads();
+    const float iq = 1.0f / sqrtf(sums[0] + DR_UNIT_EPS) * a.q_scale;
+    const float ik = 1.0f / sqrtf(sums[1] + DR_UNIT_EPS);
+    const float kq = sums[2] * iq * ik, g = gb[0], beta = gb[1];
+    const f32x2 g2 = pack2(g, g);
+    for (int c0 = 0; c0 < a.fr; c0 += 32 * C) {
+        if (c0 > 0) load_columns(c0);
+        f32x2 dk[C], dq[C];
+#pragma unroll
+        for (int ci = 0; ci < C; ++ci) dk[ci] = dq[ci] = 0ull;
+#pragma unroll
+        for (int i = 0; i < R4; ++i) {
+            const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(k_s + 32 * i + 4 * grp);
+            const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(q_s + 32 * i + 4 * grp);
+#pragma unroll
+            for (int ci = 0; ci < C; ++ci) {
+                dk[ci] = fma2(s[ci][i][0], k.x, dk[ci]);
+                dq[ci] = fma2(s[ci][i][0], q.x, dq[ci]);
+                dk[ci] = fma2(s[ci][i][1], k.y, dk[ci]);
+                dq[ci] = fma2(s[ci][i][1], q.y, dq[ci]);
+            }
+        }
+        f32x2 u2[C];
+#pragma unroll
+        for (int ci = 0; ci < C; ++ci) {
+            const int col = c0 + (warp * C + ci) * 4 + (lane >> 3);
+            const float sk = column_sum(sum2(dk[ci])) * ik, sq = column_sum(sum2(dq[ci])) * iq;
+            const float u = col < a.fr ? beta * fmaf(-g, sk, v_s[col]) : 0.f;
+            u2[ci] = pack2(u * ik, u * ik);
+            if (grp == 0 && col < a.fr) o_s[col] = fmaf(g, sq, kq * u);
+        }
+#pragma unroll
+        for (int i = 0; i < R4; ++i) {
+            const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(k_s + 32 * i + 4 * grp);
+#pragma unroll
+            for (int ci = 0; ci < C; ++ci) {
+                const int col = c0 + (warp * C + ci) * 4 + (lane >> 3);
+                if (col < a.fr)
+                    *reinterpret_cast<ulonglong2*>(S + (size_t)col * ER + 32 * i) =
+                        make_ulonglong2(fma2(k.x, u2[ci], mul2(g2, s[ci][i][0])),
+                                        fma2(k.y, u2[ci], mul2(g2, s[ci][i][1])));
+            }
+        }
+    }
+    __syncthreads();
+    float ss = 0.f;
+    for (int c = lane; c < a.f; c += 32) ss = fmaf(o_s[c], o_s[c], ss);     // every warp for itself
+    const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)a.f + eps);
+    for (int c = threadIdx.x; c < a.f; c += DT_THREADS) {
+        const float z = a.at(t, a.g_col + head * a.f + c);
+        Elem<T>::store(out + (size_t)t * a.H * a.f + head * a.f + c,
+                       o_s[c] * inv * norm_w[c] * silu1(z));
+    }
+}
+
+DeltaArgs make_args(const float* proj, int n_parts, long long part_stride, int width, int qkv_col,
+                    int a_col, int b_col, int g_col, const void* conv, int conv_dtype, int taps,
+                    const float* a_exp, const float* dt_bias, const int* state_slot,
+                    const int* cu_q, const int* req_of_token, const int* positions, float* state,
+                    long long state_stride, int n_tokens, int n_requests, int H, int G, int e,
+                    int f) {
+    DeltaArgs a;
+    a.proj = proj; a.n_parts = n_parts; a.part_stride = part_stride; a.width = width;
+    a.qkv_col = qkv_col; a.a_col = a_col; a.b_col = b_col; a.g_col = g_col; a.conv = conv;
+    a.conv_dtype = conv_dtype; a.taps = taps; a.channels = 2 * G * e + H * f; a.a_exp = a_exp;
+    a.dt_bias = dt_bias; a.state_slot = state_slot; a.cu_q = cu_q; a.req_of_token = req_of_token;
+    a.positions = positions; a.state = state; a.state_stride = state_stride;
+    a.n_tokens = n_tokens; a.n_requests = n_requests; a.H = H; a.G = G; a.e = e; a.f = f;
+    a.er = (e + 31) / 32 * 32;
+    a.fr = (f + 15) / 16 * 16;
+    a.ring_at = (long long)H * a.fr * a.er;
+    a.q_scale = 1.0f / sqrtf((float)e);
+    return a;
+}
+bool sizes_ok(const DeltaArgs& a) {
+    return a.H > 0 && a.G > 0 && a.H % a.G == 0 && a.e > 0 && a.e <= 256 && a.f > 0 && a.taps >= 1 &&
+           a.n_parts >= 1 && a.state_stride % 4 == 0 &&
+           a.state_stride >= a.ring_at + (long long)a.taps * a.channels;
+}
+
+template <int NI>
+int launch_prep(const DeltaArgs& a, float* out, cudaStream_t stream) {
+    const dim3 grid((a.n_tokens + DP_RUN - 1) / DP_RUN, (a.G + a.H + DP_WARPS - 1) / DP_WARPS);
+    if (a.taps <= 4) MLS_LAUNCH((delta_prep_kernel<NI, 4>), grid, dim3(DP_WARPS * 32), 0, stream, a, out);
+    else if (a.taps <= 8) MLS_LAUNCH((delta_prep_kernel<NI, 8>), grid, dim3(DP_WARPS * 32), 0, stream, a, out);
+    else MLS_LAUNCH((delta_prep_kernel<NI, 16>), grid, dim3(DP_WARPS * 32), 0, stream, a, out);
+    return launch_status();
+}
+template <int R4>
+int launch_scan(const DeltaArgs& a, const float* rows, float* out, cudaStream_t stream) {
+    const size_t smem = (size_t)2 * DS_TOKENS * (2 * 32 * R4 + DS_COLS + 4) * sizeof(float);
+    if (smem > 48 * 1024) {
+        const int rc = (int)cudaFuncSetAttribute(delta_scan_kernel<R4>,
+                                                 cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (rc) return rc;
+    }
+    MLS_LAUNCH((delta_scan_kernel<R4>), dim3(a.fr / DS_COLS, a.H, a.n_requests), dim3(DS_THREADS),
+               smem, stream, a, rows, out);
+    return launch_status();
+}
+template <int R4, int C>
+int launch_step(const DeltaArgs& a, const float* norm_w, float eps, void* out, int dtype,
+                cudaStream_t stream) {
+    const size_t smem = ((size_t)2 * 32 * R4 + 2 * a.fr + 2 * (2 * a.e + a.f)) * sizeof(float);
+    if (smem > 200 * 1024) return MLS_ERR_UNSUPPORTED;
+    if (dtype == MLS_BF16) {
+        auto kernel = delta_step_kernel<R4, C, __nv_bfloat16>;
+        if (smem > 48 * 1024) {
+            const int rc = (int)cudaFuncSetAttribute(
+                kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+            if (rc) return rc;
+        }
+        MLS_LAUNCH(kernel, dim3(a.H, a.n_requests), dim3(DT_THREADS), smem, stream, a, norm_w, eps,
+                   (__nv_bfloat16*)out);
+    } else {
+        auto kernel = delta_step_kernel<R4, C, float>;
+        if (smem > 48 * 1024) {
+            const int rc = (int)cudaFuncSetAttribute(
+                kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+            if (rc) return rc;
+        }
+        MLS_LAUNCH(kernel, dim3(a.H, a.n_requests), dim3(DT_THREADS), smem, stream, a, norm_w, eps,
+                   (float*)out);
+    }
+    return launch_status();
+}
+}  // namespace
+
+// Floats of one prepared row, and of a request's state.
+MLS_API int mls_delta_row_floats(int H, int G, int e, int f) {
+    return row_layout(H, G, (e + 31) / 32 * 32, (f + 15) / 16 * 16).row;
+}
+MLS_API long long mls_delta_state_floats(int H, int G, int e, int f, int taps) {
+    const long long s = (long long)H * ((f + 15) / 16 * 16) * ((e + 31) / 32 * 32) +
+                        (long long)taps * (2LL * G * e + (long long)H * f);
+    return (s + 3) / 4 * 4;
+}
+
+// Preparation and scan of the tokens of a step (rows: scratch, [T, mls_delta_row_floats]);
+// out [T, H f] float32.
+MLS_API int mls_delta_prep(const float* proj, int width, int qkv_col, int a_col, int b_col,
+                           const void* conv, int conv_dtype, int taps, const float* a_exp,
+                           const float* dt_bias, const int* state_slot, const int* cu_q,
+                           const int* req_of_token, const int* positions, float* state,
+                           long long state_stride, int n_tokens, int n_requests, int H, int G,
+                           int e, int f, float* rows, cudaStream_t stream) {
+    if (n_tokens <= 0 || n_requests <= 0) return 0;
+    const DeltaArgs a = make_args(proj, 1, 0, width, qkv_col, a_col, b_col, 0, conv, conv_dtype, taps,
+                                  a_exp, dt_bias, state_slot, cu_q, req_of_token, positions, state,
+                                  state_stride, n_tokens, n_requests, H, G, e, f);
+    if (!sizes_ok(a) || taps > 16 || a.fr > 256) return MLS_ERR_UNSUPPORTED;
+    const int ni = (max(a.er, a.fr) + 31) / 32;
+    if (ni <= 1) return launch_prep<1>(a, rows, stream);
+    if (ni <= 2) return launch_prep<2>(a, rows, stream);
+    if (ni <= 4) return launch_prep<4>(a, rows, stream);
+    return launch_prep<8>(a, rows, stream);
+}
+
+MLS_API int mls_delta_scan(const float* rows, const float* proj, int width, int qkv_col, int taps,
+                           const int* state_slot, const int* cu_q, const int* positions,
+                           float* state, long long state_stride, int n_tokens, int n_requests,
+                           int H, int G, int e, int f, float* out, cudaStream_t stream) {
+    if (n_tokens <= 0 || n_requests <= 0) return 0;
+    const DeltaArgs a = make_args(proj, 1, 0, width, qkv_col, 0, 0, 0, nullptr, 0, taps, nullptr, nullptr,
+                                  state_slot, cu_q, nullptr, positions, state, state_stride,
+                                  n_tokens, n_requests, H, G, e, f);
+    if (!sizes_ok(a) || n_requests > 65535 || H > 65535) return MLS_ERR_UNSUPPORTED;
+    switch (a.er / 32) {
+        case 1: return launch_scan<1>(a, rows, out, stream);
+        case 2: return launch_scan<2>(a, rows, out, stream);
+        case 3: return launch_scan<3>(a, rows, out, stream);
+        case 4: return launch_scan<4>(a, rows, out, stream);
+        case 5: return launch_scan<5>(a, rows, out, stream);
+        case 6: return launch_scan<6>(a, rows, out, stream);
+        case 7: return launch_scan<7>(a, rows, out, stream);
+        default: return launch_scan<8>(a, rows, out, stream);
+    }
+}
+
+// A step of one token a request, to the gated and normed heads: out [T, H f] in `dtype`.
+MLS_API int mls_delta_step(const float* proj, int n_parts, long long part_stride, int width,
+                           int qkv_col, int a_col, int b_col, int g_col, const void* conv,
+                           int conv_dtype, int taps, const float* a_exp, const float* dt_bias,
+                           const float* norm_w, float eps, const int* state_slot, const int* cu_q,
+                           const int* positions, float* state, long long state_stride,
+                           int n_requests, int H, int G, int e, int f, void* out, int dtype,
+                           cudaStream_t stream) {
+    if (n_requests <= 0) return 0;
+    const DeltaArgs a = make_args(proj, n_parts, part_stride, width, qkv_col, a_col, b_col, g_col, conv,
+                                  conv_dtype, taps, a_exp, dt_bias, state_slot, cu_q, nullptr,
+                                  positions, state, state_stride, n_requests, n_requests, H, G, e, f);
+    if (!sizes_ok(a) || n_requests > 65535) return MLS_ERR_UNSUPPORTED;
+    switch (a.er / 32) {
+        case 1: return launch_step<1, 8>(a, norm_w, eps, out, dtype, stream);
+        case 2: return launch_step<2, 8>(a, norm_w, eps, out, dtype, stream);
+        case 3: return launch_step<3, 4>(a, norm_w, eps, out, dtype, stream);
+        case 4: return launch_step<4, 4>(a, norm_w, eps, out, dtype, stream);
+        case 5: return launch_step<5, 2>(a, norm_w, eps, out, dtype, stream);
+        case 6: return launch_step<6, 2>(a, norm_w, eps, out, dtype, stream);
+        case 7: return launch_step<7, 2>(a, norm_w, eps, out, dtype, stream);
+        default: return launch_step<8, 2>(a, norm_w, eps, out, dtype, stream);
+    }
+}

@@ -6,6 +6,8 @@
 //                                                                  the weights [e] serve all heads
 //   q_h <- q_h * (1 + coef * ln(floor((p + 1) / every) + 1))      the query's temperature at
 //                                                                  position p, optional
+//   v <- (1 - lambda) v + lambda v_first           optional: v_first [T, all v entries], float32,
+//                    are the step's values of an earlier layer, which that layer leaves there
 //
 // q goes to the row the attention kernels read ([T, q_width], head h at h * hd), k and v into
 // the pages at the step's slots.  Heads are hd wide in both places: the entries past e (past
@@ -27,7 +29,8 @@ head_prep_kernel(const float* __restrict__ proj, int proj_width, int q_col, int 
                  const float* __restrict__ b_q, const float* __restrict__ b_k,
                  const float* __restrict__ b_v, const float* __restrict__ w_q,
                  const float* __restrict__ w_k, float eps, float temp_coef, int temp_every,
-                 float v_scale, const int* __restrict__ positions,
+                 float v_scale, float* __restrict__ v_first, int v_mode, float v_lambda,
+                 const int* __restrict__ positions,
                  const int* __restrict__ slot_map, T* __restrict__ q_out, int q_width,
                  T* __restrict__ k_pool, T* __restrict__ v_pool, int block_size, int n_pages,
                  int n_tokens, int n_heads, int n_kv, int e, int f, int hd, int writes,
@@ -83,6 +86,11 @@ head_prep_kernel(const float* __restrict__ proj, int proj_width, int q_col, int 
             if (i < width) {
                 x = (src[i] + (bias ? bias[i] : 0.f)) * mul;
                 if (w) x *= w[i];
+                if (kind == 2 && v_mode != 0) {
+                    float* first = v_first + ((size_t)t * n_kv + head) * f + i;
+                    if (v_mode == 1) *first = x;
+                    else x = (1.0f - v_lambda) * x + v_lambda * *first;
+                }
             }
             Elem<T>::store(dst + i, x);
         }
@@ -97,26 +105,29 @@ head_prep_kernel(const float* __restrict__ proj, int proj_width, int q_col, int 
 MLS_API int mls_head_prep_store(const float* proj, int proj_width, int q_col, int k_col, int v_col,
                                 const float* b_q, const float* b_k, const float* b_v,
                                 const float* w_q, const float* w_k, float eps, float temp_coef,
-                                int temp_every, float v_scale, const int* positions,
+                                int temp_every, float v_scale, float* v_first, int v_mode,
+                                float v_lambda, const int* positions,
                                 const int* slot_map, void* q_out, int q_width, int dtype,
                                 void* k_pool, void* v_pool, int block_size, int n_pages,
                                 int n_tokens, int n_heads, int n_kv, int e, int f, int hd,
                                 int writes, int* status, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
-    if (e <= 0 || f <= 0 || hd < e || hd < f || n_heads <= 0 || n_kv <= 0) return MLS_ERR_UNSUPPORTED;
+    if (e <= 0 || f <= 0 || hd < e || hd < f || n_heads <= 0 || n_kv <= 0 ||
+        v_mode < 0 || v_mode > 2 || (v_mode && (!v_first || !writes)))
+        return MLS_ERR_UNSUPPORTED;
     const int units = n_heads + (writes ? 2 * n_kv : 0);
     const int threads = n_tokens > 64 ? HP_THREADS
         : (32 * units < HP_THREADS ? HP_THREADS : (32 * units > HP_MAX_THREADS ? HP_MAX_THREADS : 32 * units));
     if (dtype == MLS_BF16)
         MLS_LAUNCH((head_prep_kernel<__nv_bfloat16>), dim3(n_tokens), dim3(threads), 0, stream,
                    proj, proj_width, q_col, k_col, v_col, b_q, b_k, b_v, w_q, w_k, eps, temp_coef,
-                   temp_every, v_scale, positions, slot_map, (__nv_bfloat16*)q_out, q_width,
+                   temp_every, v_scale, v_first, v_mode, v_lambda, positions, slot_map, (__nv_bfloat16*)q_out, q_width,
                    (__nv_bfloat16*)k_pool, (__nv_bfloat16*)v_pool, block_size, n_pages, n_tokens,
                    n_heads, n_kv, e, f, hd, writes, status);
     else
         MLS_LAUNCH((head_prep_kernel<float>), dim3(n_tokens), dim3(threads), 0, stream, proj,
                    proj_width, q_col, k_col, v_col, b_q, b_k, b_v, w_q, w_k, eps, temp_coef,
-                   temp_every, v_scale, positions, slot_map, (float*)q_out, q_width,
+                   temp_every, v_scale, v_first, v_mode, v_lambda, positions, slot_map, (float*)q_out, q_width,
                    (float*)k_pool, (float*)v_pool, block_size, n_pages, n_tokens, n_heads, n_kv,
                    e, f, hd, writes, status);
     return launch_status();

@@ -96,13 +96,19 @@ struct RowParts {
 };
 
 // Entry i of a vector of n entries whose first `dims` turn, entry j with entry j + dims/2
-// (j < dims/2), by the token's angle j, whose cosine is cs[j] and sine cs[dims/2 + j]; the
-// others pass.  get(j) reads entry j.
+// (j < dims/2; `interleaved`: entry 2j with entry 2j + 1), by the token's angle j, whose cosine
+// is cs[j] and sine cs[dims/2 + j]; the others pass.  get(j) reads entry j.
 template <typename Get>
-__device__ __forceinline__ float rotated_entry(Get get, int i, int dims,
+__device__ __forceinline__ float rotated_entry(Get get, int i, int dims, int interleaved,
                                                const float* __restrict__ cs) {
     const int half = dims >> 1;
     if (i >= dims) return get(i);
+    if (interleaved) {
+        const int j = i >> 1;
+        const float c = cs[j], s = cs[half + j];
+        const float u = get(2 * j), v = get(2 * j + 1);
+        return (i & 1) ? v * c + u * s : u * c - v * s;
+    }
     const int j = i < half ? i : i - half;
     const float c = cs[j], s = cs[half + j];
     const float u = get(j), v = get(j + half);
@@ -159,7 +165,8 @@ __device__ __forceinline__ void store4(__nv_bfloat16* dst, float4 v) {
 template <typename T>
 __global__ void __launch_bounds__(LT_THREADS)
 latent_rope_prep_kernel(const RowParts proj, int q_col, int kv_col, int n_heads, int e, int g,
-                        int r, int rp, int rot_dims, const double* __restrict__ freq,
+                        int r, int rp, int rot_dims, int interleaved,
+                        const double* __restrict__ freq,
                         const int* __restrict__ positions, const void* __restrict__ wkv,
                         int w_dtype, float eps, T* __restrict__ q_plain, T* __restrict__ q_in,
                         int q_in_width, int has_kv, const int* __restrict__ slot_map,
@@ -228,7 +235,7 @@ latent_rope_prep_kernel(const RowParts proj, int q_col, int kv_col, int n_heads,
         if (i < g)
             v = rotated_entry(
                 [&](int j) { return staged ? sq[h * g + j] : proj.at(t, q_col + h * hw + e + j); },
-                i, rot_dims, cs);
+                i, rot_dims, interleaved, cs);
         Elem<T>::store(q_in + (size_t)t * q_in_width + (size_t)h * rp + r + i, v);
     }
     if (!has_kv) return;
@@ -248,13 +255,15 @@ latent_rope_prep_kernel(const RowParts proj, int q_col, int kv_col, int n_heads,
         if (c < r)
             v = down(c) * inv * (staged ? swn[c] : load_as_float(wkv, c, w_dtype));
         else if (c < r + g)
-            v = rotated_entry([&](int j) { return down(r + j); }, c - r, rot_dims, cs);
+            v = rotated_entry([&](int j) { return down(r + j); }, c - r, rot_dims,
+                              interleaved, cs);
         Elem<T>::store(dst + c, v);
     }
     clear_page_tail<T>(tail, slot, block_size, pool_slots / block_size, 1, rp, pool, pool);
 }
 
-// o[t, c] *= sigmoid(gate[t, gate_col + c]), the gate read from a float32 projection row.
+// o[t, c] *= sigmoid(gate[t, gate_col + c / per]), the gate read from a float32 projection row;
+// `per` neighbouring entries share a gate (1: each has its own; a head's size: one a head).
 // by4: four entries a thread where widths and offsets are multiples of four.
 __device__ __forceinline__ float4 load4(const float* src) {
     return *reinterpret_cast<const float4*>(src);
@@ -268,8 +277,8 @@ __device__ __forceinline__ float4 load4(const __nv_bfloat16* src) {
 
 template <typename T>
 __global__ void __launch_bounds__(256)
-sigmoid_gate_kernel(T* __restrict__ o, const RowParts proj, int gate_col, int n_tokens, int n,
-                    int by4) {
+sigmoid_gate_kernel(T* __restrict__ o, const RowParts proj, int gate_col, int per, int n_tokens,
+                    int n, int by4) {
     chain_release();
     chain_wait();
     if (by4) {
@@ -278,7 +287,13 @@ sigmoid_gate_kernel(T* __restrict__ o, const RowParts proj, int gate_col, int n_
         for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total;
              idx += (size_t)gridDim.x * blockDim.x) {
             const int t = (int)(idx / n4), c = (int)(idx - (size_t)t * n4) << 2;
-            const float4 z = row_parts_at4(proj, t, gate_col + c);
+            float4 z;
+            if (per == 1) {
+                z = row_parts_at4(proj, t, gate_col + c);
+            } else {
+                const float one = proj.at(t, gate_col + c / per);
+                z = make_float4(one, one, one, one);
+            }
             T* at = o + (size_t)t * n + c;
             float4 v = load4(at);
             v.x = v.x / (1.0f + expf(-z.x));
@@ -293,7 +308,7 @@ sigmoid_gate_kernel(T* __restrict__ o, const RowParts proj, int gate_col, int n_
     for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total;
          idx += (size_t)gridDim.x * blockDim.x) {
         const int t = (int)(idx / n), c = (int)(idx - (size_t)t * n);
-        const float z = proj.at(t, gate_col + c);
+        const float z = proj.at(t, gate_col + c / per);
         Elem<T>::store(o + idx, Elem<T>::load(o + idx) / (1.0f + expf(-z)));
     }
 }
@@ -395,8 +410,8 @@ MLS_API int mls_headwise_linear(const void* in, long long in_row, long long in_h
 
 MLS_API int mls_latent_rope_prep(const float* proj, int n_parts, long long part_stride,
                                  int proj_width, int q_col, int kv_col, int n_tokens, int n_heads,
-                                 int e, int g, int r, int rp, int rot_dims, const double* freq,
-                                 const int* positions, const void* wkv, int w_dtype, float eps,
+                                 int e, int g, int r, int rp, int rot_dims, int interleaved,
+                                 const double* freq, const int* positions, const void* wkv, int w_dtype, float eps,
                                  void* q_plain, void* q_in, int q_in_width, int dtype, int has_kv,
                                  const int* slot_map, void* pool, int block_size,
                                  long long pool_slots, int* status, cudaStream_t stream) {
@@ -420,34 +435,36 @@ MLS_API int mls_latent_rope_prep(const float* proj, int n_parts, long long part_
                     reinterpret_cast<uintptr_t>(proj) % 16 == 0;
     if (dtype == MLS_BF16)
         MLS_LAUNCH((latent_rope_prep_kernel<__nv_bfloat16>), dim3(n_tokens), dim3(LT_THREADS), smem,
-                   stream, rows, q_col, kv_col, n_heads, e, g, r, rp, rot_dims, freq, positions, wkv,
-                   w_dtype, eps, (__nv_bfloat16*)q_plain, (__nv_bfloat16*)q_in, q_in_width, has_kv,
+                   stream, rows, q_col, kv_col, n_heads, e, g, r, rp, rot_dims, interleaved, freq,
+                   positions, wkv, w_dtype, eps, (__nv_bfloat16*)q_plain, (__nv_bfloat16*)q_in, q_in_width, has_kv,
                    slot_map, (__nv_bfloat16*)pool, block_size, (int)pool_slots, by4, kv4, staged,
                    status);
     else
         MLS_LAUNCH((latent_rope_prep_kernel<float>), dim3(n_tokens), dim3(LT_THREADS), smem, stream,
-                   rows, q_col, kv_col, n_heads, e, g, r, rp, rot_dims, freq, positions, wkv, w_dtype,
-                   eps, (float*)q_plain, (float*)q_in, q_in_width, has_kv, slot_map, (float*)pool,
+                   rows, q_col, kv_col, n_heads, e, g, r, rp, rot_dims, interleaved, freq, positions,
+                   wkv, w_dtype, eps, (float*)q_plain, (float*)q_in, q_in_width, has_kv, slot_map, (float*)pool,
                    block_size, (int)pool_slots, by4, kv4, staged, status);
     return launch_status();
 }
 
 MLS_API int mls_sigmoid_gate(void* o, int dtype, const float* proj, int n_parts,
-                             long long part_stride, int proj_width, int gate_col, int n_tokens,
-                             int n, cudaStream_t stream) {
+                             long long part_stride, int proj_width, int gate_col, int per,
+                             int n_tokens, int n, cudaStream_t stream) {
     if (n_tokens <= 0 || n <= 0) return 0;
-    if (n_parts < 1) return MLS_ERR_UNSUPPORTED;
+    if (n_parts < 1 || per < 1) return MLS_ERR_UNSUPPORTED;
     const RowParts rows{proj, n_parts, part_stride, proj_width};
-    const int by4 = n % 4 == 0 && gate_col % 4 == 0 && proj_width % 4 == 0 && part_stride % 4 == 0 &&
-                    reinterpret_cast<uintptr_t>(proj) % 16 == 0 &&
+    const int by4 = n % 4 == 0 &&
+                    (per == 1 ? gate_col % 4 == 0 && proj_width % 4 == 0 && part_stride % 4 == 0 &&
+                                    reinterpret_cast<uintptr_t>(proj) % 16 == 0
+                              : per % 4 == 0) &&
                     reinterpret_cast<uintptr_t>(o) % 16 == 0;
     const size_t want = ((size_t)n_tokens * (by4 ? n / 4 : n) + 255) / 256;
     const int blocks = (int)(want < (size_t)(8 * sm_count()) ? want : 8 * sm_count());
     if (dtype == MLS_BF16)
         MLS_LAUNCH((sigmoid_gate_kernel<__nv_bfloat16>), dim3(blocks), dim3(256), 0, stream,
-                   (__nv_bfloat16*)o, rows, gate_col, n_tokens, n, by4);
+                   (__nv_bfloat16*)o, rows, gate_col, per, n_tokens, n, by4);
     else
         MLS_LAUNCH((sigmoid_gate_kernel<float>), dim3(blocks), dim3(256), 0, stream, (float*)o, rows,
-                   gate_col, n_tokens, n, by4);
+                   gate_col, per, n_tokens, n, by4);
     return launch_status();
 }

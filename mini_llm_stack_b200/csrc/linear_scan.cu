@@ -218,11 +218,11 @@ linear_scan_kernel(const void* __restrict__ a_src, int a_dtype, int a_row, int a
     }
 }
 
-// One warp a (token, head).
+// One warp a (token, head).  The gate's rows may be float32 whatever the output's type.
 template <typename T>
 __global__ void __launch_bounds__(128)
-scan_finish_kernel(const float* __restrict__ o, const T* __restrict__ gate, int gate_row,
-                   int gate_off, const void* __restrict__ w, int w_dtype, float eps,
+scan_finish_kernel(const float* __restrict__ o, const void* __restrict__ gate, int gate_dtype,
+                   int gate_row, int gate_off, const void* __restrict__ w, int w_dtype, float eps,
                    T* __restrict__ out, int n_tokens, int n_heads, int f) {
     chain_release();
     chain_wait();
@@ -236,7 +236,7 @@ scan_finish_kernel(const float* __restrict__ o, const T* __restrict__ gate, int 
     const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)f + eps);
     for (int j = lane; j < f; j += 32) {
         const int c = head * f + j;
-        const float z = Elem<T>::load(gate + (size_t)t * gate_row + gate_off + c);
+        const float z = load_as_float(gate, (size_t)t * gate_row + gate_off + c, gate_dtype);
         float v = row[j] * inv;
         if (w) v *= load_as_float(w, c, w_dtype);
         Elem<T>::store(out + (size_t)t * n_heads * f + c, v * (z / (1.0f + expf(-z))));
@@ -379,19 +379,19 @@ MLS_API int mls_linear_scan(const void* a_src, int a_dtype, int a_row, int a_off
 #undef LS_GO
 }
 
-MLS_API int mls_scan_finish(const float* o, const void* gate, int act_dtype, int gate_row,
+MLS_API int mls_scan_finish(const float* o, const void* gate, int gate_dtype, int gate_row,
                             int gate_off, const void* w, int w_dtype, float eps, void* out,
-                            int n_tokens, int n_heads, int f, cudaStream_t stream) {
+                            int act_dtype, int n_tokens, int n_heads, int f, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     const long long units = (long long)n_tokens * n_heads;
     const int blocks = (int)((units + 3) / 4);
     if (act_dtype == MLS_BF16)
         MLS_LAUNCH((scan_finish_kernel<__nv_bfloat16>), dim3(blocks), dim3(128), 0, stream, o,
-                   (const __nv_bfloat16*)gate, gate_row, gate_off, w, w_dtype, eps,
+                   gate, gate_dtype, gate_row, gate_off, w, w_dtype, eps,
                    (__nv_bfloat16*)out, n_tokens, n_heads, f);
     else
         MLS_LAUNCH((scan_finish_kernel<float>), dim3(blocks), dim3(128), 0, stream, o,
-                   (const float*)gate, gate_row, gate_off, w, w_dtype, eps, (float*)out, n_tokens,
+                   gate, gate_dtype, gate_row, gate_off, w, w_dtype, eps, (float*)out, n_tokens,
                    n_heads, f);
     return launch_status();
 }

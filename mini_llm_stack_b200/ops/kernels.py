@@ -72,16 +72,18 @@ class SplitParts:
 
     Their sum, taken in the order of the slices, is the product.  ``add_rmsnorm``
     adds them up while it reads the residual row anyway, which saves the kernel
-    that would do nothing else.  The parts live in one scratch buffer of the
-    kernels' owner: they are read (or given up) before the next product that
-    wants the buffer, which otherwise takes the ordinary way.
+    that would do nothing else.  The parts live in a scratch buffer of the
+    kernels' owner (one for each name a product may ask for, ``lend``): they are read (or
+    given up) before the next product that wants the buffer, which otherwise takes the
+    ordinary way.
     """
 
-    __slots__ = ("parts", "_ops")
+    __slots__ = ("parts", "_ops", "_lent")
 
-    def __init__(self, parts, ops):
+    def __init__(self, parts, ops, lent: str = "kept"):
         self.parts = parts
         self._ops = ops
+        self._lent = lent
 
     @property
     def shape(self):
@@ -89,7 +91,7 @@ class SplitParts:
 
     def release(self) -> None:
         if self._ops is not None:
-            self._ops._parts_busy = False
+            self._ops._parts_busy.discard(self._lent)
             self._ops = None
 
     def float(self):
@@ -150,7 +152,7 @@ class Ops:
         self._transposed: dict = {}              # id(weight) -> (weight, its transposed view)
         self._gemm = None
         self._tiles_set = False
-        self._parts_busy = False
+        self._parts_busy: set = set()            # scratch buffers lent to products left as parts
         self.attention_impl = os.environ.get("MLS_B200_ATTENTION", "auto")
         self.gemm_impl = os.environ.get("MLS_B200_GEMM", "auto")
         self.generation = 0          # grows whenever a buffer kernels were given moves
@@ -362,9 +364,10 @@ class Ops:
         fn(("never", "auto", "always").index(mode))
 
     def _gemm_bf16(self, a, w, out, m: int, n: int, k: int, epilogue: int = 0,
-                   leave_parts: bool = False, gate=None):
+                   leave_parts: str | None = None, gate=None):
         """The tcgen05 product.  ``leave_parts``: the K-parts are not added up but
-        returned as ``SplitParts`` (the caller has checked that there are several)."""
+        returned as ``SplitParts`` in the scratch buffer of that name (the caller has checked
+        that there are several)."""
         self._gemm_library()
         if self.gemm_impl == "tcgen05-tiles" or self._tiles_set:
             # prompts of more than 128 rows on one CTA a tile instead of pairs of CTAs
@@ -377,7 +380,7 @@ class Ops:
         if swap:
             splits = self._gemm_splits(m, n, k)
             if splits > 1:
-                tag = "gemm_kept_parts" if leave_parts else "gemm_partials"
+                tag = f"gemm_{leave_parts}_parts" if leave_parts else "gemm_partials"
                 partial = self.scratch(tag, splits * m * n)
                 sums = 0 if leave_parts else 1
         else:
@@ -399,23 +402,24 @@ class Ops:
                           m, n, k, swap, splits, epilogue, _ptr(partial), _ptr(self.status),
                           self._stream()), "gemm_bf16")
         if leave_parts:
-            self._parts_busy = True
-            return SplitParts(partial[:splits * m * n].view(splits, m, n), self)
+            self._parts_busy.add(leave_parts)
+            return SplitParts(partial[:splits * m * n].view(splits, m, n), self, leave_parts)
         return None
 
-    def linear_parts(self, a, w, out):
+    def linear_parts(self, a, w, out, lend: str = "kept"):
         """A product for a consumer that can add up K-parts while it reads its input
         anyway (``add_rmsnorm`` for what goes to the residual stream, ``rope_store``
         for q, k and v): returns ``out``, filled, or the product's parts
-        (``SplitParts``) with ``out`` untouched."""
+        (``SplitParts``) with ``out`` untouched.  ``lend``: the scratch buffer the parts are
+        left in; two products whose parts are wanted at the same time name different ones."""
         m, k = a.shape
         n = w.shape[0]
         if (0 < m <= 64 and n % 4 == 0 and w.dtype == torch.bfloat16
-                and not self._parts_busy
+                and lend not in self._parts_busy
                 and w.shape == (n, k) and a.is_contiguous() and w.is_contiguous()
                 and self._use_own_gemm(m, n, k) and self._gemm_splits(m, n, k) > 1):
             a16 = a if a.dtype == torch.bfloat16 else a.to(torch.bfloat16)
-            return self._gemm_bf16(a16, w, None, m, n, k, leave_parts=True)
+            return self._gemm_bf16(a16, w, None, m, n, k, leave_parts=lend)
         self.linear(a, w, out)
         return out
 
@@ -517,8 +521,8 @@ class Ops:
 
     def require_attention(self, hd: int, n_heads: int = 0, n_kv: int = 0) -> None:
         """Make sure attention kernels for this head size exist, or say why not."""
-        _need(hd % 16 == 0 and 16 <= hd <= 512,
-              f"attention kernels take head sizes 16..512 in steps of 16, not {hd}")
+        _need(hd % 16 == 0 and 16 <= hd <= 1024,
+              f"attention kernels take head sizes 16..1024 in steps of 16, not {hd}")
         if hd > 256:
             return          # beyond the tensor-core kernels: the one-warp-per-row kernel, both types
         if self.act_dtype == torch.bfloat16 and hd not in self._attention_libs:
@@ -553,7 +557,7 @@ class Ops:
 
     def attention_tensor_cores(self, hd: int) -> bool:
         """Whether the tensor-core attention kernels take this step's attention (else
-        the one-warp-per-row kernel does, which takes every head size up to 512)."""
+        the one-warp-per-row kernel does, which takes every head size up to 1024)."""
         return (self.act_dtype == torch.bfloat16 and self.attention_impl != "simt"
                 and hd <= 256 and hd % 16 == 0)
 
@@ -798,8 +802,8 @@ class Ops:
                                  [_P, _I, _I, _I, _P, _I, _P, _LL, _I, _I, _P, _P, _I, _P])}
         elif name == "headprep":
             fns = {"prep": _decl(lib, "mls_head_prep_store",
-                                 [_P, _I, _I, _I, _I, _P, _P, _P, _P, _P, _F, _F, _I, _F, _P, _P, _P,
-                                  _I, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P])}
+                                 [_P, _I, _I, _I, _I, _P, _P, _P, _P, _P, _F, _F, _I, _F, _P, _I, _F,
+                                  _P, _P, _P, _I, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P])}
         elif name == "side":
             fns = {"settle_cast": _decl(lib, "mls_settle_cast",
                                         [_P, _P, _I, _I, _LL, _P, _I, _I, _I, _P]),
@@ -814,11 +818,28 @@ class Ops:
                    "finish_row": _decl(lib, "mls_scan_finish_row",
                                        [_P, _P, _I, _I, _I, _P, _F, _F, _P, _LL, _I, _I, _P]),
                    "finish": _decl(lib, "mls_scan_finish",
-                                   [_P, _P, _I, _I, _I, _P, _I, _F, _P, _I, _I, _I, _P]),
+                                   [_P, _P, _I, _I, _I, _P, _I, _F, _P, _I, _I, _I, _I, _P]),
                    "rotate": _decl(lib, "mls_rotate_rows",
                                    [_P, _I, _I, _I, _I, _P, _P, _I, _F, _P, _I, _I, _I, _P]),
                    "decay": _decl(lib, "mls_decay_lowrank",
                                   [_P, _I, _P, _P, _I, _P, _I, _I, _P])}
+        elif name == "gatednorm":
+            fns = {"add": _decl(lib, "mls_add_gated_norm",
+                                [_P, _P, _I, _I, _LL, _P, _I, _I, _LL, _I, _I, _P, _P, _I, _P, _I, _F,
+                                 _P, _I, _P, _P, _I, _I, _P])}
+        elif name == "delta":
+            fns = {"row": _decl(lib, "mls_delta_row_floats", [_I, _I, _I, _I]),
+                   "state": _decl(lib, "mls_delta_state_floats", [_I, _I, _I, _I, _I],
+                                  restype=ctypes.c_longlong),
+                   "prep": _decl(lib, "mls_delta_prep",
+                                 [_P, _I, _I, _I, _I, _P, _I, _I, _P, _P, _P, _P, _P, _P, _P, _LL, _I,
+                                  _I, _I, _I, _I, _I, _P, _P]),
+                   "scan": _decl(lib, "mls_delta_scan",
+                                 [_P, _P, _I, _I, _I, _P, _P, _P, _P, _LL, _I, _I, _I, _I, _I, _I, _P,
+                                  _P]),
+                   "step": _decl(lib, "mls_delta_step",
+                                 [_P, _I, _LL, _I, _I, _I, _I, _I, _P, _I, _I, _P, _P, _P, _F, _P, _P,
+                                  _P, _P, _LL, _I, _I, _I, _I, _I, _P, _I, _P])}
         else:
             raise KernelError(f"no kernels of a part called {name!r}")
         self._part_libs[name] = fns
@@ -1118,13 +1139,14 @@ class Ops:
 
     def latent_rope_prep(self, proj, q_col: int, kv_col: int, n_heads: int, e: int, g: int,
                          r: int, rp: int, rot_dims: int, freq, w_kv, eps: float, q_plain, q_in,
-                         cache, step) -> None:
+                         cache, step, interleaved: bool = False) -> None:
         """From the float32 projection row ``[... q heads (e plain | g rotated) ... r + g
         down-projected ...]`` (a tensor or ``SplitParts``): the heads' plain parts into
         ``q_plain [T, H * e]``, their rotated parts into ``q_in[t, h * rp + r : + g]`` (zeros up
         to ``rp``), and, if the call writes its cache, ``[unit_rms(down[:r]) * w_kv | rotated
         down[r:] | 0]`` into the pool at the step's slots.  The first ``rot_dims`` of the g
-        entries turn, entry i with i + rot_dims/2, by ``position * freq[i]`` (float64)."""
+        entries turn, entry i with i + rot_dims/2 (``interleaved``: 2i with 2i + 1), by
+        ``position * freq[i]`` (float64)."""
         t = step.n_tokens
         ptr, n_parts, stride, width = self._row_parts(proj, t, "latent_rope_prep")
         writes = bool(cache.writes)
@@ -1141,21 +1163,22 @@ class Ops:
         self.launches += 1
         _check(self._part_lib("latent")["rope_prep"](
             ptr, n_parts, stride, width, q_col, kv_col, t, n_heads, e, g, r, rp, rot_dims,
-            _ptr(freq), _ptr(step.positions), _ptr(w_kv) if writes else None,
+            1 if interleaved else 0, _ptr(freq), _ptr(step.positions), _ptr(w_kv) if writes else None,
             _code(w_kv.dtype) if writes else 0, float(eps), _ptr(q_plain), _ptr(q_in),
             q_in.shape[1], _code(pool.dtype), 1 if writes else 0, _ptr(grp.slot_map), _ptr(pool),
             grp.block_size, pool.shape[1] * pool.shape[2], _ptr(self.status), self._stream()),
             "latent_rope_prep")
 
-    def sigmoid_gate(self, o, proj, gate_col: int) -> None:
-        """``o[t, c] *= sigmoid(proj[t, gate_col + c])``; ``proj`` a float32 tensor or the
-        ``SplitParts`` of its product."""
+    def sigmoid_gate(self, o, proj, gate_col: int, per: int = 1) -> None:
+        """``o[t, c] *= sigmoid(proj[t, gate_col + c // per])`` (``per``: so many neighbouring
+        entries share a gate); ``proj`` a float32 tensor or the ``SplitParts`` of its product."""
         t, n = o.shape
         ptr, n_parts, stride, width = self._row_parts(proj, t, "sigmoid_gate")
-        _need(o.is_contiguous() and gate_col + n <= width, "sigmoid_gate: operands")
+        _need(o.is_contiguous() and per >= 1 and n % per == 0 and gate_col + n // per <= width,
+              "sigmoid_gate: operands")
         self.launches += 1
         _check(self._part_lib("latent")["gate"](
-            _ptr(o), _code(o.dtype), ptr, n_parts, stride, width, gate_col, t, n,
+            _ptr(o), _code(o.dtype), ptr, n_parts, stride, width, gate_col, per, t, n,
             self._stream()), "sigmoid_gate")
 
     def settle_concat(self, x, delta, other, out) -> None:
@@ -1309,18 +1332,19 @@ class Ops:
 
     def scan_finish(self, o, gate, gate_off: int, weight, eps: float, out, n_heads: int,
                     f: int) -> None:
-        """``out = o / rms_per_head(o) * weight * silu(gate)`` (``weight`` may be None)."""
+        """``out = o / rms_per_head(o) * weight * silu(gate)`` (``weight`` may be None; the
+        gate's rows are of ``out``'s type or float32)."""
         t = o.shape[0]
         _need(o.shape == (t, n_heads * f) and o.dtype == torch.float32 and o.is_contiguous()
               and out.shape == (t, n_heads * f) and out.is_contiguous()
-              and out.dtype == gate.dtype and gate.is_contiguous()
+              and gate.dtype in (out.dtype, torch.float32) and gate.is_contiguous()
               and gate.shape[1] >= gate_off + n_heads * f, "scan_finish: operands")
         _need(weight is None or weight.shape == (n_heads * f,), "scan_finish: bad weight")
         self.launches += 1
         _check(self._part_lib("scan")["finish"](
             _ptr(o), _ptr(gate), _code(gate.dtype), gate.shape[1], gate_off, _ptr(weight),
-            _code(weight.dtype) if weight is not None else 0, float(eps), _ptr(out), t, n_heads,
-            f, self._stream()), "scan_finish")
+            _code(weight.dtype) if weight is not None else 0, float(eps), _ptr(out),
+            _code(out.dtype), t, n_heads, f, self._stream()), "scan_finish")
 
     def scan_finish_row(self, o, gate, gate_off: int, weight, eps: float, out,
                         out_scale: float = 1.0) -> None:
@@ -1340,14 +1364,16 @@ class Ops:
 
     def head_prep_store(self, proj, cols: tuple, biases, norms, eps: float, q_temp, v_scale: float,
                         q_out, cache, step, n_heads: int, n_kv: int, e: int, f: int,
-                        hd: int) -> None:
+                        hd: int, v_first=None, v_lambda=None) -> None:
         """From the float32 projection ``proj [T, W]`` with q, k and v heads (``e``, ``e`` and
         ``f`` entries each) from the columns ``cols = (q, k, v)`` on: add ``biases = (b_q, b_k,
         b_v)`` (float32, or None), RMS-normalise every q and k head with ``norms = (w_q, w_k)``
         (float32 [e], or None), multiply q by ``1 + coef * ln(floor((p + 1) / every) + 1)``
         (``q_temp = (coef, every)`` or None) and v by ``v_scale``; q goes to ``q_out`` (head h
         at column ``h * hd``), k and v into the pages at the step's slots, every head padded
-        with zeros to ``hd`` entries; the rest of a page a request enters is cleared."""
+        with zeros to ``hd`` entries; the rest of a page a request enters is cleared.
+        ``v_first [T, G * f]`` float32 with ``v_lambda`` None: the values are left there as well;
+        with a number: they become ``(1 - v_lambda) * v + v_lambda * v_first``."""
         g = step.groups[cache.group]
         t = step.n_tokens
         pool = cache.k_pool
@@ -1366,11 +1392,16 @@ class Ops:
         _need(b_q is None or (b_q.numel() == n_heads * e and b_k.numel() == n_kv * e
                               and b_v.numel() == n_kv * f), "head_prep_store: bad biases")
         _need(w_q is None or (w_q.numel() == e and w_k.numel() == e), "head_prep_store: bad norms")
+        _need(v_first is None or (v_first.shape == (t, n_kv * f) and v_first.dtype == torch.float32
+                                  and v_first.is_contiguous() and cache.writes),
+              "head_prep_store: bad first values")
+        v_mode = 0 if v_first is None else (1 if v_lambda is None else 2)
         coef, every = q_temp if q_temp else (0.0, 0)
         self.launches += 1
         _check(self._part_lib("headprep")["prep"](
             _ptr(proj), proj.shape[1], cols[0], cols[1], cols[2], _ptr(b_q), _ptr(b_k), _ptr(b_v),
             _ptr(w_q), _ptr(w_k), float(eps), float(coef), int(every), float(v_scale),
+            _ptr(v_first), v_mode, float(v_lambda or 0.0),
             _ptr(step.positions), _ptr(g.slot_map), _ptr(q_out), q_out.shape[1], _code(pool.dtype),
             _ptr(pool), _ptr(cache.v_pool), g.block_size, pool.shape[1], t, n_heads, n_kv, e, f,
             hd, 1 if cache.writes else 0, _ptr(self.status), self._stream()), "head_prep_store")
@@ -1417,6 +1448,135 @@ class Ops:
             "rms_scale")
         if isinstance(y, SplitParts):
             y.release()
+
+    def add_gated_norm(self, x, y, gate, gate_bias, post_w, norm_w, eps: float, h, rows=None,
+                       n_rows: int = 0, y_out=None) -> None:
+        """``y`` (a sublayer's result: a tensor or ``SplitParts``) times ``sigmoid(gate +
+        gate_bias)``, RMS-normed with ``post_w``, added to the float32 stream ``x``; ``h`` is the
+        stream's RMS norm with ``norm_w``.  ``gate``: None, ``(float32 or bfloat16 rows, first
+        column)`` or ``SplitParts``; ``gate_bias`` float32 [d] or None.  A norm's weight is
+        float32, a vector [d] or one number.  With ``rows`` only those rows are read and ``x`` stays as
+        it is.  ``x`` None and ``h`` None with ``y_out`` (float32): only the gated and normed
+        ``y`` is written."""
+        src = x if x is not None else y_out
+        t, d = src.shape
+        n_out = t if rows is None else n_rows
+        _need(x is None or (x.dtype == torch.float32 and x.is_contiguous()),
+              "add_gated_norm: x must be float32")
+        _need(h is None or (h.shape == (n_out, d) and h.is_contiguous()), "add_gated_norm: bad output")
+        _need(y_out is None or (y_out.shape == (n_out, d) and y_out.dtype == torch.float32
+                                and y_out.is_contiguous()), "add_gated_norm: bad result")
+        for w in (post_w, norm_w):
+            _need(w is None or (w.dtype == torch.float32 and w.numel() in (1, d) and w.is_contiguous()),
+                  "add_gated_norm: a norm's weight is float32, one number or one a coordinate")
+        _need(gate_bias is None or (gate_bias.dtype == torch.float32 and gate_bias.shape == (d,)
+                                    and gate_bias.is_contiguous()), "add_gated_norm: bad gate bias")
+        _need(rows is None or (rows.dtype == torch.int32 and rows.numel() >= n_rows),
+              "add_gated_norm: bad row indices")
+        yp, ycode, yparts, ystride = self._delta_args(y, t, d, "add_gated_norm")
+        zp, zcode, zparts, zstride, zrow, zcol = None, 0, 1, 0, 0, 0
+        if isinstance(gate, SplitParts):
+            zp, zcode, zparts, zstride = self._delta_args(gate, t, d, "add_gated_norm: gate")
+            zrow = d
+        elif gate is not None:
+            z, zcol = gate
+            _need(z.is_contiguous() and z.shape[0] == t and z.shape[1] >= zcol + d,
+                  "add_gated_norm: bad gate rows")
+            zp, zcode, zrow = z.data_ptr(), _code(z.dtype), z.shape[1]
+        self.launches += 1
+        _check(self._part_lib("gatednorm")["add"](
+            _ptr(x), yp, ycode, yparts, ystride, zp, zcode, zparts, zstride, zrow, zcol,
+            _ptr(gate_bias), _ptr(post_w), 1 if post_w.numel() > 1 else 0, _ptr(norm_w),
+            1 if norm_w is not None and norm_w.numel() > 1 else 0, float(eps), _ptr(h),
+            _code(h.dtype) if h is not None else 0, _ptr(y_out), _ptr(rows), n_out, d,
+            self._stream()), "add_gated_norm")
+        for p in (y, gate):
+            if isinstance(p, SplitParts):
+                p.release()
+
+    def delta_rows(self, n_heads: int, n_kv: int, e: int, f: int) -> int:
+        """Floats of a token's prepared row (``delta_prep``)."""
+        return int(self._part_lib("delta")["row"](n_heads, n_kv, e, f))
+
+    def delta_state_floats(self, n_heads: int, n_kv: int, e: int, f: int, taps: int) -> int:
+        """Floats of a request's state: the matrices and the convolution's inputs."""
+        return int(self._part_lib("delta")["state"](n_heads, n_kv, e, f, taps))
+
+    def _delta_need(self, conv, taps: int, state, n_heads: int, n_kv: int, e: int, f: int,
+                    what: str) -> None:
+        c = 2 * n_kv * e + n_heads * f
+        _need(n_heads % n_kv == 0 and conv.shape == (c, taps) and conv.is_contiguous(),
+              f"{what}: bad convolution weights")
+        _need(state.dtype == torch.float32 and state.stride(1) == 1
+              and state.shape[1] >= self.delta_state_floats(n_heads, n_kv, e, f, taps),
+              f"{what}: bad state")
+
+    def delta_prep(self, proj, cols: tuple, conv, taps: int, a_exp, dt_bias, state, step,
+                   n_heads: int, n_kv: int, e: int, f: int, rows) -> None:
+        """From float32 projection rows with ``[q heads | k heads | v heads]`` from column
+        ``cols[0]`` on, the decay's and the step size's pre-activations (one a head) at ``cols[1]``
+        and ``cols[2]``: convolution over time (``conv [channels, taps]``; inputs before the step
+        from ``state``), silu, q and k as unit vectors (q times e^-1/2), the decay
+        ``exp(-a_exp * softplus(a + dt_bias))`` and ``sigmoid(b)``, as ``rows`` for
+        ``delta_scan``."""
+        t = step.n_tokens
+        self._delta_need(conv, taps, state, n_heads, n_kv, e, f, "delta_prep")
+        _need(proj.dtype == torch.float32 and proj.is_contiguous() and proj.shape[0] == t
+              and proj.shape[1] >= max(cols[0] + conv.shape[0], cols[1] + n_heads, cols[2] + n_heads),
+              "delta_prep: bad projection")
+        _need(a_exp.shape == dt_bias.shape == (n_heads,) and a_exp.dtype == dt_bias.dtype
+              == torch.float32, "delta_prep: bad decay parameters")
+        _need(rows.dtype == torch.float32 and rows.is_contiguous()
+              and rows.shape == (t, self.delta_rows(n_heads, n_kv, e, f)), "delta_prep: bad rows")
+        self.launches += 1
+        _check(self._part_lib("delta")["prep"](
+            _ptr(proj), proj.shape[1], cols[0], cols[1], cols[2], _ptr(conv), _code(conv.dtype), taps,
+            _ptr(a_exp), _ptr(dt_bias), _ptr(step.state_slot), _ptr(step.cu_q),
+            _ptr(step.req_of_token), _ptr(step.positions), _ptr(state), state.stride(0), t,
+            step.n_requests, n_heads, n_kv, e, f, _ptr(rows), self._stream()), "delta_prep")
+
+    def delta_scan(self, rows, proj, col: int, taps: int, state, step, n_heads: int, n_kv: int,
+                   e: int, f: int, out) -> None:
+        """Walk every request's tokens through ``S <- g S; u = b (v - S^T k); S <- S + k u^T;
+        o = S^T q``: ``rows`` from ``delta_prep``, ``out [T, H * f]`` float32.  Also keeps the
+        convolution's last inputs, the q | k | v columns of ``proj`` from ``col`` on."""
+        t = step.n_tokens
+        _need(rows.dtype == torch.float32 and rows.is_contiguous()
+              and rows.shape == (t, self.delta_rows(n_heads, n_kv, e, f)), "delta_scan: bad rows")
+        _need(proj.dtype == torch.float32 and proj.is_contiguous() and proj.shape[0] == t
+              and proj.shape[1] >= col + 2 * n_kv * e + n_heads * f, "delta_scan: bad projection")
+        _need(state.dtype == torch.float32 and state.stride(1) == 1
+              and state.shape[1] >= self.delta_state_floats(n_heads, n_kv, e, f, taps),
+              "delta_scan: bad state")
+        _need(out.shape == (t, n_heads * f) and out.dtype == torch.float32 and out.is_contiguous(),
+              "delta_scan: bad out")
+        self.launches += 1
+        _check(self._part_lib("delta")["scan"](
+            _ptr(rows), _ptr(proj), proj.shape[1], col, taps, _ptr(step.state_slot), _ptr(step.cu_q),
+            _ptr(step.positions), _ptr(state), state.stride(0), t, step.n_requests, n_heads, n_kv, e,
+            f, _ptr(out), self._stream()), "delta_scan")
+
+    def delta_step(self, proj, cols: tuple, conv, taps: int, a_exp, dt_bias, norm_w, eps: float,
+                   state, step, n_heads: int, n_kv: int, e: int, f: int, out) -> None:
+        """A step of one token a request in one kernel: ``delta_prep``, ``delta_scan`` and the
+        head norm (``norm_w [f]``, float32, for all heads) with the silu gate, whose pre-activation
+        starts at ``cols[3]``.  ``proj``: a float32 tensor or the ``SplitParts`` of its product."""
+        t = step.n_tokens
+        ptr, n_parts, stride, width = self._row_parts(proj, t, "delta_step")
+        self._delta_need(conv, taps, state, n_heads, n_kv, e, f, "delta_step")
+        _need(step.max_q_len == 1 and t == step.n_requests, "delta_step: single tokens only")
+        _need(width >= max(cols[0] + conv.shape[0], cols[1] + n_heads, cols[2] + n_heads,
+                           cols[3] + n_heads * f), "delta_step: bad projection")
+        _need(a_exp.shape == dt_bias.shape == (n_heads,) and a_exp.dtype == dt_bias.dtype
+              == norm_w.dtype == torch.float32 and norm_w.shape == (f,), "delta_step: bad parameters")
+        _need(out.shape == (t, n_heads * f) and out.is_contiguous(), "delta_step: bad out")
+        self.launches += 1
+        _check(self._part_lib("delta")["step"](
+            ptr, n_parts, stride, width, cols[0], cols[1], cols[2], cols[3], _ptr(conv),
+            _code(conv.dtype), taps, _ptr(a_exp), _ptr(dt_bias), _ptr(norm_w), float(eps),
+            _ptr(step.state_slot), _ptr(step.cu_q), _ptr(step.positions), _ptr(state),
+            state.stride(0), step.n_requests, n_heads, n_kv, e, f, _ptr(out), _code(out.dtype),
+            self._stream()), "delta_step")
 
     def rotate_rows(self, src, q_off: int, k_off: int, positions, freq, dims: int,
                     k_scale: float, out, n_heads: int, e: int) -> None:

@@ -51,6 +51,8 @@ MODULES = {
     "scan": ["linear_scan.cu"],
     "headprep": ["head_prep.cu"],
     "side": ["side_input.cu"],
+    "gatednorm": ["gated_norm.cu"],
+    "delta": ["delta_rule.cu"],
 }
 
 
@@ -63,7 +65,8 @@ def all_modules(head_sizes=()) -> list:
         out.append(("gemm", {}))
     out.append(("argmax_static", {}))
     out += [(name, {}) for name in ("layernorm", "tanhnorm", "latent", "mlstm", "experts",
-                                    "shortconv", "scan", "headprep", "side")]
+                                    "shortconv", "scan", "headprep", "side", "gatednorm",
+                                    "delta")]
     return out
 
 

@@ -17,7 +17,7 @@ from dataclasses import dataclass
 
 import torch
 
-from .base import CacheHandle, Mixer, PagedKV, StepContext, TensorSpec
+from .base import CacheHandle, Mixer, PagedKV, StepContext, TensorSpec, stack_rows
 
 
 @dataclass(frozen=True)
@@ -203,6 +203,18 @@ def distance_slopes(n_heads: int) -> list:
     return [2.0 ** (-8.0 * (h + 1) / n_heads) for h in range(n_heads)]
 
 
+class FirstValues:
+    """The values one layer leaves for later layers of the same step to mix into theirs: float32
+    rows ``[T, kv heads * value size]``, before the cache's rounding.  Nothing of it outlives a
+    step.  The mixers that share it are built with it; the one that runs first fills it."""
+
+    def __init__(self, n_kv_heads: int, v_dim: int, name: str = "first_values"):
+        self.width, self.name = int(n_kv_heads) * int(v_dim), name
+
+    def rows(self, runtime, n_tokens: int):
+        return runtime.buffer(self.name, (n_tokens, self.width), torch.float32)
+
+
 class UnrotatedAttention(Mixer):
     """Grouped-query attention in which nothing is rotated; positions enter through options.
 
@@ -214,7 +226,11 @@ class UnrotatedAttention(Mixer):
         q <- q * (1 + coef * ln(floor((p + 1) / every) + 1))   ``q_temp = (coef, every)``
         score_ij = (q_i . k_j) * scale - slope_h * (i - j)     ``slopes`` (one a head)
         j visible to i iff j <= i and (i - j < window or j < keep_first)
-        softmax over the visible keys, with ``zero_sink`` plus one term exp(0) without a value
+        v <- (1 - lambda) v + lambda v_first      ``first_values``: v_first the values of the
+                                                  layer that fills it (``fills_first``), for the
+                                                  same token; the mixed v is cached
+        softmax over the visible keys, with ``zero_sink`` plus one term exp(0) without a value,
+        with ``sink`` plus one term exp(sink_h), a learned number a head that is not scaled
         o <- o * sigmoid(W_g h)                   element by element (``gate``)
         out = W_o concat_h(o)
 
@@ -227,12 +243,14 @@ class UnrotatedAttention(Mixer):
     one, and ``padded_columns`` says how that mixer's projection has to be laid out."""
 
     decode_capturable = prompt_capturable = True   # forward only launches kernels on the current stream
+    takes_rider = True
 
     def __init__(self, d_model: int, n_heads: int, n_kv_heads: int, head_dim: int, v_dim: int,
                  scale: float, eps: float = 1e-6, window=None, keep_first: int = 0,
                  qkv_bias: bool = False, head_norm: bool = False, slopes=None,
                  zero_sink: bool = False, q_temp=None, gate: bool = False, v_scale: float = 1.0,
-                 project: bool = True):
+                 project: bool = True, sink: bool = False, first_values=None,
+                 fills_first: bool = False):
         if n_heads % n_kv_heads:
             raise ValueError("n_heads must be a multiple of n_kv_heads")
         if slopes is not None and len(slopes) != n_heads:
@@ -247,6 +265,14 @@ class UnrotatedAttention(Mixer):
         self.zero_sink, self.gate = bool(zero_sink), bool(gate)
         self.q_temp = (float(q_temp[0]), int(q_temp[1])) if q_temp else None
         self.v_scale, self.project = float(v_scale), bool(project)
+        self.has_sink = bool(sink)
+        if self.has_sink and self.zero_sink:
+            raise ValueError("one sink a head, learned or zero")
+        self.first_values, self.fills_first = first_values, bool(fills_first)
+        if first_values is not None and first_values.width != self.n_kv_heads * self.v_dim:
+            raise ValueError("layers that mix their values have as many values a token")
+        self.mix_share = None
+        self.rider_col, self._rider_rows = -1, None
         self.pad_dim = -(-max(self.head_dim, self.v_dim) // 16) * 16     # the kernels' head size
         self.out_width = self.n_heads * self.pad_dim
 
@@ -261,6 +287,11 @@ class UnrotatedAttention(Mixer):
         if self.head_norm:
             out.update({"q.norm": TensorSpec((e,), kind="vector", init="ones"),
                         "k.norm": TensorSpec((e,), kind="vector", init="ones")})
+        if self.first_values is not None:
+            # (the layer that fills it has the number too and does not use it)
+            out["vmix"] = TensorSpec((), kind="vector", init="zeros")
+        if self.has_sink:
+            out["sink"] = TensorSpec((self.n_heads,), kind="vector", init="zeros")
         if self.gate:
             out["g"] = TensorSpec((self.n_heads * f, d))
         if self.project:
@@ -282,16 +313,17 @@ class UnrotatedAttention(Mixer):
         """``w_o [d, H * f]`` with zero columns where the heads' outputs are padded."""
         return self.pad_rows(w_o.t().contiguous()).t().contiguous()
 
-    def bind(self, tensors: dict, runtime) -> None:
+    def bind(self, tensors: dict, runtime, rider=None) -> None:
         self.runtime = runtime
         ops = runtime.ops
         parts = [tensors["q"], tensors["k"], tensors["v"]]
         if self.gate:
             parts.append(self.pad_rows(tensors["g"]))
-        if len({p.dtype for p in parts}) > 1:
-            parts = [p.float() for p in parts]
-        # one projection for everything that reads the mixer's input: [q | k | v | gate]
-        self.w_in = ops.prepare_weight(torch.cat(parts, dim=0))
+        if rider is not None:
+            self.rider_col = sum(p.shape[0] for p in parts)
+            parts.append(rider)
+        # one projection for everything that reads the mixer's input: [q | k | v | gate | rider]
+        self.w_in = ops.prepare_weight(stack_rows(parts, 8 if rider is not None else 1))
         cq, ck = self.n_heads * self.head_dim, self.n_kv_heads * self.head_dim
         self.cols = (0, cq, cq + ck)
         self.gate_col = cq + ck + self.n_kv_heads * self.v_dim
@@ -304,6 +336,10 @@ class UnrotatedAttention(Mixer):
                        if self.slope_values is not None else None)
         self.sink = (torch.zeros(self.n_heads, dtype=f32, device=runtime.device)
                      if self.zero_sink else None)
+        if self.has_sink:
+            self.sink = tensors["sink"].to(f32).contiguous()
+        if self.first_values is not None and not self.fills_first:
+            self.mix_share = float(tensors["vmix"])          # read once, at load time
         if self.project:
             self.w_o = ops.prepare_weight(self.padded_columns(tensors["o"]))
         ops.require_part("headprep")
@@ -333,9 +369,12 @@ class UnrotatedAttention(Mixer):
         proj = rt.buffer("attn_proj", (t, self.w_in.shape[0]), torch.float32)
         ops.linear(h, self.w_in, proj)
         q_row = rt.buffer("qkv", (t, (self.n_heads + 2 * self.n_kv_heads) * hd), rt.act_dtype)
+        self._rider_rows = proj
+        first = self.first_values.rows(rt, t) if self.first_values is not None else None
         ops.head_prep_store(proj, self.cols, self.biases, self.norms, self.eps, self.q_temp,
                             self.v_scale, q_row, cache, step, self.n_heads, self.n_kv_heads,
-                            self.head_dim, self.v_dim, hd)
+                            self.head_dim, self.v_dim, hd, v_first=first,
+                            v_lambda=self.mix_share)
         ops.paged_attention(q_row, out, cache, step, self.n_heads, self.n_kv_heads, hd, self.scale,
                             self.window or 0, plan=self.plan(step), sink=self.sink,
                             slopes=self.slopes, keep_first=self.keep_first,
@@ -351,3 +390,6 @@ class UnrotatedAttention(Mixer):
         self.heads(h, step, cache, o)
         delta = rt.buffer("delta", (step.n_tokens, self.d_model), rt.act_dtype)
         return rt.ops.linear_parts(o, self.w_o, delta)
+
+    def rider(self):
+        return self._rider_rows, self.rider_col

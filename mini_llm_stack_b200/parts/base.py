@@ -225,11 +225,29 @@ class Norm(Part):
 
 
 class Mixer(Part):
+    """A mixer with ``takes_rider`` lets a weight ``[n, d_model]`` of its block ride on the product
+    that reads the mixer's input anyway (``bind(tensors, runtime, rider=weight)``); after
+    ``forward``, ``rider()`` gives ``(float32 rows [T, *], first column)`` of its n results,
+    which stay readable until the next mixer of the kind runs."""
+
+    takes_rider = False
+
     def cache_spec(self):
         return None
 
     def forward(self, h, step: StepContext, cache: CacheHandle):
         raise NotImplementedError
+
+
+def stack_rows(matrices: list, multiple: int = 8):
+    """Matrices ``[n_i, k]`` on top of one another, zero rows below up to a multiple of
+    ``multiple`` (a row of the product then starts at a 16-byte place)."""
+    if len({m.dtype for m in matrices}) > 1:
+        matrices = [m.float() for m in matrices]
+    n = sum(m.shape[0] for m in matrices)
+    if n % multiple:
+        matrices = [*matrices, matrices[0].new_zeros((multiple - n % multiple, matrices[0].shape[1]))]
+    return torch.cat(matrices, dim=0)
 
 
 class FeedForward(Part):

@@ -1,5 +1,5 @@
-"""The arrangement of a layer's parts: the pre-norm residual block, and the block with a norm
-before and behind every sublayer.
+"""The arrangement of a layer's parts: the pre-norm residual block, the block with a norm before
+and behind every sublayer, and that block with a gate on every sublayer's result.
 
 Reference (train/model.py:200-217): ``x = x + mixer(norm_a(x))``;
 ``x = x + feed_forward(norm_b(x))``.  The block owns the order and the names
@@ -8,7 +8,9 @@ its parts' tensors carry in a weight file; the parts own the math.
 
 from __future__ import annotations
 
-from .base import CacheHandle, Part, ResidualStream, StepContext
+import torch
+
+from .base import CacheHandle, Part, ResidualStream, StepContext, TensorSpec
 
 
 def join_name(prefix: str, name: str) -> str:
@@ -119,7 +121,6 @@ class SandwichBlock(PreNormBlock):
         return [(n, p) for n, p in zip(self.names, parts) if p is not None]
 
     def tensor_specs(self) -> dict:
-        from .base import TensorSpec
         out = super().tensor_specs()
         if self.scale_names is not None:
             out[self.scale_names[0]] = TensorSpec((self.d_model,), kind="vector", init="ones")
@@ -147,3 +148,69 @@ class SandwichBlock(PreNormBlock):
             return
         h = self.ffn_norm.forward(stream)
         self._push(stream, self.ffn_post, self.ffn.forward(h, step), self.scales[1])
+
+
+class GatedSandwichBlock(SandwichBlock):
+    """A norm before and behind each sublayer and a full gate on its result: with
+    ``h = pre(x)``, ``x <- x + post(sublayer(h) * sigmoid(W h + b))`` for the mixer, then for the
+    feed-forward.  The gate, the norm behind the sublayer, the sum and the next norm are one
+    kernel (``RMSNorm.gated``).  The mixer's gate rides on the product that reads the mixer's
+    input where the mixer allows it (``Mixer.takes_rider``); the feed-forward's is a product of
+    its own whose K-parts may be left to that kernel.
+
+    ``gate_names``: prefixes of the two gates' matrices; their biases carry ``.b`` behind it."""
+
+    def __init__(self, mixer_norm, mixer, mixer_post, ffn_norm, ffn, ffn_post, d_model: int,
+                 names=("norm1", "mix", "norm1b", "norm2", "mlp", "norm2b"),
+                 gate_names=("rg1", "rg2")):
+        super().__init__(mixer_norm, mixer, mixer_post, ffn_norm, ffn, ffn_post, d_model,
+                         names=names, scale_names=None)
+        self.gate_names = tuple(gate_names)
+        self.gate_w, self.gate_b = [None, None], [None, None]
+
+    def _gates(self):
+        return self.gate_names if self.ffn is not None else self.gate_names[:1]
+
+    def tensor_specs(self) -> dict:
+        out = super().tensor_specs()
+        d = self.d_model
+        for n in self._gates():
+            out[n] = TensorSpec((d, d))
+            out[join_name(n, "b")] = TensorSpec((d,), kind="vector", init="zeros")
+        return out
+
+    def bind(self, tensors: dict, runtime) -> None:
+        self.runtime = runtime
+        self.gate_w, self.gate_b = [None, None], [None, None]
+        for i, n in enumerate(self._gates()):
+            self.gate_w[i] = tensors[n]
+            self.gate_b[i] = tensors[join_name(n, "b")].float().contiguous()
+        for prefix, part in self._named_parts():
+            mine = under_prefix(tensors, prefix)
+            if part is self.mixer and part.takes_rider:
+                part.bind(mine, runtime, rider=self.gate_w[0])
+                self.gate_w[0] = None
+            else:
+                part.bind(mine, runtime)
+        self.gate_w = [None if w is None else runtime.ops.prepare_weight(w) for w in self.gate_w]
+        runtime.ops.require_part("gatednorm")
+
+    def _gate(self, i: int, h):
+        """The gate's pre-activation as a product of its own (maybe left as its K-parts)."""
+        rt = self.runtime
+        z = rt.buffer("residual_gate", (h.shape[0], self.d_model), torch.float32)
+        got = rt.ops.linear_parts(h, self.gate_w[i], z, lend="gate")
+        return (z, 0) if got is z else got
+
+    def forward(self, stream: ResidualStream, step: StepContext, cache: CacheHandle) -> None:
+        h = self.mixer_norm.forward(stream)
+        gate = self._gate(0, h) if self.gate_w[0] is not None else None
+        y = self.mixer.forward(h, step, cache)
+        if isinstance(y, tuple):
+            raise TypeError("a mixer with an output bias does not fit a gated block")
+        stream.push(self.mixer_post.gated(y, gate or self.mixer.rider(), self.gate_b[0]))
+        if self.ffn is None:
+            return
+        h = self.ffn_norm.forward(stream)
+        gate = self._gate(1, h)
+        stream.push(self.ffn_post.gated(self.ffn.forward(h, step), gate, self.gate_b[1]))

@@ -20,7 +20,7 @@ from __future__ import annotations
 import torch
 
 from .attention import plan_paged_attention
-from .base import CacheHandle, Mixer, PagedKV, StepContext, TensorSpec
+from .base import CacheHandle, Mixer, PagedKV, StepContext, TensorSpec, stack_rows
 
 
 class LatentAttention(Mixer):
@@ -115,7 +115,7 @@ class RotaryLatentAttention(Mixer):
                                                  entries) rotated: one key part for all heads
         score_h(i, j) = (a_hi . W_uk[h] c_j + b_hi . k_j) * scale,   0 <= i - j < window
         p = exp(score) / (sum_j exp(score) + exp(sink_h));   o_h = sum_j p_j W_uv[h] c_j
-        out = W_o (concat_h o_h * sigmoid(W_g x))
+        out = W_o (concat_h o_h * sigmoid(W_g x))       (``gate="head"``: one gate entry a head)
 
     Only ``[c | k]`` is cached (``PagedKV(1, r + g rounded up, shared_kv=True)``), and keys
     and values are never rebuilt: the query's plain part is taken into the latent space
@@ -124,24 +124,29 @@ class RotaryLatentAttention(Mixer):
     weighted latent.  A mixer with ``own_cache=False`` has no ``W_dkv``: its call reads the
     slot another layer's call fills (``LayerCall.writes`` False).  ``cache_window``: how many
     of the latest tokens the cache keeps (at least ``window``; larger when a reader of this
-    cache sees further back; None: all).  ``position``: a ``PartialRotary`` with the "half"
-    pairing over the first ``position.dims`` of the g entries, or None."""
+    cache sees further back; None: all).  ``position``: a ``PartialRotary`` (either pairing) over
+    the first ``position.dims`` of the g entries, or None."""
 
     decode_capturable = prompt_capturable = True
+    takes_rider = True
     PAD = 16
 
     def __init__(self, d_model: int, n_heads: int, qk_dim: int, rot_dim: int, v_dim: int,
                  kv_rank: int, scale: float, eps: float, position=None, window=None,
-                 sink: bool = True, gate: bool = True, own_cache: bool = True,
+                 sink: bool = True, gate=True, own_cache: bool = True,
                  cache_window=None):
         self.d_model, self.n_heads = int(d_model), int(n_heads)
         self.qk_dim, self.rot_dim, self.v_dim = int(qk_dim), int(rot_dim), int(v_dim)
         self.kv_rank, self.scale, self.eps = int(kv_rank), float(scale), float(eps)
         self.position, self.window = position, window
+        if gate not in (True, False, None, "head"):
+            raise ValueError(f"gate: one entry a value (True), one a head ('head') or none, not {gate!r}")
         self.has_sink, self.has_gate, self.own_cache = bool(sink), bool(gate), bool(own_cache)
+        self.gate_per = self.v_dim if gate == "head" else 1     # values that share a gate entry
+        self.rider_col, self._rider_rows = -1, None
         self.cache_window = cache_window if own_cache else None
-        if position is not None and (position.pairing != "half" or position.dims > self.rot_dim):
-            raise ValueError("the rotated part turns entry i with entry i + dims/2, dims <= rot_dim")
+        if position is not None and position.dims > self.rot_dim:
+            raise ValueError("the rotated part turns its first dims entries, dims <= rot_dim")
         if own_cache and window is not None and cache_window is not None and cache_window < window:
             raise ValueError("the cache keeps fewer tokens than the window sees")
         width = self.kv_rank + self.rot_dim
@@ -158,7 +163,7 @@ class RotaryLatentAttention(Mixer):
         if self.has_sink:
             out["sink"] = TensorSpec((h,), kind="vector", init="zeros")
         if self.has_gate:
-            out["g"] = TensorSpec((h * self.v_dim, d))
+            out["g"] = TensorSpec((h * self.v_dim // self.gate_per, d))
         out["o"] = TensorSpec((d, h * self.v_dim))
         return out
 
@@ -167,24 +172,29 @@ class RotaryLatentAttention(Mixer):
             return None
         return PagedKV(1, self.pool_width, self.cache_window, shared_kv=True)
 
-    def bind(self, tensors: dict, runtime) -> None:
+    def bind(self, tensors: dict, runtime, rider=None) -> None:
         self.runtime = runtime
         ops = runtime.ops
         h, e, f, r = self.n_heads, self.qk_dim, self.v_dim, self.kv_rank
-        # one product for everything that reads the mixer's input: [q | gate | down]
-        rows = [tensors["q"]]
-        self.gate_col = self.kv_col = -1
-        at = rows[0].shape[0]
-        if self.has_gate:
-            rows.append(tensors["g"])
-            self.gate_col, at = at, at + rows[-1].shape[0]
+        # one product for everything that reads the mixer's input: [q | gate | down | rider], a
+        # gate of one entry a head last (the other columns then start where whole heads end)
+        named = [("q", tensors["q"])]
+        if self.has_gate and self.gate_per == 1:
+            named.append(("gate", tensors["g"]))
         if self.own_cache:
-            rows.append(tensors["dkv"])
-            self.kv_col, at = at, at + rows[-1].shape[0]
-        if len({t.dtype for t in rows}) > 1:
-            rows = [t.float() for t in rows]
-        self.w_in = ops.prepare_weight(torch.cat(rows, dim=0))
-        self.in_width = at
+            named.append(("kv", tensors["dkv"]))
+        if rider is not None:
+            named.append(("rider", rider))
+        if self.has_gate and self.gate_per > 1:
+            named.append(("gate", tensors["g"]))
+        cols, at = {}, 0
+        for name, w in named:
+            cols[name], at = at, at + w.shape[0]
+        self.gate_col, self.kv_col = cols.get("gate", -1), cols.get("kv", -1)
+        self.rider_col = cols.get("rider", -1)
+        aligned = 8 if (rider is not None or self.gate_per > 1) else 1
+        self.w_in = ops.prepare_weight(stack_rows([w for _, w in named], aligned))
+        self.in_width = self.w_in.shape[0]
         self.w_norm = tensors["dkv.norm"].contiguous() if self.own_cache else None
         # W_uk[h]^T as [H, r, e] and W_uv[h] as [H, f, r]
         self.w_into = tensors["uk"].view(h, e, r).transpose(1, 2).contiguous()
@@ -216,14 +226,19 @@ class RotaryLatentAttention(Mixer):
                                "without reads another call's")
         # float32 rows: the norm of the latent, the rotation and the gate see no 16-bit rounding
         proj = rt.buffer("latent_in", (t, self.in_width), torch.float32)
-        proj = ops.linear_parts(h, self.w_in, proj)
+        if self.rider_col >= 0:
+            ops.linear(h, self.w_in, proj)           # read once more after the output product
+            self._rider_rows = proj
+        else:
+            proj = ops.linear_parts(h, self.w_in, proj)
         q_plain = rt.buffer("latent_q_plain", (t, nh * e), rt.act_dtype)
         # the kernels read a row of [q heads | k heads | v heads]; only the q heads are there
         q_in = rt.buffer("latent_q_in", (t, (nh + 2) * rp), rt.act_dtype)
         pos = self.position
         ops.latent_rope_prep(proj, 0, self.kv_col, nh, e, g, r, rp, pos.dims if pos else 0,
                              pos.freq if pos else None, self.w_norm, self.eps, q_plain, q_in,
-                             cache, step)
+                             cache, step,
+                             interleaved=bool(pos) and pos.pairing == "interleaved")
         ops.headwise_linear(q_plain, e, self.w_into, q_in, rp, t)
         o_in = rt.buffer("latent_o_in", (t, nh * rp), rt.act_dtype)
         ops.paged_attention(q_in, o_in, cache, step, nh, 1, rp, self.scale, self.window or 0,
@@ -231,8 +246,11 @@ class RotaryLatentAttention(Mixer):
         o = rt.buffer("attn_out", (t, nh * f), rt.act_dtype)
         ops.headwise_linear(o_in, rp, self.w_out_of, o, f, t)
         if self.has_gate:
-            ops.sigmoid_gate(o, proj, self.gate_col)
+            ops.sigmoid_gate(o, proj, self.gate_col, per=self.gate_per)
         if hasattr(proj, "release"):
             proj.release()
         delta = rt.buffer("delta", (t, self.d_model), rt.act_dtype)
         return ops.linear_parts(o, self.w_o, delta)
+
+    def rider(self):
+        return self._rider_rows, self.rider_col

@@ -1,4 +1,5 @@
-"""Mixers that carry a matrix state per head from token to token: wkv and retention.
+"""Mixers that carry a matrix state per head from token to token: wkv, retention, lightning
+attention and the gated delta rule.
 
 Both keep ``S [e, f]`` per head (key size e, value size f) in the request's state slot
 (``FixedState``, float32, zero when the slot is claimed) and walk a step's tokens through
@@ -25,7 +26,7 @@ from __future__ import annotations
 
 import torch
 
-from .base import CacheHandle, FixedState, Mixer, StepContext, TensorSpec
+from .base import CacheHandle, FixedState, Mixer, StepContext, TensorSpec, stack_rows
 
 
 class WkvMixer(Mixer):
@@ -235,3 +236,115 @@ class LightningAttention(Mixer):
         self.heads(h, step, cache, y)
         delta = rt.buffer("delta", (step.n_tokens, self.d_model), rt.act_dtype)
         return rt.ops.linear_parts(y, self.w_o, delta)
+
+
+class GatedDeltaMixer(Mixer):
+    """The gated delta rule: the state forgets what it holds under the token's key before it
+    takes the token's value in.
+
+    With H value heads of size f and G key heads of size e (value head h reads key head
+    ``h // (H/G)``), per token:
+
+        q, k, v = silu(conv(W_q h)), silu(conv(W_k h)), silu(conv(W_v h))   causal, ``taps`` taps a channel
+        q, k <- q / |q| * e^-1/2, k / |k|              |x| = sqrt(sum(x^2) + 1e-6), per head
+        b = sigmoid(W_b h);   g = exp(-exp(A_log) * softplus(W_a h + dt_bias))    one a value head
+        S <- g S;   u = b (v - S^T k);   S <- S + k u^T;   o = S^T q
+        out = W_o (o / rms_per_head(o) * w * silu(W_g h))            w [f] for all heads
+
+    State and convolution inputs live in the request's state slot (float32; layout in
+    ``csrc/delta_rule.cu``).  One product, float32 out, reads the mixer's input: ``[q | k | v |
+    gate | rider | b | a]``; everything from there to the gated heads is float32.  A step of one
+    token a request runs as one kernel between the two products; other steps prepare their
+    rows, walk them through the state and finish them in three."""
+
+    decode_capturable = prompt_capturable = True
+    takes_rider = True
+    MAX_TAPS, MAX_SIZE = 16, 256
+
+    def __init__(self, d_model: int, n_heads: int, n_kv_heads: int, qk_dim: int, v_dim: int,
+                 taps: int, eps: float):
+        if n_heads % n_kv_heads:
+            raise ValueError("n_heads must be a multiple of n_kv_heads")
+        if not 1 <= taps <= self.MAX_TAPS or not 0 < qk_dim <= self.MAX_SIZE or \
+                not 0 < v_dim <= self.MAX_SIZE:
+            raise ValueError(f"the delta rule's kernels take 1..{self.MAX_TAPS} taps and heads of "
+                             f"up to {self.MAX_SIZE} entries, not {taps} taps, {qk_dim} and {v_dim}")
+        self.d_model, self.n_heads, self.n_kv_heads = int(d_model), int(n_heads), int(n_kv_heads)
+        self.qk_dim, self.v_dim, self.taps = int(qk_dim), int(v_dim), int(taps)
+        self.eps = float(eps)
+        self._rider_rows, self.rider_col = None, -1
+
+    def tensor_specs(self) -> dict:
+        d, h, e, f = self.d_model, self.n_heads, self.qk_dim, self.v_dim
+        ck, cv = self.n_kv_heads * e, h * f
+        return {"q": TensorSpec((ck, d)), "q.conv": TensorSpec((ck, self.taps)),
+                "k": TensorSpec((ck, d)), "k.conv": TensorSpec((ck, self.taps)),
+                "v": TensorSpec((cv, d)), "v.conv": TensorSpec((cv, self.taps)),
+                "b": TensorSpec((h, d)),
+                "A_log": TensorSpec((h,), kind="vector", init="zeros"),
+                "norm": TensorSpec((f,), kind="vector", init="ones"),
+                "a": TensorSpec((h, d)),
+                "dt_bias": TensorSpec((h,), kind="vector", init="zeros"),
+                "g": TensorSpec((cv, d)), "o": TensorSpec((d, cv))}
+
+    def state_floats(self) -> int:
+        """The matrices with padded rows and columns, then the convolution's inputs."""
+        e = -(-self.qk_dim // 32) * 32
+        f = -(-self.v_dim // 16) * 16
+        channels = 2 * self.n_kv_heads * self.qk_dim + self.n_heads * self.v_dim
+        return -(-(self.n_heads * e * f + self.taps * channels) // 4) * 4
+
+    def cache_spec(self):
+        return FixedState((self.state_floats(),), torch.float32)
+
+    def bind(self, tensors: dict, runtime, rider=None) -> None:
+        self.runtime = runtime
+        ops = runtime.ops
+        ops.require_part("delta")
+        ops.require_part("scan")                     # the heads' norm and gate live there
+        sizes = (self.n_heads, self.n_kv_heads, self.qk_dim, self.v_dim)
+        if ops.delta_state_floats(*sizes, self.taps) != self.state_floats():
+            raise RuntimeError("the delta rule's kernels lay the state out differently")
+        named = [("q", tensors["q"]), ("k", tensors["k"]), ("v", tensors["v"]),
+                 ("g", tensors["g"])]
+        if rider is not None:
+            named.append(("rider", rider))
+        named += [("b", tensors["b"]), ("a", tensors["a"])]
+        cols, at = {}, 0
+        for name, w in named:
+            cols[name], at = at, at + w.shape[0]
+        self.cols = (cols["q"], cols["a"], cols["b"], cols["g"])
+        self.rider_col = cols.get("rider", -1)
+        self.w_in = ops.prepare_weight(stack_rows([w for _, w in named]))
+        self.conv = stack_rows([tensors[f"{n}.conv"] for n in "qkv"], 1).contiguous()
+        f32 = torch.float32
+        self.a_exp = torch.exp(tensors["A_log"].to(f32)).contiguous()
+        self.dt_bias = tensors["dt_bias"].to(f32).contiguous()
+        self.norm_w = tensors["norm"].to(f32).contiguous()
+        self.norm_row = self.norm_w.repeat(self.n_heads).contiguous()
+        self.w_o = ops.prepare_weight(tensors["o"])
+        self.row_floats = ops.delta_rows(*sizes)
+
+    def forward(self, h, step: StepContext, cache: CacheHandle):
+        rt, ops = self.runtime, self.runtime.ops
+        t = step.n_tokens
+        nh, nk, e, f = self.n_heads, self.n_kv_heads, self.qk_dim, self.v_dim
+        proj = rt.buffer("delta_proj", (t, self.w_in.shape[0]), torch.float32)
+        ops.linear(h, self.w_in, proj)
+        self._rider_rows = proj
+        y = rt.buffer("attn_out", (t, nh * f), rt.act_dtype)
+        if step.max_q_len == 1:
+            ops.delta_step(proj, self.cols, self.conv, self.taps, self.a_exp, self.dt_bias,
+                           self.norm_w, self.eps, cache.state, step, nh, nk, e, f, y)
+        else:
+            rows = rt.buffer("delta_rows", (t, self.row_floats), torch.float32)
+            ops.delta_prep(proj, self.cols, self.conv, self.taps, self.a_exp, self.dt_bias,
+                           cache.state, step, nh, nk, e, f, rows)
+            o = rt.buffer("scan_out", (t, nh * f), torch.float32)
+            ops.delta_scan(rows, proj, self.cols[0], self.taps, cache.state, step, nh, nk, e, f, o)
+            ops.scan_finish(o, proj, self.cols[3], self.norm_row, self.eps, y, nh, f)
+        delta = rt.buffer("delta", (t, self.d_model), rt.act_dtype)
+        return ops.linear_parts(y, self.w_o, delta)
+
+    def rider(self):
+        return self._rider_rows, self.rider_col

@@ -1,5 +1,6 @@
-"""Norms: RMS norm with a learned weight, layer norm with a weight and no bias, and the norm
-without statistics (a scaled tanh with a weight and a bias).
+"""Norms: RMS norm with a learned weight (a vector or one number; also behind a sublayer, with a
+gate on the sublayer's result), layer norm with a weight and no bias, and the norm without
+statistics (a scaled tanh with a weight and a bias).
 
 Reference formula (train/model.py:29-33): ``xf = x.float()``;
 ``y = xf * rsqrt(mean(xf**2, -1) + eps)``; ``out = (y * w.float()).to(x.dtype)``.
@@ -15,27 +16,72 @@ import torch
 from .base import Norm, ResidualStream, TensorSpec
 
 
+class GatedDelta:
+    """A sublayer's output that is still to be gated and normed before it joins the residual
+    stream: ``norm(delta * sigmoid(gate + bias))``.  ``gate``: None, ``(rows, first column)``
+    or ``SplitParts``.  A norm that knows the kind (``RMSNorm.forward``) does it in the pass in
+    which it adds the delta; any other consumer gets the values through ``resolve()`` (one kernel
+    of its own, float32)."""
+
+    def __init__(self, delta, norm: "RMSNorm", gate=None, bias=None):
+        self.delta, self.norm, self.gate, self.bias = delta, norm, gate, bias
+
+    @property
+    def shape(self):
+        return self.delta.shape
+
+    def release(self) -> None:
+        for p in (self.delta, self.gate):
+            if hasattr(p, "release"):
+                p.release()
+
+    def resolve(self):
+        rt = self.norm.runtime
+        t, d = self.delta.shape
+        out = rt.buffer("gated_delta", (t, d), torch.float32)
+        rt.ops.add_gated_norm(None, self.delta, self.gate, self.bias, self.norm.weight32, None,
+                              self.norm.eps, None, y_out=out)
+        return out
+
+    def float(self):
+        return self.resolve()
+
+
 class RMSNorm(Norm):
     decode_capturable = prompt_capturable = True   # forward only launches kernels on the current stream
 
-    def __init__(self, dim: int, eps: float, tensor_name: str = "weight", one_plus: bool = False):
+    def __init__(self, dim: int, eps: float, tensor_name: str = "weight", one_plus: bool = False,
+                 scalar: bool = False):
         """``tensor_name``: the local name of the weight ("" = the part's own prefix).
         ``one_plus``: the weight is stored around zero and multiplies as ``1 + w`` (the sum is
-        taken once, in float32, when the weight is bound)."""
+        taken once, in float32, when the weight is bound).  ``scalar``: the weight is one number
+        for all coordinates (a tensor without dimensions).
+
+        Behind a sublayer the norm does not run by itself: ``gated(delta, gate, bias)`` wraps
+        the sublayer's output, and the norm that adds it to the stream does all of it in one
+        kernel."""
         self.dim = int(dim)
         self.eps = float(eps)
         self.tensor_name = tensor_name
-        self.one_plus = bool(one_plus)
-        self.weight = None
+        self.one_plus, self.scalar = bool(one_plus), bool(scalar)
+        self.weight = self.weight32 = None
 
     def tensor_specs(self) -> dict:
-        return {self.tensor_name: TensorSpec((self.dim,), kind="vector",
+        return {self.tensor_name: TensorSpec(() if self.scalar else (self.dim,), kind="vector",
                                              init="zeros" if self.one_plus else "ones")}
 
     def bind(self, tensors: dict, runtime) -> None:
         self.runtime = runtime
         w = tensors[self.tensor_name]
-        self.weight = (w.float() + 1.0).contiguous() if self.one_plus else w.contiguous()
+        w = w.float() + 1.0 if self.one_plus else w
+        self.weight32 = w.float().reshape(-1).contiguous()
+        self.weight = (w.reshape(1).expand(self.dim) if self.scalar else w).contiguous()
+
+    def gated(self, delta, gate=None, bias=None) -> GatedDelta:
+        """``delta`` (a tensor or ``SplitParts``) as what the gate, then this norm, make of it,
+        for ``ResidualStream.push``."""
+        self.runtime.ops.require_part("gatednorm")
+        return GatedDelta(delta, self, gate, bias)
 
     def forward(self, stream: ResidualStream, rows=None, n_rows: int = 0):
         """Add the pending delta into the stream, return the normalised rows.
@@ -50,6 +96,13 @@ class RMSNorm(Norm):
             # (also before picked rows: the addends go into every row of the stream)
             rt.ops.residual_add(stream.x, more_rows, more_vec)
         delta = stream.take_pending()
+        if isinstance(delta, GatedDelta) and delta.norm.eps == self.eps:
+            n = stream.x.shape[0] if rows is None else n_rows
+            h = rt.buffer("normed" if rows is None else "normed_rows", (n, self.dim), rt.act_dtype)
+            rt.ops.add_gated_norm(stream.x, delta.delta, delta.gate, delta.bias,
+                                  delta.norm.weight32, self.weight32, self.eps, h, rows=rows,
+                                  n_rows=n_rows)
+            return h
         if rows is None:
             t = stream.x.shape[0]
             h = rt.buffer("normed", (t, self.dim), rt.act_dtype)

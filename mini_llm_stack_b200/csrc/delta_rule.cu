@@ -199,6 +199,7 @@ template <int NI, int TT>
 __global__ void __launch_bounds__(DP_WARPS * 32)
 delta_prep_kernel(const DeltaArgs a, float* __restrict__ out) {
     chain_release();
+    __shared__ float kq_s[DP_WARPS][DP_RUN];
     const int lane = threadIdx.x & 31, unit = blockIdx.y * DP_WARPS + (threadIdx.x >> 5);
     if (unit >= a.G + a.H) return;
     const RowLayout lay = row_layout(a.H, a.G, a.er, a.fr);
@@ -222,12 +223,17 @@ delta_prep_kernel(const DeltaArgs a, float* __restrict__ out) {
                 hk.fill(a, t, i_t, p, ring, lane);
                 r_now = r;
             }
-            float yq[NI], yk[NI];
+            // the next token's inputs are under way while this one's are worked on
+            float yq[NI], yk[NI], nq[NI], nk[NI];
+            const int next = min(t + 1, t_end - 1);
+            hq.load(a, next, lane, nq);
+            hk.load(a, next, lane, nk);
             hq.step(xq, yq);
             hk.step(xk, yk);
-            if (t + 1 < t_end) {
-                hq.load(a, t + 1, lane, xq);
-                hk.load(a, t + 1, lane, xk);
+#pragma unroll
+            for (int i = 0; i < NI; ++i) {
+                xq[i] = nq[i];
+                xk[i] = nk[i];
             }
             float sq = 0.f, sk = 0.f, sqk = 0.f;
 #pragma unroll
@@ -249,14 +255,16 @@ delta_prep_kernel(const DeltaArgs a, float* __restrict__ out) {
                     row[lay.k_off + unit * a.er + c] = yk[i] * ik;
                 }
             }
-            for (int hh = lane; hh < ratio; hh += 32) {
-                const int head = unit * ratio + hh;
-                const float za = a.proj[(size_t)t * a.width + a.a_col + head] + a.dt_bias[head];
-                const float zb = a.proj[(size_t)t * a.width + a.b_col + head];
-                const float g = expf(-a.a_exp[head] * softplus1(za));
-                *reinterpret_cast<float4*>(row + lay.s_off + 4 * head) =
-                    make_float4(g, sigmoid1(zb), kq, 0.f);
-            }
+            if (lane == 0) kq_s[threadIdx.x >> 5][t - t_begin] = kq;
+        }
+        // the scalars of the run's tokens and of the value heads that share this key head
+        __syncwarp();
+        for (int u = lane; u < (t_end - t_begin) * ratio; u += 32) {
+            const int tt = u / ratio, head = unit * ratio + u - tt * ratio;
+            const float* src = a.proj + (size_t)(t_begin + tt) * a.width;
+            const float g = expf(-a.a_exp[head] * softplus1(src[a.a_col + head] + a.dt_bias[head]));
+            *reinterpret_cast<float4*>(out + (size_t)(t_begin + tt) * lay.row + lay.s_off + 4 * head) =
+                make_float4(g, sigmoid1(src[a.b_col + head]), kq_s[threadIdx.x >> 5][tt], 0.f);
         }
     } else {
         const int head = unit - a.G;
@@ -271,9 +279,11 @@ delta_prep_kernel(const DeltaArgs a, float* __restrict__ out) {
                 hv.fill(a, t, t - a.cu_q[r], a.positions[t], a.ring(a.state_slot[r]), lane);
                 r_now = r;
             }
-            float y[NI];
+            float y[NI], nx[NI];
+            hv.load(a, min(t + 1, t_end - 1), lane, nx);
             hv.step(x, y);
-            if (t + 1 < t_end) hv.load(a, t + 1, lane, x);
+#pragma unroll
+            for (int i = 0; i < NI; ++i) x[i] = nx[i];
             float* row = out + (size_t)t * lay.row + lay.v_off + head * a.fr;
 #pragma unroll
             for (int i = 0; i < NI; ++i) {

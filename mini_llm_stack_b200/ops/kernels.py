@@ -763,10 +763,10 @@ class Ops:
                    "headwise": _decl(lib, "mls_headwise_linear",
                                      [_P, _LL, _LL, _P, _P, _LL, _LL, _I, _I, _I, _I, _I, _P]),
                    "rope_prep": _decl(lib, "mls_latent_rope_prep",
-                                      [_P, _I, _LL, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P,
+                                      [_P, _I, _LL, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P,
                                        _P, _I, _F, _P, _P, _I, _I, _I, _P, _P, _I, _LL, _P, _P]),
                    "gate": _decl(lib, "mls_sigmoid_gate",
-                                 [_P, _I, _P, _I, _LL, _I, _I, _I, _I, _P])}
+                                 [_P, _I, _P, _I, _LL, _I, _I, _I, _I, _I, _P])}
         elif name == "tanhnorm":
             fns = {"add_tanh_norm": _decl(lib, "mls_add_tanh_norm",
                                           [_P, _P, _I, _I, _LL, _P, _F, _P, _P, _P, _F, _P, _P, _I,

@@ -1,5 +1,5 @@
-"""``bench.py --design zededra | logulix | zefenex | movazen``: prefill and decode throughput of the design's
-layers at sizes that resemble a real model's, beside the dense Llama-style decoder at equal
+"""``bench.py --design zededra | logulix | zefenex | movazen | nekedra``: prefill and decode
+throughput of the design's layers at sizes that resemble a real model's, beside the dense Llama-style decoder at equal
 size.
 
 Every model has random weights (N(0, 0.02^2), drawn on the device), ``--layers`` layers
@@ -126,16 +126,45 @@ def movazen_config(s: dict, kind: str, layers: int, vocab: int = 32000) -> dict:
             "embedding": {"scale": 1.0}, "token_side": {"dim": 256}, "layers": stack}
 
 
+def nekedra_config(s: dict, kind: str, layers: int, vocab: int = 32000) -> dict:
+    """Layers of one kind of Nekedra mixer with the gated unit of the dense decoder's width, gated
+    residuals and norms on both sides: the delta rule with as many value heads as the dense
+    decoder has heads over half as many key heads (keys and values of the head size, four taps),
+    Zefenex's latent attention without window and sink and with one gate a head, attention with
+    the dense decoder's heads, biases, sinks and mixed values; or the three in turns."""
+    kv = max(1, s["kv_rank"] // (2 * s["dim"]), s["heads"] // 16)
+    heads, dim, g = s["heads"], s["dim"], s["kv_rank"] // 4
+    mixers = {
+        "delta": {"type": "delta", "mixer": {"conv": 4, "dim": dim, "heads": heads,
+                                             "kv_heads": heads // 2, "vdim": dim}},
+        "latent": {"type": "latent_attention",
+                   "mixer": {"dim": dim - g, "heads": heads, "kv_rank": s["kv_rank"] - g,
+                             "rot_dim": g, "rot": {"base": 1e6, "dims": g}, "scale": dim ** -0.5,
+                             "vdim": dim}},
+        "attention": {"type": "attention",
+                      "mixer": {"dim": dim, "heads": heads, "kv_heads": kv, "scale": dim ** -0.5,
+                                "v_mix": True, "vdim": dim}}}
+    dense = {"ff": s["ff"], "kind": "dense"}
+    turns = ["delta", "attention", "delta", "latent"] if kind == "turns_dense" else \
+        [kind.split("_")[0]]
+    stack = [dict(mixers[turns[i % len(turns)]], mlp=dense) for i in range(layers)]
+    return {"architecture": "Nekedra", "vocab": vocab, "width": s["width"], "norm": {"eps": 1e-6},
+            "layers": stack}
+
+
 DESIGNS = {
     "zededra": (zededra_config, ("latent_dense", "latent_moe", "mlstm_dense")),
     "logulix": (logulix_config, ("attention_dense", "wkv_dense", "retention_dense")),
     "zefenex": (zefenex_config, ("latent_dense", "latent_moe", "shared_cache_dense")),
     "movazen": (movazen_config, ("attention_moe", "parallel_moe", "mixers_only")),
+    "nekedra": (nekedra_config, ("delta_dense", "latent_dense", "attention_dense", "turns_dense")),
 }
 # rows of another design measured beside a design's own: the closest existing layers
 BESIDE = {"zefenex": (("zededra", "latent_dense"), ("zededra", "latent_moe")),
           "movazen": (("zefenex", "latent_moe"), ("logulix", "attention_dense"),
-                      ("logulix", "retention_dense"))}
+                      ("logulix", "retention_dense")),
+          "nekedra": (("logulix", "retention_dense"), ("zefenex", "latent_dense"),
+                      ("logulix", "attention_dense"))}
 
 
 def llama_config(s: dict, layers: int, vocab: int = 32000) -> dict:
@@ -155,7 +184,8 @@ _LEAVES = ("embed", "add_rmsnorm", "gather_add_rmsnorm", "add_layernorm", "resid
            "tail_update", "token_shift_mix", "linear_scan", "scan_finish", "rotate_rows",
            "decay_lowrank", "relu_squared", "scale_", "settle_concat", "add_tanh_norm",
            "latent_rope_prep", "sigmoid_gate", "softcap_", "head_prep_store", "settle_cast",
-           "gelu_gate_rows", "rms_scale", "scan_finish_row")
+           "gelu_gate_rows", "rms_scale", "scan_finish_row", "add_gated_norm", "delta_prep",
+           "delta_scan", "delta_step")
 _PRODUCTS = ("linear", "linear_parts", "linear_swiglu", "linear_clamped_glu",
              "linear_relu_squared")
 

@@ -29,9 +29,9 @@
 // A warp owns four columns of S with eight lanes a column; a lane keeps er / 8 rows of its
 // column in registers, four neighbouring rows at a time (16-byte accesses of the state and of
 // k and q), and multiplies them two at a time (fma.rn.f32x2).  The sum over the rows is the
-// lane's own in a fixed order and three shuffles: a token's bits depend neither on the batch
-// nor on how the tokens were cut into steps (in steps that run the same kernel).
-// Everything is float32.
+// lane's own in a fixed order and three shuffles: a token's bits do not depend on the batch.
+// The scan takes two tokens at a time from a portion's start, which moves the last bits where
+// a cut separates two tokens.  Everything is float32.
 #include "common.cuh"
 
 namespace {
@@ -77,6 +77,7 @@ __device__ __forceinline__ float column_sum(float v) {
     v += __shfl_xor_sync(0xffffffffu, v, 4);
     return v;
 }
+__device__ __forceinline__ const float* nearer(const float* a, const float* b) { return a < b ? a : b; }
 __device__ __forceinline__ void copy16(void* dst, const void* src) {
     const unsigned d = (unsigned)__cvta_generic_to_shared(dst);
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(d), "l"(src) : "memory");
@@ -355,7 +356,30 @@ delta_scan_kernel(const DeltaArgs a, const float* __restrict__ rows, float* __re
         }
     }
     const bool writes = grp == 0 && col < a.f;
-    float* o_col = out + (size_t)t0 * a.H * a.f + (size_t)head * a.f + col;
+    const size_t o_row = (size_t)a.H * a.f;
+    float* o_at = out + (size_t)t0 * o_row + (size_t)head * a.f + col;
+    auto load_rows = [&](ulonglong2 (&v)[R4], const float* src) {
+#pragma unroll
+        for (int i = 0; i < R4; ++i) v[i] = *reinterpret_cast<const ulonglong2*>(src + 32 * i + 4 * grp);
+    };
+    auto state_dot = [&](const ulonglong2 (&v)[R4]) {         // this lane's share of S^T v
+        f32x2 d0 = 0ull, d1 = 0ull;
+#pragma unroll
+        for (int i = 0; i < R4; ++i) {
+            d0 = fma2(s[i][0], v[i].x, d0);
+            d1 = fma2(s[i][1], v[i].y, d1);
+        }
+        return sum2(add2(d0, d1));
+    };
+    auto dot = [&](const ulonglong2 (&u)[R4], const ulonglong2 (&v)[R4]) {
+        f32x2 d0 = 0ull, d1 = 0ull;
+#pragma unroll
+        for (int i = 0; i < R4; ++i) {
+            d0 = fma2(u[i].x, v[i].x, d0);
+            d1 = fma2(u[i].y, v[i].y, d1);
+        }
+        return sum2(add2(d0, d1));
+    };
     for (int b0 = 0; b0 < n; b0 += DS_TOKENS) {
         const int nb = min(DS_TOKENS, n - b0);
         if (b0 + DS_TOKENS < n) {
@@ -366,51 +390,70 @@ delta_scan_kernel(const DeltaArgs a, const float* __restrict__ rows, float* __re
         }
         __syncthreads();
         const float* tok = smem + (size_t)((b0 / DS_TOKENS) & 1) * DS_TOKENS * TOK;
-        ulonglong2 k[R4], q[R4];
+        const float* last = tok + (nb - 1) * TOK;
+        ulonglong2 ka[R4], qa[R4], kb[R4], qb[R4];
+        load_rows(qa, tok);
+        load_rows(ka, tok + ER);
+        load_rows(qb, nearer(tok + TOK, last));
+        load_rows(kb, nearer(tok + TOK, last) + ER);
+        // Two tokens at a time: both tokens' products with the state before them cross the lanes
+        // together, and what the first token changed of the second's follows from the products
+        // of their keys and query.
+        for (; tok < last; tok += 2 * TOK) {
+            float sqa = state_dot(qa), sqb = state_dot(qb), ska = state_dot(ka), skb = state_dot(kb);
+            float kkb = dot(ka, kb), kqb = dot(ka, qb);
+            const float va = tok[2 * ER + my], vb = tok[TOK + 2 * ER + my];
+            const float4 ca = *reinterpret_cast<const float4*>(tok + 2 * ER + DS_COLS);
+            const float4 cb = *reinterpret_cast<const float4*>(tok + TOK + 2 * ER + DS_COLS);
+            const float* nxt = nearer(tok + 2 * TOK, last);
+            const float* nxt2 = nearer(tok + 3 * TOK, last);
+            load_rows(qa, nxt);
+            load_rows(qb, nxt2);
 #pragma unroll
-        for (int i = 0; i < R4; ++i) {
-            q[i] = *reinterpret_cast<const ulonglong2*>(tok + 32 * i + 4 * grp);
-            k[i] = *reinterpret_cast<const ulonglong2*>(tok + ER + 32 * i + 4 * grp);
-        }
-        for (int tt = 0; tt < nb; ++tt, tok += TOK) {
-            f32x2 dk[2] = {0ull, 0ull}, dq[2] = {0ull, 0ull};
-#pragma unroll
-            for (int i = 0; i < R4; ++i) {
-                dk[0] = fma2(s[i][0], k[i].x, dk[0]);
-                dk[1] = fma2(s[i][1], k[i].y, dk[1]);
+            for (int o = 1; o < 8; o <<= 1) {
+                ska += __shfl_xor_sync(0xffffffffu, ska, o);
+                skb += __shfl_xor_sync(0xffffffffu, skb, o);
+                kkb += __shfl_xor_sync(0xffffffffu, kkb, o);
+                sqa += __shfl_xor_sync(0xffffffffu, sqa, o);
+                sqb += __shfl_xor_sync(0xffffffffu, sqb, o);
+                kqb += __shfl_xor_sync(0xffffffffu, kqb, o);
             }
-#pragma unroll
-            for (int i = 0; i < R4; ++i) {
-                dq[0] = fma2(s[i][0], q[i].x, dq[0]);
-                dq[1] = fma2(s[i][1], q[i].y, dq[1]);
-            }
-            const float vj = tok[2 * ER + my];
-            const float4 sc = *reinterpret_cast<const float4*>(tok + 2 * ER + DS_COLS);
-            float sk = column_sum(sum2(add2(dk[0], dk[1])));
-            float sq = column_sum(sum2(add2(dq[0], dq[1])));
-            // the next token's key and query come while the sums cross the lanes
-            ulonglong2 kn[R4];
-            const float* nxt = tt + 1 < nb ? tok + TOK : tok;
-#pragma unroll
-            for (int i = 0; i < R4; ++i) {
-                q[i] = *reinterpret_cast<const ulonglong2*>(nxt + 32 * i + 4 * grp);
-                kn[i] = *reinterpret_cast<const ulonglong2*>(nxt + ER + 32 * i + 4 * grp);
-            }
-            const f32x2 g2 = pack2(sc.x, sc.x);
+            const float gab = ca.x * cb.x;
+            const f32x2 g2 = pack2(gab, gab);
 #pragma unroll
             for (int i = 0; i < R4; ++i) {
                 s[i][0] = mul2(g2, s[i][0]);
                 s[i][1] = mul2(g2, s[i][1]);
             }
-            const float u = sc.y * fmaf(-sc.x, sk, vj);
-            const f32x2 u2 = pack2(u, u);
+            const float ua = ca.y * fmaf(-ca.x, ska, va);
+            const float ub = cb.y * fmaf(-cb.x, fmaf(ca.x, skb, kkb * ua), vb);
+            const float wa = cb.x * ua;                  // the first write, decayed once
+            const f32x2 a2 = pack2(wa, wa), b2 = pack2(ub, ub);
 #pragma unroll
             for (int i = 0; i < R4; ++i) {
-                s[i][0] = fma2(k[i].x, u2, s[i][0]);
-                s[i][1] = fma2(k[i].y, u2, s[i][1]);
-                k[i] = kn[i];
+                s[i][0] = fma2(kb[i].x, b2, fma2(ka[i].x, a2, s[i][0]));
+                s[i][1] = fma2(kb[i].y, b2, fma2(ka[i].y, a2, s[i][1]));
             }
-            if (writes) o_col[(size_t)(b0 + tt) * a.H * a.f] = fmaf(sc.x, sq, sc.z * u);
+            load_rows(ka, nxt + ER);
+            load_rows(kb, nxt2 + ER);
+            if (writes) {
+                o_at[0] = fmaf(ca.x, sqa, ca.z * ua);
+                o_at[o_row] = fmaf(cb.x, fmaf(ca.x, sqb, kqb * ua), cb.z * ub);
+            }
+            o_at += 2 * o_row;
+        }
+        if (tok == last) {
+            const float sk = column_sum(state_dot(ka)), sq = column_sum(state_dot(qa));
+            const float4 c = *reinterpret_cast<const float4*>(tok + 2 * ER + DS_COLS);
+            const float u = c.y * fmaf(-c.x, sk, tok[2 * ER + my]);
+            const f32x2 g2 = pack2(c.x, c.x), u2 = pack2(u, u);
+#pragma unroll
+            for (int i = 0; i < R4; ++i) {
+                s[i][0] = fma2(ka[i].x, u2, mul2(g2, s[i][0]));
+                s[i][1] = fma2(ka[i].y, u2, mul2(g2, s[i][1]));
+            }
+            if (writes) o_at[0] = fmaf(c.x, sq, c.z * u);
+            o_at += o_row;
         }
         __syncthreads();                                // before this buffer is fetched into again
     }

@@ -94,9 +94,15 @@ __device__ __forceinline__ void store_pack(void* base, size_t i, int dtype, cons
 }
 
 // N: entries a thread takes at a time (4: every row starts at a 16-byte place; else 1).
-// VEC: such groups a thread keeps in registers, threads * N * VEC >= d.
-template <int N, int VEC, int MAX_THREADS>
-__global__ void __launch_bounds__(MAX_THREADS) add_gated_norm_kernel(const GatedNormArgs a) {
+// VEC: such groups a thread keeps in registers, threads * N * VEC >= d.  PARTS: the result or
+// the gate may come as K-parts (few rows); without, the kernel has registers for more blocks an
+// SM, whose rows' loads and block sums then overlap.
+constexpr int blocks_an_sm(int vec, int max_threads, bool parts) {
+    return parts || max_threads > 256 ? 1 : vec <= 1 ? 6 : vec <= 2 ? 5 : vec <= 4 ? 3 : 1;
+}
+template <int N, int VEC, int MAX_THREADS, bool PARTS>
+__global__ void __launch_bounds__(MAX_THREADS, blocks_an_sm(VEC, MAX_THREADS, PARTS))
+add_gated_norm_kernel(const GatedNormArgs a) {
     chain_release();
     __shared__ float scratch[33];
     const int groups = a.d / N, i = blockIdx.x;
@@ -109,11 +115,11 @@ __global__ void __launch_bounds__(MAX_THREADS) add_gated_norm_kernel(const Gated
     for (int k = 0; k < VEC; ++k) {
         const int c = ((int)threadIdx.x + k * (int)blockDim.x) * N;
         if (c < groups * N) {
-            y[k] = load_parts<N>(a.y, at + c, a.y_dtype, a.y_parts, (size_t)a.y_stride);
+            y[k] = load_parts<N>(a.y, at + c, a.y_dtype, PARTS ? a.y_parts : 1, (size_t)a.y_stride);
             if (a.x) x[k] = load_pack<N>(a.x, at + c, MLS_F32);
             if (a.z) {
                 Pack<N> z = load_parts<N>(a.z, (size_t)t * a.z_row + a.z_col + c, a.z_dtype,
-                                          a.z_parts, (size_t)a.z_stride);
+                                          PARTS ? a.z_parts : 1, (size_t)a.z_stride);
                 if (a.z_bias) {
                     const Pack<N> b = load_pack<N>(a.z_bias, c, MLS_F32);
 #pragma unroll
@@ -195,12 +201,14 @@ MLS_API int mls_add_gated_norm(float* x, const void* y, int y_dtype, int y_parts
     while (threads < 1024 && threads * 4 < groups) threads <<= 1;
     const int vec = (groups + threads - 1) / threads;
     if (vec > 16) return MLS_ERR_UNSUPPORTED;
-#define GN_GO(N, V)                                                                                  \
-    do {                                                                                             \
-        if (threads <= 256)                                                                          \
-            MLS_LAUNCH((add_gated_norm_kernel<N, V, 256>), dim3(n_out), dim3(threads), 0, stream, a); \
-        else                                                                                         \
-            MLS_LAUNCH((add_gated_norm_kernel<N, V, 1024>), dim3(n_out), dim3(threads), 0, stream, a); \
+    const bool parts = y_parts > 1 || (z && z_parts > 1);
+#define GN_RUN(N, V, M, P) \
+    MLS_LAUNCH((add_gated_norm_kernel<N, V, M, P>), dim3(n_out), dim3(threads), 0, stream, a)
+#define GN_GO(N, V)                                \
+    do {                                           \
+        if (threads > 256) GN_RUN(N, V, 1024, true); \
+        else if (parts) GN_RUN(N, V, 256, true);   \
+        else GN_RUN(N, V, 256, false);             \
     } while (0)
     if (by4) {
         if (vec <= 1) GN_GO(4, 1);
@@ -214,5 +222,6 @@ MLS_API int mls_add_gated_norm(float* x, const void* y, int y_dtype, int y_parts
         else GN_GO(1, 16);
     }
 #undef GN_GO
+#undef GN_RUN
     return launch_status();
 }

@@ -229,8 +229,13 @@ def test_delta_scan_alone_and_a_used_slot(rt32):
     state[1].zero_()
     third, _ = case.prompt(ops, state, [(0, 0, 120), ], [1], torch.float32)
     rest, _ = case.prompt(ops, state, [(0, 120, 300)], [1], torch.float32)
-    # cutting a prompt changes no bit
+    # an even cut leaves the scan's pairs of tokens as they are and changes no bit; an odd one
+    # changes no more than the last bits
     assert np.array_equal(np.concatenate([third, rest]), first)
+    state[1].zero_()
+    odd = [case.prompt(ops, state, [(0, a, b)], [1], torch.float32)[0]
+           for a, b in ((0, 121), (121, 124), (124, 300))]
+    assert np.abs(np.concatenate(odd) - first).max() < 2e-6 * scale
 
 
 def test_delta_bfloat16_outputs(rt32):

@@ -33,6 +33,7 @@
 // The scan takes two tokens at a time from a portion's start, which moves the last bits where
 // a cut separates two tokens.  Everything is float32.
 #include "common.cuh"
+#include "tma.cuh"
 
 namespace {
 constexpr float DR_UNIT_EPS = 1e-6f;     // inside the root of the unit vectors
@@ -77,12 +78,6 @@ __device__ __forceinline__ float column_sum(float v) {
     v += __shfl_xor_sync(0xffffffffu, v, 4);
     return v;
 }
-__device__ __forceinline__ const float* nearer(const float* a, const float* b) { return a < b ? a : b; }
-__device__ __forceinline__ void copy16(void* dst, const void* src) {
-    const unsigned d = (unsigned)__cvta_generic_to_shared(dst);
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(d), "l"(src) : "memory");
-}
-
 // Sizes, places and parameters every kernel here needs.
 struct DeltaArgs {
     const float* proj;                 // [parts][T, width]: q heads | k heads | v heads, gates, ...
@@ -121,17 +116,28 @@ struct DeltaArgs {
     }
 };
 
-// The rows the scan reads, float32: [q: G er | k: G er | v: H fr | (decay, step, k . q, 0): 4 H].
-struct RowLayout {
-    int k_off, v_off, s_off, row;
+// What the scan reads, float32, so that the tokens of a pass are one run of memory each:
+//   [G][T][q: er | k: er]      [H][fr / 16][T][16 values]      [H][T][DR_SCALARS]
+// with the scalars of a value head and token: decay, step, k . q, k' . k, k' . q, 0, 0, 0, where k'
+// is the key of the token before (anything where a request's tokens of the step begin).
+constexpr int DR_SCALARS = 8, DR_COLS = 16;
+struct Prepared {
+    size_t v_at, s_at;                 // where the values and the scalars begin
+    size_t T;
+    int er, fr;
+    __host__ __device__ Prepared(int n_tokens, int H, int G, int er_, int fr_)
+        : v_at((size_t)n_tokens * G * 2 * er_), s_at(v_at + (size_t)n_tokens * H * fr_),
+          T((size_t)n_tokens), er(er_), fr(fr_) {}
+    __host__ __device__ size_t qk(int kv, int t) const { return ((size_t)kv * T + t) * 2 * er; }
+    __host__ __device__ size_t v(int head, int chunk, int t) const {
+        return v_at + (((size_t)head * (fr / DR_COLS) + chunk) * T + t) * DR_COLS;
+    }
+    __host__ __device__ size_t scalars(int head, int t) const {
+        return s_at + ((size_t)head * T + t) * DR_SCALARS;
+    }
 };
-__host__ __device__ inline RowLayout row_layout(int H, int G, int er, int fr) {
-    RowLayout l;
-    l.k_off = G * er;
-    l.v_off = 2 * G * er;
-    l.s_off = l.v_off + H * fr;
-    l.row = l.s_off + 4 * H;
-    return l;
+__host__ __device__ inline int prepared_floats(int H, int G, int er, int fr) {      // a token's share
+    return 2 * G * er + H * (fr + DR_SCALARS);
 }
 
 // A head's channels spread over a warp (channel lane + 32 i) with the convolution's weights and
@@ -200,10 +206,10 @@ template <int NI, int TT>
 __global__ void __launch_bounds__(DP_WARPS * 32)
 delta_prep_kernel(const DeltaArgs a, float* __restrict__ out) {
     chain_release();
-    __shared__ float kq_s[DP_WARPS][DP_RUN];
+    __shared__ float dots_s[DP_WARPS][DP_RUN][3];
     const int lane = threadIdx.x & 31, unit = blockIdx.y * DP_WARPS + (threadIdx.x >> 5);
     if (unit >= a.G + a.H) return;
-    const RowLayout lay = row_layout(a.H, a.G, a.er, a.fr);
+    const Prepared to(a.n_tokens, a.H, a.G, a.er, a.fr);
     const int t_begin = blockIdx.x * DP_RUN, t_end = min(t_begin + DP_RUN, a.n_tokens);
     int r_now = -1;
     if (unit < a.G) {
@@ -212,10 +218,15 @@ delta_prep_kernel(const DeltaArgs a, float* __restrict__ out) {
         hq.init(a, unit * a.e, a.e, lane);
         hk.init(a, (a.G + unit) * a.e, a.e, lane);
         chain_wait();
-        float xq[NI], xk[NI];
-        hq.load(a, t_begin, lane, xq);
-        hk.load(a, t_begin, lane, xk);
-        for (int t = t_begin; t < t_end; ++t) {
+        // the token before the run as well, if it is of the same request: its key is wanted
+        const int t_first = t_begin > 0 && a.req_of_token[t_begin - 1] == a.req_of_token[t_begin]
+            ? t_begin - 1 : t_begin;
+        float xq[NI], xk[NI], kp[NI];
+        hq.load(a, t_first, lane, xq);
+        hk.load(a, t_first, lane, xk);
+#pragma unroll
+        for (int i = 0; i < NI; ++i) kp[i] = 0.f;
+        for (int t = t_first; t < t_end; ++t) {
             const int r = a.req_of_token[t];
             if (r != r_now) {
                 const float* ring = a.ring(a.state_slot[r]);
@@ -236,36 +247,43 @@ delta_prep_kernel(const DeltaArgs a, float* __restrict__ out) {
                 xq[i] = nq[i];
                 xk[i] = nk[i];
             }
-            float sq = 0.f, sk = 0.f, sqk = 0.f;
+            float sq = 0.f, sk = 0.f, sqk = 0.f, spk = 0.f, spq = 0.f;
 #pragma unroll
             for (int i = 0; i < NI; ++i) {
                 if (lane + 32 * i >= a.e) yq[i] = yk[i] = 0.f;
                 sq = fmaf(yq[i], yq[i], sq);
                 sk = fmaf(yk[i], yk[i], sk);
                 sqk = fmaf(yq[i], yk[i], sqk);
+                spk = fmaf(kp[i], yk[i], spk);
+                spq = fmaf(kp[i], yq[i], spq);
             }
             const float iq = 1.0f / sqrtf(warp_sum(sq) + DR_UNIT_EPS) * a.q_scale;
             const float ik = 1.0f / sqrtf(warp_sum(sk) + DR_UNIT_EPS);
             const float kq = warp_sum(sqk) * iq * ik;
-            float* row = out + (size_t)t * lay.row;
+            const float pk = warp_sum(spk) * ik, pq = warp_sum(spq) * iq;
+            float* row = out + to.qk(unit, t);
 #pragma unroll
             for (int i = 0; i < NI; ++i) {
                 const int c = lane + 32 * i;
-                if (c < a.er) {
-                    row[unit * a.er + c] = yq[i] * iq;
-                    row[lay.k_off + unit * a.er + c] = yk[i] * ik;
+                kp[i] = yk[i] * ik;
+                if (t >= t_begin && c < a.er) {
+                    row[c] = yq[i] * iq;
+                    row[a.er + c] = kp[i];
                 }
             }
-            if (lane == 0) kq_s[threadIdx.x >> 5][t - t_begin] = kq;
+            if (t >= t_begin && lane < 3)
+                dots_s[threadIdx.x >> 5][t - t_begin][lane] = lane == 0 ? kq : lane == 1 ? pk : pq;
         }
         // the scalars of the run's tokens and of the value heads that share this key head
         __syncwarp();
         for (int u = lane; u < (t_end - t_begin) * ratio; u += 32) {
             const int tt = u / ratio, head = unit * ratio + u - tt * ratio;
             const float* src = a.proj + (size_t)(t_begin + tt) * a.width;
+            const float* dots = dots_s[threadIdx.x >> 5][tt];
             const float g = expf(-a.a_exp[head] * softplus1(src[a.a_col + head] + a.dt_bias[head]));
-            *reinterpret_cast<float4*>(out + (size_t)(t_begin + tt) * lay.row + lay.s_off + 4 * head) =
-                make_float4(g, sigmoid1(src[a.b_col + head]), kq_s[threadIdx.x >> 5][tt], 0.f);
+            float4* dst = reinterpret_cast<float4*>(out + to.scalars(head, t_begin + tt));
+            dst[0] = make_float4(g, sigmoid1(src[a.b_col + head]), dots[0], dots[1]);
+            dst[1] = make_float4(dots[2], 0.f, 0.f, 0.f);
         }
     } else {
         const int head = unit - a.G;
@@ -285,56 +303,62 @@ delta_prep_kernel(const DeltaArgs a, float* __restrict__ out) {
             hv.step(x, y);
 #pragma unroll
             for (int i = 0; i < NI; ++i) x[i] = nx[i];
-            float* row = out + (size_t)t * lay.row + lay.v_off + head * a.fr;
 #pragma unroll
             for (int i = 0; i < NI; ++i) {
                 const int c = lane + 32 * i;
-                if (c < a.fr) row[c] = c < a.f ? y[i] : 0.f;
+                if (c < a.fr)
+                    out[to.v(head, c / DR_COLS, t) + c % DR_COLS] = c < a.f ? y[i] : 0.f;
             }
         }
     }
 }
 
-constexpr int DS_COLS = 16;            // columns of S a CTA of the scan owns
+constexpr int DS_COLS = DR_COLS;       // columns of S a CTA of the scan owns
 constexpr int DS_THREADS = 128;        // four warps, four columns each
 constexpr int DS_TOKENS = 16;          // tokens in one of the two buffers
 
 // R4: groups of four rows a lane keeps, er = 32 R4.
 template <int R4>
 __global__ void __launch_bounds__(DS_THREADS)
-delta_scan_kernel(const DeltaArgs a, const float* __restrict__ rows, float* __restrict__ out) {
-    constexpr int ER = 32 * R4;
-    constexpr int TOK = 2 * ER + DS_COLS + 4;          // floats of a token in shared memory
+delta_scan_kernel(const DeltaArgs a, const float* __restrict__ rows, float* __restrict__ out,
+                  int* status) {
+    using namespace mls_tma;
+    constexpr int ER = 32 * R4, QK = 2 * ER;           // floats of a token's q and k
+    constexpr int V_AT = DS_TOKENS * QK, S_AT = V_AT + DS_TOKENS * DS_COLS;
+    constexpr int BUF = S_AT + DS_TOKENS * DR_SCALARS;
     chain_release();
-    extern __shared__ __align__(16) float smem[];      // [2][DS_TOKENS][TOK]
+    // two buffers, and room for the rows read ahead behind the last token (not used)
+    extern __shared__ __align__(128) float smem[];
+    __shared__ int arrived;
+    __shared__ __align__(8) uint64_t full_bars[2];
     const int r = blockIdx.z, head = blockIdx.y, col0 = blockIdx.x * DS_COLS;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, grp = lane & 7;
     const int my = warp * 4 + (lane >> 3), col = col0 + my;
-    const RowLayout lay = row_layout(a.H, a.G, ER, a.fr);
+    const Prepared from(a.n_tokens, a.H, a.G, ER, a.fr);
     const int t0 = a.cu_q[r], n = a.cu_q[r + 1] - t0;
     if (n <= 0) return;
     const int slot = a.state_slot[r];
+    if (threadIdx.x == 0) {
+        mbar_init((uint32_t)__cvta_generic_to_shared(&full_bars[0]), 1);
+        mbar_init((uint32_t)__cvta_generic_to_shared(&full_bars[1]), 1);
+        fence_barrier_init();
+    }
+    __syncthreads();
     chain_wait();
-    const int kv = head / (a.H / a.G);
-    const float* q_src = rows + kv * ER;
-    const float* k_src = rows + lay.k_off + kv * ER;
-    const float* v_src = rows + lay.v_off + head * a.fr + col0;
-    const float* s_src = rows + lay.s_off + 4 * head;
-    auto fetch = [&](int b0) {                          // the copies of tokens b0 .. into their buffer
-        const int nb = min(DS_TOKENS, n - b0);
-        float* dst = smem + (size_t)((b0 / DS_TOKENS) & 1) * DS_TOKENS * TOK;
-        constexpr int U = ER / 4, PER = 2 * U + DS_COLS / 4 + 1;
-        for (int u = threadIdx.x; u < nb * PER; u += DS_THREADS) {
-            const int tt = u / PER, i = u - tt * PER;
-            const size_t t = (size_t)(t0 + b0 + tt) * lay.row;
-            const float* src = i < U ? q_src + t + 4 * i
-                : i < 2 * U ? k_src + t + 4 * (i - U)
-                : i < 2 * U + DS_COLS / 4 ? v_src + t + 4 * (i - 2 * U) : s_src + t;
-            copy16(dst + (size_t)tt * TOK + 4 * i, src);
-        }
-        asm volatile("cp.async.commit_group;" ::: "memory");
+    auto fetch = [&](int b0) {                          // one thread: tokens b0 .. into their buffer
+        const int which = (b0 / DS_TOKENS) & 1;
+        const uint32_t nb = (uint32_t)min(DS_TOKENS, n - b0);
+        const uint32_t bar = (uint32_t)__cvta_generic_to_shared(&full_bars[which]);
+        const uint32_t dst = (uint32_t)__cvta_generic_to_shared(smem + (size_t)which * BUF);
+        mbar_arrive_expect_tx(bar, nb * (uint32_t)((QK + DS_COLS + DR_SCALARS) * sizeof(float)));
+        bulk_load_1d(dst, rows + from.qk(head / (a.H / a.G), t0 + b0), nb * QK * 4, bar);
+        bulk_load_1d(dst + V_AT * 4, rows + from.v(head, blockIdx.x, t0 + b0), nb * DS_COLS * 4, bar);
+        bulk_load_1d(dst + S_AT * 4, rows + from.scalars(head, t0 + b0), nb * DR_SCALARS * 4, bar);
     };
-    fetch(0);
+    if (threadIdx.x == 0) {
+        fetch(0);
+        if (n > DS_TOKENS) fetch(DS_TOKENS);
+    }
     float* S = a.state + (size_t)slot * a.state_stride + ((size_t)head * a.fr + col) * ER + 4 * grp;
     f32x2 s[R4][2];
 #pragma unroll
@@ -371,52 +395,42 @@ delta_scan_kernel(const DeltaArgs a, const float* __restrict__ rows, float* __re
         }
         return sum2(add2(d0, d1));
     };
-    auto dot = [&](const ulonglong2 (&u)[R4], const ulonglong2 (&v)[R4]) {
-        f32x2 d0 = 0ull, d1 = 0ull;
-#pragma unroll
-        for (int i = 0; i < R4; ++i) {
-            d0 = fma2(u[i].x, v[i].x, d0);
-            d1 = fma2(u[i].y, v[i].y, d1);
-        }
-        return sum2(add2(d0, d1));
-    };
     for (int b0 = 0; b0 < n; b0 += DS_TOKENS) {
-        const int nb = min(DS_TOKENS, n - b0);
-        if (b0 + DS_TOKENS < n) {
-            fetch(b0 + DS_TOKENS);
-            asm volatile("cp.async.wait_group 1;" ::: "memory");
-        } else {
-            asm volatile("cp.async.wait_group 0;" ::: "memory");
-        }
+        const int nb = min(DS_TOKENS, n - b0), pass = b0 / DS_TOKENS;
+        if (threadIdx.x == 0)
+            arrived = mbar_wait((uint32_t)__cvta_generic_to_shared(&full_bars[pass & 1]),
+                                (pass >> 1) & 1) ? 1 : 0;
         __syncthreads();
-        const float* tok = smem + (size_t)((b0 / DS_TOKENS) & 1) * DS_TOKENS * TOK;
-        const float* last = tok + (nb - 1) * TOK;
+        if (!arrived) {                                 // every thread leaves at the same place
+            if (threadIdx.x == 0 && status) atomicOr(status, MLS_STATUS_TIMEOUT);
+            return;
+        }
+        const float* tok = smem + (size_t)(pass & 1) * BUF;          // q and k of the present token
+        const float* v_at = tok + V_AT + my;
+        const float* s_at = tok + S_AT;
+        const float* last = tok + (nb - 1) * QK;
         ulonglong2 ka[R4], qa[R4], kb[R4], qb[R4];
         load_rows(qa, tok);
         load_rows(ka, tok + ER);
-        load_rows(qb, nearer(tok + TOK, last));
-        load_rows(kb, nearer(tok + TOK, last) + ER);
+        load_rows(qb, tok + QK);
+        load_rows(kb, tok + QK + ER);
         // Two tokens at a time: both tokens' products with the state before them cross the lanes
         // together, and what the first token changed of the second's follows from the products
-        // of their keys and query.
-        for (; tok < last; tok += 2 * TOK) {
+        // of its key with the second's key and query.
+        for (; tok < last; tok += 2 * QK) {
             float sqa = state_dot(qa), sqb = state_dot(qb), ska = state_dot(ka), skb = state_dot(kb);
-            float kkb = dot(ka, kb), kqb = dot(ka, qb);
-            const float va = tok[2 * ER + my], vb = tok[TOK + 2 * ER + my];
-            const float4 ca = *reinterpret_cast<const float4*>(tok + 2 * ER + DS_COLS);
-            const float4 cb = *reinterpret_cast<const float4*>(tok + TOK + 2 * ER + DS_COLS);
-            const float* nxt = nearer(tok + 2 * TOK, last);
-            const float* nxt2 = nearer(tok + 3 * TOK, last);
-            load_rows(qa, nxt);
-            load_rows(qb, nxt2);
+            const float va = v_at[0], vb = v_at[DS_COLS];
+            const float4 ca = *reinterpret_cast<const float4*>(s_at);
+            const float4 cb = *reinterpret_cast<const float4*>(s_at + DR_SCALARS);
+            const float kqb = s_at[DR_SCALARS + 4];
+            load_rows(qa, tok + 2 * QK);
+            load_rows(qb, tok + 3 * QK);
 #pragma unroll
             for (int o = 1; o < 8; o <<= 1) {
                 ska += __shfl_xor_sync(0xffffffffu, ska, o);
                 skb += __shfl_xor_sync(0xffffffffu, skb, o);
-                kkb += __shfl_xor_sync(0xffffffffu, kkb, o);
                 sqa += __shfl_xor_sync(0xffffffffu, sqa, o);
                 sqb += __shfl_xor_sync(0xffffffffu, sqb, o);
-                kqb += __shfl_xor_sync(0xffffffffu, kqb, o);
             }
             const float gab = ca.x * cb.x;
             const f32x2 g2 = pack2(gab, gab);
@@ -426,7 +440,7 @@ delta_scan_kernel(const DeltaArgs a, const float* __restrict__ rows, float* __re
                 s[i][1] = mul2(g2, s[i][1]);
             }
             const float ua = ca.y * fmaf(-ca.x, ska, va);
-            const float ub = cb.y * fmaf(-cb.x, fmaf(ca.x, skb, kkb * ua), vb);
+            const float ub = cb.y * fmaf(-cb.x, fmaf(ca.x, skb, cb.w * ua), vb);
             const float wa = cb.x * ua;                  // the first write, decayed once
             const f32x2 a2 = pack2(wa, wa), b2 = pack2(ub, ub);
 #pragma unroll
@@ -434,18 +448,20 @@ delta_scan_kernel(const DeltaArgs a, const float* __restrict__ rows, float* __re
                 s[i][0] = fma2(kb[i].x, b2, fma2(ka[i].x, a2, s[i][0]));
                 s[i][1] = fma2(kb[i].y, b2, fma2(ka[i].y, a2, s[i][1]));
             }
-            load_rows(ka, nxt + ER);
-            load_rows(kb, nxt2 + ER);
+            load_rows(ka, tok + 2 * QK + ER);
+            load_rows(kb, tok + 3 * QK + ER);
             if (writes) {
                 o_at[0] = fmaf(ca.x, sqa, ca.z * ua);
                 o_at[o_row] = fmaf(cb.x, fmaf(ca.x, sqb, kqb * ua), cb.z * ub);
             }
             o_at += 2 * o_row;
+            v_at += 2 * DS_COLS;
+            s_at += 2 * DR_SCALARS;
         }
         if (tok == last) {
             const float sk = column_sum(state_dot(ka)), sq = column_sum(state_dot(qa));
-            const float4 c = *reinterpret_cast<const float4*>(tok + 2 * ER + DS_COLS);
-            const float u = c.y * fmaf(-c.x, sk, tok[2 * ER + my]);
+            const float4 c = *reinterpret_cast<const float4*>(s_at);
+            const float u = c.y * fmaf(-c.x, sk, v_at[0]);
             const f32x2 g2 = pack2(c.x, c.x), u2 = pack2(u, u);
 #pragma unroll
             for (int i = 0; i < R4; ++i) {
@@ -455,7 +471,8 @@ delta_scan_kernel(const DeltaArgs a, const float* __restrict__ rows, float* __re
             if (writes) o_at[0] = fmaf(c.x, sq, c.z * u);
             o_at += o_row;
         }
-        __syncthreads();                                // before this buffer is fetched into again
+        __syncthreads();                                // every read of this buffer is done
+        if (threadIdx.x == 0 && b0 + 2 * DS_TOKENS < n) fetch(b0 + 2 * DS_TOKENS);
     }
 #pragma unroll
     for (int i = 0; i < R4; ++i)
@@ -472,7 +489,7 @@ delta_step_kernel(const DeltaArgs a, const float* __restrict__ norm_w, float eps
                   T* __restrict__ out) {
     constexpr int ER = 32 * R4;
     chain_release();
-    extern __shared__ __align__(16) float smem[];
+    extern __shared__ __align__(128) float smem[];
     float* q_s = smem;                                  // [ER]
     float* k_s = q_s + ER;                              // [ER]
     float* v_s = k_s + ER;                              // [fr]
@@ -643,15 +660,17 @@ int launch_prep(const DeltaArgs& a, float* out, cudaStream_t stream) {
     return launch_status();
 }
 template <int R4>
-int launch_scan(const DeltaArgs& a, const float* rows, float* out, cudaStream_t stream) {
-    const size_t smem = (size_t)2 * DS_TOKENS * (2 * 32 * R4 + DS_COLS + 4) * sizeof(float);
-    if (smem > 48 * 1024) {
+int launch_scan(const DeltaArgs& a, const float* rows, float* out, int* status,
+                cudaStream_t stream) {
+    constexpr size_t qk = 2 * 32 * R4;
+    const size_t smem = (2 * DS_TOKENS * (qk + DS_COLS + DR_SCALARS) + 4 * qk) * sizeof(float);
+    if (smem > 40 * 1024) {                             // (static shared memory comes on top)
         const int rc = (int)cudaFuncSetAttribute(delta_scan_kernel<R4>,
                                                  cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (rc) return rc;
     }
     MLS_LAUNCH((delta_scan_kernel<R4>), dim3(a.fr / DS_COLS, a.H, a.n_requests), dim3(DS_THREADS),
-               smem, stream, a, rows, out);
+               smem, stream, a, rows, out, status);
     return launch_status();
 }
 template <int R4, int C>
@@ -661,7 +680,7 @@ int launch_step(const DeltaArgs& a, const float* norm_w, float eps, void* out, i
     if (smem > 200 * 1024) return MLS_ERR_UNSUPPORTED;
     if (dtype == MLS_BF16) {
         auto kernel = delta_step_kernel<R4, C, __nv_bfloat16>;
-        if (smem > 48 * 1024) {
+        if (smem > 40 * 1024) {
             const int rc = (int)cudaFuncSetAttribute(
                 kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
             if (rc) return rc;
@@ -670,7 +689,7 @@ int launch_step(const DeltaArgs& a, const float* norm_w, float eps, void* out, i
                    (__nv_bfloat16*)out);
     } else {
         auto kernel = delta_step_kernel<R4, C, float>;
-        if (smem > 48 * 1024) {
+        if (smem > 40 * 1024) {
             const int rc = (int)cudaFuncSetAttribute(
                 kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
             if (rc) return rc;
@@ -682,9 +701,9 @@ int launch_step(const DeltaArgs& a, const float* norm_w, float eps, void* out, i
 }
 }  // namespace
 
-// Floats of one prepared row, and of a request's state.
+// Floats of a token's share of what the scan reads, and of a request's state.
 MLS_API int mls_delta_row_floats(int H, int G, int e, int f) {
-    return row_layout(H, G, (e + 31) / 32 * 32, (f + 15) / 16 * 16).row;
+    return prepared_floats(H, G, (e + 31) / 32 * 32, (f + 15) / 16 * 16);
 }
 MLS_API long long mls_delta_state_floats(int H, int G, int e, int f, int taps) {
     const long long s = (long long)H * ((f + 15) / 16 * 16) * ((e + 31) / 32 * 32) +
@@ -715,21 +734,22 @@ MLS_API int mls_delta_prep(const float* proj, int width, int qkv_col, int a_col,
 MLS_API int mls_delta_scan(const float* rows, const float* proj, int width, int qkv_col, int taps,
                            const int* state_slot, const int* cu_q, const int* positions,
                            float* state, long long state_stride, int n_tokens, int n_requests,
-                           int H, int G, int e, int f, float* out, cudaStream_t stream) {
+                           int H, int G, int e, int f, float* out, int* status,
+                           cudaStream_t stream) {
     if (n_tokens <= 0 || n_requests <= 0) return 0;
     const DeltaArgs a = make_args(proj, 1, 0, width, qkv_col, 0, 0, 0, nullptr, 0, taps, nullptr, nullptr,
                                   state_slot, cu_q, nullptr, positions, state, state_stride,
                                   n_tokens, n_requests, H, G, e, f);
     if (!sizes_ok(a) || n_requests > 65535 || H > 65535) return MLS_ERR_UNSUPPORTED;
     switch (a.er / 32) {
-        case 1: return launch_scan<1>(a, rows, out, stream);
-        case 2: return launch_scan<2>(a, rows, out, stream);
-        case 3: return launch_scan<3>(a, rows, out, stream);
-        case 4: return launch_scan<4>(a, rows, out, stream);
-        case 5: return launch_scan<5>(a, rows, out, stream);
-        case 6: return launch_scan<6>(a, rows, out, stream);
-        case 7: return launch_scan<7>(a, rows, out, stream);
-        default: return launch_scan<8>(a, rows, out, stream);
+        case 1: return launch_scan<1>(a, rows, out, status, stream);
+        case 2: return launch_scan<2>(a, rows, out, status, stream);
+        case 3: return launch_scan<3>(a, rows, out, status, stream);
+        case 4: return launch_scan<4>(a, rows, out, status, stream);
+        case 5: return launch_scan<5>(a, rows, out, status, stream);
+        case 6: return launch_scan<6>(a, rows, out, status, stream);
+        case 7: return launch_scan<7>(a, rows, out, status, stream);
+        default: return launch_scan<8>(a, rows, out, status, stream);
     }
 }
 

@@ -836,7 +836,7 @@ class Ops:
                                   _I, _I, _I, _I, _I, _P, _P]),
                    "scan": _decl(lib, "mls_delta_scan",
                                  [_P, _P, _I, _I, _I, _P, _P, _P, _P, _LL, _I, _I, _I, _I, _I, _I, _P,
-                                  _P]),
+                                  _P, _P]),
                    "step": _decl(lib, "mls_delta_step",
                                  [_P, _I, _LL, _I, _I, _I, _I, _I, _P, _I, _I, _P, _P, _P, _F, _P, _P,
                                   _P, _P, _LL, _I, _I, _I, _I, _I, _P, _I, _P])}
@@ -1495,7 +1495,7 @@ class Ops:
                 p.release()
 
     def delta_rows(self, n_heads: int, n_kv: int, e: int, f: int) -> int:
-        """Floats of a token's prepared row (``delta_prep``)."""
+        """Floats of a token's share of what ``delta_prep`` leaves for ``delta_scan``."""
         return int(self._part_lib("delta")["row"](n_heads, n_kv, e, f))
 
     def delta_state_floats(self, n_heads: int, n_kv: int, e: int, f: int, taps: int) -> int:
@@ -1554,7 +1554,7 @@ class Ops:
         _check(self._part_lib("delta")["scan"](
             _ptr(rows), _ptr(proj), proj.shape[1], col, taps, _ptr(step.state_slot), _ptr(step.cu_q),
             _ptr(step.positions), _ptr(state), state.stride(0), t, step.n_requests, n_heads, n_kv, e,
-            f, _ptr(out), self._stream()), "delta_scan")
+            f, _ptr(out), _ptr(self.status), self._stream()), "delta_scan")
 
     def delta_step(self, proj, cols: tuple, conv, taps: int, a_exp, dt_bias, norm_w, eps: float,
                    state, step, n_heads: int, n_kv: int, e: int, f: int, out) -> None:

@@ -26,8 +26,8 @@
 // token's row never falls on a row that its own convolution reads.  Rows of positions before
 // the sequence's start are never read.
 //
-// A warp owns four columns of S with eight lanes a column; a lane keeps er / 8 rows of its
-// column in registers, four neighbouring rows at a time (16-byte accesses of the state and of
+// A warp owns columns of S with eight lanes a column; a lane keeps er / 8 rows of each of its
+// columns in registers, four neighbouring rows at a time (16-byte accesses of the state and of
 // k and q), and multiplies them two at a time (fma.rn.f32x2).  The sum over the rows is the
 // lane's own in a fixed order and three shuffles: a token's bits do not depend on the batch.
 // The scan takes two tokens at a time from a portion's start, which moves the last bits where
@@ -314,16 +314,17 @@ delta_prep_kernel(const DeltaArgs a, float* __restrict__ out) {
 }
 
 constexpr int DS_COLS = DR_COLS;       // columns of S a CTA of the scan owns
-constexpr int DS_THREADS = 128;        // four warps, four columns each
 constexpr int DS_TOKENS = 16;          // tokens in one of the two buffers
 
-// R4: groups of four rows a lane keeps, er = 32 R4.
-template <int R4>
-__global__ void __launch_bounds__(DS_THREADS)
+// R4: groups of four rows a lane keeps, er = 32 R4.  C: columns a lane keeps (a warp has 4 C): with
+// two, what a lane reads of k and q serves twice.
+template <int R4, int C>
+__global__ void __launch_bounds__(128 / C)
 delta_scan_kernel(const DeltaArgs a, const float* __restrict__ rows, float* __restrict__ out,
                   int* status) {
     using namespace mls_tma;
     constexpr int ER = 32 * R4, QK = 2 * ER;           // floats of a token's q and k
+    constexpr int DS_THREADS = 128 / C;
     constexpr int V_AT = DS_TOKENS * QK, S_AT = V_AT + DS_TOKENS * DS_COLS;
     constexpr int BUF = S_AT + DS_TOKENS * DR_SCALARS;
     chain_release();
@@ -333,7 +334,7 @@ delta_scan_kernel(const DeltaArgs a, const float* __restrict__ rows, float* __re
     __shared__ __align__(8) uint64_t full_bars[2];
     const int r = blockIdx.z, head = blockIdx.y, col0 = blockIdx.x * DS_COLS;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, grp = lane & 7;
-    const int my = warp * 4 + (lane >> 3), col = col0 + my;
+    const int my = warp * 4 * C + (lane >> 3);         // my columns: this one and every fourth behind it
     const Prepared from(a.n_tokens, a.H, a.G, ER, a.fr);
     const int t0 = a.cu_q[r], n = a.cu_q[r + 1] - t0;
     if (n <= 0) return;
@@ -359,14 +360,17 @@ delta_scan_kernel(const DeltaArgs a, const float* __restrict__ rows, float* __re
         fetch(0);
         if (n > DS_TOKENS) fetch(DS_TOKENS);
     }
-    float* S = a.state + (size_t)slot * a.state_stride + ((size_t)head * a.fr + col) * ER + 4 * grp;
-    f32x2 s[R4][2];
+    float* S = a.state + (size_t)slot * a.state_stride +
+               ((size_t)head * a.fr + col0 + my) * ER + 4 * grp;
+    f32x2 s[C][R4][2];
 #pragma unroll
-    for (int i = 0; i < R4; ++i) {
-        const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(S + 32 * i);
-        s[i][0] = v.x;
-        s[i][1] = v.y;
-    }
+    for (int ci = 0; ci < C; ++ci)
+#pragma unroll
+        for (int i = 0; i < R4; ++i) {
+            const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(S + 4 * ci * ER + 32 * i);
+            s[ci][i][0] = v.x;
+            s[ci][i][1] = v.y;
+        }
     // the convolution's last inputs (the preparation has read the older ones)
     {
         const int keep = a.taps - 1, i0 = max(0, n - keep);
@@ -379,19 +383,18 @@ delta_scan_kernel(const DeltaArgs a, const float* __restrict__ rows, float* __re
                 ring[row + c] = a.proj[(size_t)(t0 + i) * a.width + a.qkv_col + c];
         }
     }
-    const bool writes = grp == 0 && col < a.f;
     const size_t o_row = (size_t)a.H * a.f;
-    float* o_at = out + (size_t)t0 * o_row + (size_t)head * a.f + col;
+    float* o_at = out + (size_t)t0 * o_row + (size_t)head * a.f + col0 + my;
     auto load_rows = [&](ulonglong2 (&v)[R4], const float* src) {
 #pragma unroll
         for (int i = 0; i < R4; ++i) v[i] = *reinterpret_cast<const ulonglong2*>(src + 32 * i + 4 * grp);
     };
-    auto state_dot = [&](const ulonglong2 (&v)[R4]) {         // this lane's share of S^T v
+    auto state_dot = [&](const f32x2 (&st)[R4][2], const ulonglong2 (&v)[R4]) {   // a lane's share
         f32x2 d0 = 0ull, d1 = 0ull;
 #pragma unroll
         for (int i = 0; i < R4; ++i) {
-            d0 = fma2(s[i][0], v[i].x, d0);
-            d1 = fma2(s[i][1], v[i].y, d1);
+            d0 = fma2(st[i][0], v[i].x, d0);
+            d1 = fma2(st[i][1], v[i].y, d1);
         }
         return sum2(add2(d0, d1));
     };
@@ -405,78 +408,113 @@ delta_scan_kernel(const DeltaArgs a, const float* __restrict__ rows, float* __re
             if (threadIdx.x == 0 && status) atomicOr(status, MLS_STATUS_TIMEOUT);
             return;
         }
-        const float* tok = smem + (size_t)(pass & 1) * BUF;          // q and k of the present token
-        const float* v_at = tok + V_AT + my;
-        const float* s_at = tok + S_AT;
-        const float* last = tok + (nb - 1) * QK;
+        const float* buf = smem + (size_t)(pass & 1) * BUF;
         ulonglong2 ka[R4], qa[R4], kb[R4], qb[R4];
-        load_rows(qa, tok);
-        load_rows(ka, tok + ER);
-        load_rows(qb, tok + QK);
-        load_rows(kb, tok + QK + ER);
+        load_rows(qa, buf);
+        load_rows(ka, buf + ER);
+        load_rows(qb, buf + QK);
+        load_rows(kb, buf + QK + ER);
+        float keep[C];                                  // lane grp keeps the output of one token of eight
+        auto store = [&](int first, int count) {        // of the eight tokens from `first` on
+            if (grp < count) {
+#pragma unroll
+                for (int ci = 0; ci < C; ++ci)
+                    if (col0 + my + 4 * ci < a.f)
+                        o_at[(size_t)(b0 + first + grp) * o_row + 4 * ci] = keep[ci];
+            }
+        };
         // Two tokens at a time: both tokens' products with the state before them cross the lanes
         // together, and what the first token changed of the second's follows from the products
         // of its key with the second's key and query.
-        for (; tok < last; tok += 2 * QK) {
-            float sqa = state_dot(qa), sqb = state_dot(qb), ska = state_dot(ka), skb = state_dot(kb);
-            const float va = v_at[0], vb = v_at[DS_COLS];
-            const float4 ca = *reinterpret_cast<const float4*>(s_at);
-            const float4 cb = *reinterpret_cast<const float4*>(s_at + DR_SCALARS);
-            const float kqb = s_at[DR_SCALARS + 4];
+        auto pair = [&](int tt) {
+            const float* tok = buf + tt * QK;
+            const float* sc = buf + S_AT + tt * DR_SCALARS;
+            const float* v = buf + V_AT + tt * DS_COLS + my;
+            float sqa[C], sqb[C], ska[C], skb[C];
+#pragma unroll
+            for (int ci = 0; ci < C; ++ci) {
+                ska[ci] = state_dot(s[ci], ka);
+                skb[ci] = state_dot(s[ci], kb);
+                sqa[ci] = state_dot(s[ci], qa);
+                sqb[ci] = state_dot(s[ci], qb);
+            }
+            const float4 ca = *reinterpret_cast<const float4*>(sc);
+            const float4 cb = *reinterpret_cast<const float4*>(sc + DR_SCALARS);
+            const float kqb = sc[DR_SCALARS + 4];
             load_rows(qa, tok + 2 * QK);
             load_rows(qb, tok + 3 * QK);
 #pragma unroll
-            for (int o = 1; o < 8; o <<= 1) {
-                ska += __shfl_xor_sync(0xffffffffu, ska, o);
-                skb += __shfl_xor_sync(0xffffffffu, skb, o);
-                sqa += __shfl_xor_sync(0xffffffffu, sqa, o);
-                sqb += __shfl_xor_sync(0xffffffffu, sqb, o);
-            }
+            for (int o = 1; o < 8; o <<= 1)
+#pragma unroll
+                for (int ci = 0; ci < C; ++ci) {
+                    ska[ci] += __shfl_xor_sync(0xffffffffu, ska[ci], o);
+                    skb[ci] += __shfl_xor_sync(0xffffffffu, skb[ci], o);
+                    sqa[ci] += __shfl_xor_sync(0xffffffffu, sqa[ci], o);
+                    sqb[ci] += __shfl_xor_sync(0xffffffffu, sqb[ci], o);
+                }
             const float gab = ca.x * cb.x;
             const f32x2 g2 = pack2(gab, gab);
 #pragma unroll
-            for (int i = 0; i < R4; ++i) {
-                s[i][0] = mul2(g2, s[i][0]);
-                s[i][1] = mul2(g2, s[i][1]);
-            }
-            const float ua = ca.y * fmaf(-ca.x, ska, va);
-            const float ub = cb.y * fmaf(-cb.x, fmaf(ca.x, skb, cb.w * ua), vb);
-            const float wa = cb.x * ua;                  // the first write, decayed once
-            const f32x2 a2 = pack2(wa, wa), b2 = pack2(ub, ub);
+            for (int ci = 0; ci < C; ++ci) {
 #pragma unroll
-            for (int i = 0; i < R4; ++i) {
-                s[i][0] = fma2(kb[i].x, b2, fma2(ka[i].x, a2, s[i][0]));
-                s[i][1] = fma2(kb[i].y, b2, fma2(ka[i].y, a2, s[i][1]));
+                for (int i = 0; i < R4; ++i) {
+                    s[ci][i][0] = mul2(g2, s[ci][i][0]);
+                    s[ci][i][1] = mul2(g2, s[ci][i][1]);
+                }
+                const float va = v[4 * ci], vb = v[DS_COLS + 4 * ci];
+                const float ua = ca.y * fmaf(-ca.x, ska[ci], va);
+                const float ub = cb.y * fmaf(-cb.x, fmaf(ca.x, skb[ci], cb.w * ua), vb);
+                const float wa = cb.x * ua;              // the first write, decayed once
+                const f32x2 a2 = pack2(wa, wa), b2 = pack2(ub, ub);
+#pragma unroll
+                for (int i = 0; i < R4; ++i) {
+                    s[ci][i][0] = fma2(kb[i].x, b2, fma2(ka[i].x, a2, s[ci][i][0]));
+                    s[ci][i][1] = fma2(kb[i].y, b2, fma2(ka[i].y, a2, s[ci][i][1]));
+                }
+                const float oa = fmaf(ca.x, sqa[ci], ca.z * ua);
+                const float ob = fmaf(cb.x, fmaf(ca.x, sqb[ci], kqb * ua), cb.z * ub);
+                if (grp == (tt & 7)) keep[ci] = oa;
+                if (grp == (tt & 7) + 1) keep[ci] = ob;
             }
             load_rows(ka, tok + 2 * QK + ER);
             load_rows(kb, tok + 3 * QK + ER);
-            if (writes) {
-                o_at[0] = fmaf(ca.x, sqa, ca.z * ua);
-                o_at[o_row] = fmaf(cb.x, fmaf(ca.x, sqb, kqb * ua), cb.z * ub);
-            }
-            o_at += 2 * o_row;
-            v_at += 2 * DS_COLS;
-            s_at += 2 * DR_SCALARS;
-        }
-        if (tok == last) {
-            const float sk = column_sum(state_dot(ka)), sq = column_sum(state_dot(qa));
-            const float4 c = *reinterpret_cast<const float4*>(s_at);
-            const float u = c.y * fmaf(-c.x, sk, v_at[0]);
-            const f32x2 g2 = pack2(c.x, c.x), u2 = pack2(u, u);
+            if ((tt & 7) == 6) store(tt - 6, 8);
+        };
+        if (nb == DS_TOKENS) {
+#pragma unroll 4
+            for (int tt = 0; tt < DS_TOKENS; tt += 2) pair(tt);
+        } else {
+            int tt = 0;
+#pragma unroll 1
+            for (; tt + 1 < nb; tt += 2) pair(tt);
+            if (tt < nb) {
+                const float4 c = *reinterpret_cast<const float4*>(buf + S_AT + tt * DR_SCALARS);
+                const f32x2 g2 = pack2(c.x, c.x);
 #pragma unroll
-            for (int i = 0; i < R4; ++i) {
-                s[i][0] = fma2(ka[i].x, u2, mul2(g2, s[i][0]));
-                s[i][1] = fma2(ka[i].y, u2, mul2(g2, s[i][1]));
+                for (int ci = 0; ci < C; ++ci) {
+                    const float sk = column_sum(state_dot(s[ci], ka)), sq = column_sum(state_dot(s[ci], qa));
+                    const float u = c.y * fmaf(-c.x, sk, buf[V_AT + tt * DS_COLS + my + 4 * ci]);
+                    const f32x2 u2 = pack2(u, u);
+#pragma unroll
+                    for (int i = 0; i < R4; ++i) {
+                        s[ci][i][0] = fma2(ka[i].x, u2, mul2(g2, s[ci][i][0]));
+                        s[ci][i][1] = fma2(ka[i].y, u2, mul2(g2, s[ci][i][1]));
+                    }
+                    if (grp == (tt & 7)) keep[ci] = fmaf(c.x, sq, c.z * u);
+                }
+                ++tt;
             }
-            if (writes) o_at[0] = fmaf(c.x, sq, c.z * u);
-            o_at += o_row;
+            if (tt & 7) store(tt & ~7, tt & 7);
         }
         __syncthreads();                                // every read of this buffer is done
         if (threadIdx.x == 0 && b0 + 2 * DS_TOKENS < n) fetch(b0 + 2 * DS_TOKENS);
     }
 #pragma unroll
-    for (int i = 0; i < R4; ++i)
-        *reinterpret_cast<ulonglong2*>(S + 32 * i) = make_ulonglong2(s[i][0], s[i][1]);
+    for (int ci = 0; ci < C; ++ci)
+#pragma unroll
+        for (int i = 0; i < R4; ++i)
+            *reinterpret_cast<ulonglong2*>(S + 4 * ci * ER + 32 * i) =
+                make_ulonglong2(s[ci][i][0], s[ci][i][1]);
 }
 
 constexpr int DT_THREADS = 256;        // eight warps of a (request, head)
@@ -659,17 +697,17 @@ int launch_prep(const DeltaArgs& a, float* out, cudaStream_t stream) {
     else MLS_LAUNCH((delta_prep_kernel<NI, 16>), grid, dim3(DP_WARPS * 32), 0, stream, a, out);
     return launch_status();
 }
-template <int R4>
+template <int R4, int C>
 int launch_scan(const DeltaArgs& a, const float* rows, float* out, int* status,
                 cudaStream_t stream) {
     constexpr size_t qk = 2 * 32 * R4;
     const size_t smem = (2 * DS_TOKENS * (qk + DS_COLS + DR_SCALARS) + 4 * qk) * sizeof(float);
     if (smem > 40 * 1024) {                             // (static shared memory comes on top)
-        const int rc = (int)cudaFuncSetAttribute(delta_scan_kernel<R4>,
-                                                 cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        const int rc = (int)cudaFuncSetAttribute(
+            delta_scan_kernel<R4, C>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (rc) return rc;
     }
-    MLS_LAUNCH((delta_scan_kernel<R4>), dim3(a.fr / DS_COLS, a.H, a.n_requests), dim3(DS_THREADS),
+    MLS_LAUNCH((delta_scan_kernel<R4, C>), dim3(a.fr / DS_COLS, a.H, a.n_requests), dim3(128 / C),
                smem, stream, a, rows, out, status);
     return launch_status();
 }
@@ -742,14 +780,14 @@ MLS_API int mls_delta_scan(const float* rows, const float* proj, int width, int 
                                   n_tokens, n_requests, H, G, e, f);
     if (!sizes_ok(a) || n_requests > 65535 || H > 65535) return MLS_ERR_UNSUPPORTED;
     switch (a.er / 32) {
-        case 1: return launch_scan<1>(a, rows, out, status, stream);
-        case 2: return launch_scan<2>(a, rows, out, status, stream);
-        case 3: return launch_scan<3>(a, rows, out, status, stream);
-        case 4: return launch_scan<4>(a, rows, out, status, stream);
-        case 5: return launch_scan<5>(a, rows, out, status, stream);
-        case 6: return launch_scan<6>(a, rows, out, status, stream);
-        case 7: return launch_scan<7>(a, rows, out, status, stream);
-        default: return launch_scan<8>(a, rows, out, status, stream);
+        case 1: return launch_scan<1, 2>(a, rows, out, status, stream);
+        case 2: return launch_scan<2, 2>(a, rows, out, status, stream);
+        case 3: return launch_scan<3, 2>(a, rows, out, status, stream);
+        case 4: return launch_scan<4, 2>(a, rows, out, status, stream);
+        case 5: return launch_scan<5, 1>(a, rows, out, status, stream);
+        case 6: return launch_scan<6, 1>(a, rows, out, status, stream);
+        case 7: return launch_scan<7, 1>(a, rows, out, status, stream);
+        default: return launch_scan<8, 1>(a, rows, out, status, stream);
     }
 }
 

@@ -779,16 +779,21 @@ MLS_API int mls_delta_scan(const float* rows, const float* proj, int width, int 
                                   state_slot, cu_q, nullptr, positions, state, state_stride,
                                   n_tokens, n_requests, H, G, e, f);
     if (!sizes_ok(a) || n_requests > 65535 || H > 65535) return MLS_ERR_UNSUPPORTED;
+    // one column a lane while every CTA has an SM to itself (more warps to hide the chain of
+    // products and sums), two beyond that (half the reads of k and q); the bits are the same
+    const bool one = (long long)(a.fr / DS_COLS) * H * n_requests <= sm_count();
+#define DS_GO(R, C) return launch_scan<R, C>(a, rows, out, status, stream)
     switch (a.er / 32) {
-        case 1: return launch_scan<1, 2>(a, rows, out, status, stream);
-        case 2: return launch_scan<2, 2>(a, rows, out, status, stream);
-        case 3: return launch_scan<3, 2>(a, rows, out, status, stream);
-        case 4: return launch_scan<4, 2>(a, rows, out, status, stream);
-        case 5: return launch_scan<5, 1>(a, rows, out, status, stream);
-        case 6: return launch_scan<6, 1>(a, rows, out, status, stream);
-        case 7: return launch_scan<7, 1>(a, rows, out, status, stream);
-        default: return launch_scan<8, 1>(a, rows, out, status, stream);
+        case 1: if (one) DS_GO(1, 1); DS_GO(1, 2);
+        case 2: if (one) DS_GO(2, 1); DS_GO(2, 2);
+        case 3: if (one) DS_GO(3, 1); DS_GO(3, 2);
+        case 4: if (one) DS_GO(4, 1); DS_GO(4, 2);
+        case 5: DS_GO(5, 1);
+        case 6: DS_GO(6, 1);
+        case 7: DS_GO(7, 1);
+        default: DS_GO(8, 1);
     }
+#undef DS_GO
 }
 
 // A step of one token a request, to the gated and normed heads: out [T, H f] in `dtype`.

@@ -238,6 +238,21 @@ def test_delta_scan_alone_and_a_used_slot(rt32):
     assert np.abs(np.concatenate(odd) - first).max() < 2e-6 * scale
 
 
+@pytest.mark.parametrize("e", [20, 64, 90, 128])
+def test_delta_scan_does_not_depend_on_the_batch(rt32, e):
+    """Alone (every block of columns has an SM to itself) and beside eleven others (it has not): the
+    same bits."""
+    ops = rt32.ops
+    case = DeltaCase(4, 2, e, 64, 3, (37,), seed=4)
+    state = case.new_state(ops, 12)
+    alone, _ = case.prompt(ops, state, [(0, 0, 37)], [5], torch.float32)
+    kept = state[5].clone()
+    state.zero_()
+    many, _ = case.prompt(ops, state, [(0, 0, 37)] * 12, list(range(12)), torch.float32)
+    assert all(np.array_equal(many[37 * i:37 * (i + 1)], alone) for i in range(12))
+    assert torch.equal(state, kept.expand(12, -1))
+
+
 def test_delta_bfloat16_outputs(rt32):
     ops = rt32.ops
     case = DeltaCase(4, 2, 64, 32, 4, (20,), seed=9)

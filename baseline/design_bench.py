@@ -1,6 +1,6 @@
 """``bench.py --design zededra | logulix | zefenex | movazen | nekedra``: prefill and decode
-throughput of the design's layers at sizes that resemble a real model's, beside the dense Llama-style decoder at equal
-size.
+throughput of the design's layers at sizes that resemble a real model's, beside the dense
+Llama-style decoder at equal size.
 
 Every model has random weights (N(0, 0.02^2), drawn on the device), ``--layers`` layers
 (default 4) and the same width, head count, head size, feed-forward width and bytes of

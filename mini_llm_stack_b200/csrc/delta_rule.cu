@@ -405,7 +405,13 @@ delta_scan_kernel(const DeltaArgs a, const float* __restrict__ rows, float* __re
                                 (pass >> 1) & 1) ? 1 : 0;
         __syncthreads();
         if (!arrived) {                                 // every thread leaves at the same place
-            if (threadIdx.x == 0 && status) atomicOr(status, MLS_STATUS_TIMEOUT);
+            if (threadIdx.x == 0) {                     // (once the copies under way are done, or given up)
+                if (status) atomicOr(status, MLS_STATUS_TIMEOUT);
+                mbar_wait((uint32_t)__cvta_generic_to_shared(&full_bars[pass & 1]), (pass >> 1) & 1);
+                if (b0 + DS_TOKENS < n)
+                    mbar_wait((uint32_t)__cvta_generic_to_shared(&full_bars[(pass + 1) & 1]),
+                              ((pass + 1) >> 1) & 1);
+            }
             return;
         }
         const float* buf = smem + (size_t)(pass & 1) * BUF;

@@ -13,8 +13,8 @@ Here the model's cache slots (one per layer call that owns a cache) are sorted
 into groups by what they need.  Slots with the same ``PagedKV`` spec share one
 page pool and one block table per request (a page id means the same page in
 every member of the group, as one table serves all layers in the reference);
-a group with a window gives pages back as soon as the window has passed them (but
-never the pages of the sequence's first ``keep_first`` tokens, if the spec names some).
+a group with a window (or with chunks) gives pages back as soon as the window (the
+chunk) has passed them (but never the pages of the sequence's first ``keep_first`` tokens, if the spec names some).
 Slots with a ``FixedState`` spec share the request's state slot.  A slot whose spec is
 ``PagedWithState`` is a member of a paged group and of a fixed group at once.
 
@@ -175,10 +175,10 @@ class CacheManager:
         """Most pages of group ``g`` a request of ``n_tokens`` holds at one time
         when it is fed at most ``portion`` tokens a step (all at once if None)."""
         need = self.pages_for(n_tokens)
-        w = g.spec.window
+        w = g.spec.span
         if w is not None and portion is not None:
-            # keys older than the window are given back after every step; one
-            # page more because the live span need not start at a page's edge
+            # keys older than the window (or of earlier chunks) are given back after every
+            # step; one page more because the live span need not start at a page's edge
             need = min(need, self.pages_for(w - 1 + portion) + 1 + self._keep_pages(g))
         return need
 
@@ -250,12 +250,11 @@ class CacheManager:
         for g in self.paged:
             if rec.length > rec.n_pages[g.gid] * self.block_size:
                 raise CacheError(f"request {owner!r} stored tokens beyond its pages")
-            w = g.spec.window
-            if w is None:
+            if g.spec.span is None:
                 continue
-            # the next query sits at position >= length and sees keys
-            # j > position - w, so every key < length - w + 1 is never read again
-            dead = max(0, rec.length - w + 1) // self.block_size
+            # the next query sits at position >= length: every key before the first one
+            # it sees is never read again
+            dead = g.spec.first_key(rec.length) // self.block_size
             dead = min(dead, rec.n_pages[g.gid])
             # (the pages given back are those from the kept ones up to ``released``)
             first = max(rec.released[g.gid], self._keep_pages(g))
@@ -281,8 +280,8 @@ class CacheManager:
         if self.fixed:
             raise CacheError("a state of fixed size cannot be taken back to an earlier token")
         for g in self.paged:
-            w = g.spec.window
-            if w is not None and rec.released[g.gid] * self.block_size > max(0, n_tokens - w + 1):
+            w = g.spec.span
+            if w is not None and rec.released[g.gid] * self.block_size > g.spec.first_key(n_tokens):
                 raise CacheError(
                     f"request {owner!r}: pages behind the window of {w} were given back; "
                     f"it cannot be cut to {n_tokens} tokens")

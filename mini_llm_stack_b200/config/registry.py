@@ -87,5 +87,5 @@ def _ensure_builtin() -> None:
     if not _builtin_done:
         _builtin_done = True
         # (they register themselves)
-        from ..parts import (llama_dense, logulix, movazen, nekedra, zededra,  # noqa: F401
-                             zefenex)
+        from ..parts import (llama_dense, logulix, movazen, nekedra, sevazen,  # noqa: F401
+                             zededra, zefenex)

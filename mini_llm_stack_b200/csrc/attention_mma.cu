@@ -49,6 +49,8 @@ struct Params {
     float* part_o;                       // [splits, T * H, HD]   (split kernel, splits > 1)
     float* part_lse;                     // [splits, T * H]       (log2 domain)
     int max_blocks, n_req, n_tokens, n_heads, n_kv, group, block_size, window, n_split;
+    int chunk;                           // > 0 (and no window): a query sees its own chunk of so many
+                                         // tokens, counted from the sequence's start
     int small_only;                      // tile kernel: 1 = skip requests the split kernel takes
     int cluster_merge;                   // split TMA kernel: the splits of a request and kv head are
                                          // one cluster and merge through shared memory
@@ -172,12 +174,12 @@ __device__ __forceinline__ bool is_small(int q_len, int group) { return q_len * 
 // tiles than the longest request's.  The step's longest context lies one past the requests'
 // in ctx_len (the batch builder puts it there): all threads of the grid, and the merge
 // kernel, work the same number out from it, also when a captured step is replayed with
-// longer contexts.  With a window a small request (at most 16 new tokens) sees at most
-// window + 15 keys, which begin anywhere in a tile.
-__device__ __forceinline__ int tiles_per_split(const int* ctx_len, int n_req, int window, int bn,
+// longer contexts.  With a window, or chunks, of `span` tokens a small request (at most 16 new
+// tokens) sees at most span + 15 keys, which begin anywhere in a tile.
+__device__ __forceinline__ int tiles_per_split(const int* ctx_len, int n_req, int span, int bn,
                                                int n_split, int keep = 0) {
     int most = (ctx_len[n_req] + bn - 1) / bn;
-    if (window > 0) most = min(most, (window + 15 + bn - 2) / bn + 1 + (keep + bn - 1) / bn);
+    if (span > 0) most = min(most, (span + 15 + bn - 2) / bn + 1 + (keep + bn - 1) / bn);
     return (max(most, 1) + n_split - 1) / n_split;
 }
 
@@ -251,7 +253,7 @@ __global__ void __launch_bounds__(NT) attention_tile_kernel(const Params P) {
     const int i_first = row0 / P.group;
     const int i_last = (min(rows, row0 + 64) - 1) / P.group;
     const int hi = pos0 + i_last;
-    const int lo = P.window > 0 ? max(0, pos0 + i_first - P.window + 1) : 0;
+    const int lo = max(0, first_visible(pos0 + i_first, P.window, P.chunk));
     const int* table = P.block_table + (size_t)r * P.max_blocks;
     const TileRange R = tile_range(lo, hi, P.keep, BN);
     const int n_tiles = R.tiles_all;
@@ -264,8 +266,8 @@ __global__ void __launch_bounds__(NT) attention_tile_kernel(const Params P) {
     const int rA = row0 + warp * 16 + (lane >> 2), rB = rA + 8;
     const int pA = rA < rows ? pos0 + rA / P.group : -1;
     const int pB = rB < rows ? pos0 + rB / P.group : -1;
-    const int loA = P.window > 0 ? pA - P.window + 1 : 0;
-    const int loB = P.window > 0 ? pB - P.window + 1 : 0;
+    const int loA = first_visible(pA, P.window, P.chunk);
+    const int loB = first_visible(pB, P.window, P.chunk);
     const float slA = P.slopes ? P.slopes[kvh * P.group + rA % P.group] * LOG2E : 0.f;
     const float slB = P.slopes ? P.slopes[kvh * P.group + rB % P.group] * LOG2E : 0.f;
 
@@ -415,12 +417,12 @@ __global__ void __launch_bounds__(NT) attention_split_kernel(const Params P) {
     const int tok0 = P.cu_q[r], ctx = P.ctx_len[r];
     const int pos0 = ctx - q_len;
     const int hi = ctx - 1;
-    const int lo = P.window > 0 ? max(0, pos0 - P.window + 1) : 0;
+    const int lo = max(0, first_visible(pos0, P.window, P.chunk));
     const int* table = P.block_table + (size_t)r * P.max_blocks;
     const TileRange R = tile_range(lo, hi, P.keep, BN);
     const int tiles_all = R.tiles_all;
     const int per = P.n_split == 1 ? tiles_all
-        : tiles_per_split(P.ctx_len, P.n_req, P.window, BN, P.n_split, P.keep);
+        : tiles_per_split(P.ctx_len, P.n_req, P.window > 0 ? P.window : P.chunk, BN, P.n_split, P.keep);
     const int t_begin = split * per, t_end = min(tiles_all, t_begin + per);
     const int n_tiles = max(0, t_end - t_begin);
     if (n_tiles == 0) return;                         // a stretch past the request's end: the merge knows
@@ -428,8 +430,8 @@ __global__ void __launch_bounds__(NT) attention_split_kernel(const Params P) {
     const int rA = lane >> 2, rB = rA + 8;
     const int pA = rA < rows ? pos0 + rA / P.group : -1;
     const int pB = rB < rows ? pos0 + rB / P.group : -1;
-    const int loA = P.window > 0 ? pA - P.window + 1 : 0;
-    const int loB = P.window > 0 ? pB - P.window + 1 : 0;
+    const int loA = first_visible(pA, P.window, P.chunk);
+    const int loB = first_visible(pB, P.window, P.chunk);
     const float slA = P.slopes ? P.slopes[kvh * P.group + rA % P.group] * LOG2E : 0.f;
     const float slB = P.slopes ? P.slopes[kvh * P.group + rB % P.group] * LOG2E : 0.f;
 
@@ -610,9 +612,9 @@ __global__ void attention_merge_kernel(const Params P) {
     __shared__ int parts_here;
     if (threadIdx.x < 32) {
         // the stretches of this request that hold tiles: the others wrote nothing
-        const int per = tiles_per_split(P.ctx_len, P.n_req, P.window, BN, P.n_split, P.keep);
+        const int per = tiles_per_split(P.ctx_len, P.n_req, P.window > 0 ? P.window : P.chunk, BN, P.n_split, P.keep);
         const int ctx = P.ctx_len[r];
-        const int lo = P.window > 0 ? max(0, ctx - q_len - P.window + 1) : 0;
+        const int lo = max(0, first_visible(ctx - q_len, P.window, P.chunk));
         const int tiles_all = tile_range(lo, ctx - 1, P.keep, BN).tiles_all;
         if (threadIdx.x == 0) parts_here = min(P.n_split, (tiles_all + per - 1) / per);
     }
@@ -787,12 +789,12 @@ attention_split_tma_kernel(const Params P, const Fused F,
     const int tok0 = P.cu_q[r], ctx = P.ctx_len[r];
     const int pos0 = ctx - q_len;
     const int hi = ctx - 1;
-    const int lo = P.window > 0 ? max(0, pos0 - P.window + 1) : 0;
+    const int lo = max(0, first_visible(pos0, P.window, P.chunk));
     const int* table = P.block_table + (size_t)r * P.max_blocks;
     const int kbase0 = (lo / BN) * BN;
     const int tiles_all = (hi - kbase0) / BN + 1;
     const int per = P.n_split == 1 ? tiles_all
-        : tiles_per_split(P.ctx_len, P.n_req, P.window, BN, P.n_split);
+        : tiles_per_split(P.ctx_len, P.n_req, P.window > 0 ? P.window : P.chunk, BN, P.n_split);
     const int t_begin = split * per, t_end = min(tiles_all, t_begin + per);
     const int n_tiles = max(0, t_end - t_begin);
     if (n_tiles == 0 && !P.cluster_merge) {           // a stretch past the request's end: the merge
@@ -859,8 +861,8 @@ attention_split_tma_kernel(const Params P, const Fused F,
     const int rA = lane >> 2, rB = rA + 8;
     const int pA = rA < rows ? pos0 + rA / P.group : -1;
     const int pB = rB < rows ? pos0 + rB / P.group : -1;
-    const int loA = P.window > 0 ? pA - P.window + 1 : 0;
-    const int loB = P.window > 0 ? pB - P.window + 1 : 0;
+    const int loA = first_visible(pA, P.window, P.chunk);
+    const int loB = first_visible(pB, P.window, P.chunk);
 
     float o[HD / 8][4];
 #pragma unroll
@@ -1211,7 +1213,7 @@ attention_tile_tma_kernel(const Params P, const __grid_constant__ CUtensorMap km
     const int i_first = row0 / P.group;
     const int i_last = (min(rows, row0 + 64) - 1) / P.group;
     const int hi = pos0 + i_last;
-    const int lo = P.window > 0 ? max(0, pos0 + i_first - P.window + 1) : 0;
+    const int lo = max(0, first_visible(pos0 + i_first, P.window, P.chunk));
     const int* table = P.block_table + (size_t)r * P.max_blocks;
     const int kbase0 = (lo / BN) * BN;
     const int n_tiles = (hi - kbase0) / BN + 1;
@@ -1262,13 +1264,13 @@ attention_tile_tma_kernel(const Params P, const __grid_constant__ CUtensorMap km
     const int rA = row0 + warp * 16 + (lane >> 2), rB = rA + 8;
     const int pA = rA < rows ? pos0 + rA / P.group : -1;
     const int pB = rB < rows ? pos0 + rB / P.group : -1;
-    const int loA = P.window > 0 ? pA - P.window + 1 : 0;
-    const int loB = P.window > 0 ? pB - P.window + 1 : 0;
+    const int loA = first_visible(pA, P.window, P.chunk);
+    const int loB = first_visible(pB, P.window, P.chunk);
     // keys up to this position are seen by all 16 rows of the warp: no mask needed
     const int first_row = row0 + warp * 16;
     const int p_first = first_row < rows ? pos0 + first_row / P.group : -1;
     const int last_row = min(rows, first_row + 16) - 1;
-    const int lo_last = P.window > 0 ? pos0 + last_row / P.group - P.window + 1 : 0;
+    const int lo_last = first_visible(pos0 + last_row / P.group, P.window, P.chunk);
     const bool full_warp = first_row + 16 <= rows;
 
     float o[HD / 8][4];
@@ -1470,6 +1472,8 @@ constexpr int SPLIT_SMEM_MERGE = (128 + 4 * 16 * HD) * 4;
 constexpr int SPLIT_SMEM = SPLIT_SMEM_PIPE > SPLIT_SMEM_MERGE ? SPLIT_SMEM_PIPE : SPLIT_SMEM_MERGE;
 }  // namespace
 
+// window > 0: a query sees the last so many tokens; chunk > 0 (and no window): its own chunk of so
+// many tokens, counted from the sequence's start, up to itself.
 // softcap c > 0: scores become c * tanh(score / c) before the softmax.  sink (float32 [H] or
 // nullptr): exp(sink_h) joins the denominator of head h's softmax.
 // n_tiles: 64-row tiles the tile kernel has to run (0: none); n_small: 1 if any
@@ -1482,7 +1486,7 @@ MLS_API int mls_attention_mma(const void* qkv, void* out, const void* k_pool, co
                               int n_small, int n_split, float* part_o, float* part_lse,
                               long long pool_pages, int* status, int use_tma,
                               const float* sink, const float* slopes, int keep_first,
-                              long long out_stride, cudaStream_t stream) {
+                              long long out_stride, int chunk, cudaStream_t stream) {
     if (n_tokens <= 0 || n_req <= 0) return 0;
     if (n_heads % n_kv || n_split < 1 || n_split > MAX_SPLITS ||
         (n_split > 1 && (!part_o || !part_lse)))
@@ -1520,6 +1524,7 @@ MLS_API int mls_attention_mma(const void* qkv, void* out, const void* k_pool, co
     P.group = n_heads / n_kv;
     P.block_size = block_size;
     P.window = window;
+    P.chunk = window > 0 ? 0 : chunk;
     P.n_split = n_split;
     P.small_only = n_small ? 1 : 0;
     P.cluster_merge = 0;
@@ -1642,6 +1647,7 @@ MLS_API int mls_attention_decode_fused(const float* parts, int n_parts, long lon
     P.group = n_heads / n_kv;
     P.block_size = block_size;
     P.window = window;
+    P.chunk = 0;
     P.n_split = n_split;
     P.small_only = 1;
     P.cluster_merge = 0;

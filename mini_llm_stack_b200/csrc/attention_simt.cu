@@ -11,6 +11,8 @@
 // holds exp(sink_h): a term without key or value, not scaled and not capped.  With slopes
 // (one number per q head) the score loses slope_h * (p - j), the distance to the key, before
 // the cap.  With keep_first > 0 a window does not hide the sequence's first keep_first keys.
+// With chunks of c tokens (and no window) the query at position p sees its own chunk, keys
+// floor(p / c) c .. p.
 // A row of `out` may be wider than the heads (out_stride elements a token).  The paged walk follows the reference's decode
 // kernel (kernels/paged_attention.py:34-88): page = table[r, j / block],
 // offset = j % block, online softmax over chunks of keys.
@@ -69,7 +71,7 @@ attention_simt_kernel(const T* __restrict__ qkv, T* __restrict__ out,
                       int n_tokens, int n_heads, int n_kv, int hd, int block_size, float scale,
                       int window, float softcap, long long n_pages,
                       const float* __restrict__ sink, const float* __restrict__ slopes,
-                      int keep_first, long long out_stride) {
+                      int keep_first, long long out_stride, int chunk) {
     chain_release();
     chain_wait();
     __shared__ float q_s[WARPS][MAX_HD];
@@ -86,7 +88,7 @@ attention_simt_kernel(const T* __restrict__ qkv, T* __restrict__ out,
     for (int i = lane; i < hd; i += 32) q_s[warp][i] = Elem<T>::load(qp + i);
     __syncwarp();
 
-    const int j_lo = window > 0 ? max(0, p - window + 1) : 0;
+    const int j_lo = max(0, first_visible(p, window, chunk));
     const int* table = block_table + (size_t)r * max_blocks;
     const int nd = (hd + 31) / 32;
 
@@ -149,7 +151,7 @@ MLS_API int mls_attention_simt(const void* qkv, void* out, int dtype, const void
                                int n_heads, int n_kv, int hd, int block_size, float scale,
                                int window, float softcap, long long n_pages, const float* sink,
                                const float* slopes, int keep_first, long long out_stride,
-                               cudaStream_t stream) {
+                               int chunk, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (hd > MOST_HD || hd <= 0 || n_heads % n_kv) return MLS_ERR_UNSUPPORTED;
     if (out_stride <= 0) out_stride = (long long)n_heads * hd;
@@ -159,7 +161,7 @@ MLS_API int mls_attention_simt(const void* qkv, void* out, int dtype, const void
     MLS_LAUNCH((attention_simt_kernel<T, HD>), dim3(blocks), dim3(WARPS * 32), 0, stream,          \
                (const T*)qkv, (T*)out, (const T*)k_pool, (const T*)v_pool, block_table, max_blocks, \
                positions, req_of_token, n_tokens, n_heads, n_kv, hd, block_size, scale, window,    \
-               softcap, n_pages, sink, slopes, keep_first, out_stride)
+               softcap, n_pages, sink, slopes, keep_first, out_stride, window > 0 ? 0 : chunk)
     if (dtype == MLS_BF16) {
         if (hd <= 512) SIMT_GO(__nv_bfloat16, 512);
         else SIMT_GO(__nv_bfloat16, MOST_HD);

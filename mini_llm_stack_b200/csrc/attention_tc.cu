@@ -71,6 +71,8 @@ struct Params {
     const int* cu_q;
     const int* ctx_len;
     int max_blocks, n_req, n_heads, n_kv, group, block_size, window, small_only;
+    int chunk;                           // > 0 (and no window): a query sees its own chunk of so many
+                                         // tokens, counted from the sequence's start
     int two_tiles;                       // 1: a CTA owns two row tiles; 0: one, its keys in halves
     float scale_log2;
     float cap_over_scale, tanh_arg;      // a cap c on the scores: c / scale and 2 log2(e) scale / c
@@ -145,7 +147,7 @@ attention_tc_kernel(const Params P, const __grid_constant__ CUtensorMap kmap,
     const int i_first = row0 / P.group;
     const int i_last = (min(rows, row0 + tile_rows) - 1) / P.group;
     const int hi = pos0 + i_last;
-    const int lo = P.window > 0 ? max(0, pos0 + i_first - P.window + 1) : 0;
+    const int lo = max(0, first_visible(pos0 + i_first, P.window, P.chunk));
     const int* table = P.block_table + (size_t)r * P.max_blocks;
     const int kbase0 = (lo / BN) * BN;
     // with kept first keys: first the tiles of kept keys that lie wholly before the window's
@@ -343,7 +345,7 @@ attention_tc_kernel(const Params P, const __grid_constant__ CUtensorMap kmap,
         // lanes of tensor memory of its quarter (warp index modulo four).
         const int c = chain;
         const int pos = live ? pos0 + ti : -1;
-        const int lo_row = P.window > 0 ? pos - P.window + 1 : 0;
+        const int lo_row = first_visible(pos, P.window, P.chunk);
         const float slope_raw =
             (EXTRA && P.slopes && live) ? P.slopes[kvh * P.group + g] * P.inv_scale : 0.f;
         const uint32_t lane_base = (uint32_t)(quarter * 32) << 16;
@@ -613,7 +615,7 @@ MLS_API int mls_attention_tc(const void* qkv, void* out, const void* k_pool, con
                              float scale, int window, float softcap, int n_tiles, int n_tiles_wide,
                              int skip_small, long long pool_pages, int* status,
                              const float* sink, long long out_stride, const float* slopes,
-                             int keep_first, cudaStream_t stream) {
+                             int keep_first, int chunk, cudaStream_t stream) {
 #if MLS_HEAD_DIM == 64 || MLS_HEAD_DIM == 128
     if (n_tiles <= 0 || n_req <= 0) return 0;
     if (n_heads % n_kv) return MLS_ERR_UNSUPPORTED;
@@ -647,6 +649,7 @@ MLS_API int mls_attention_tc(const void* qkv, void* out, const void* k_pool, con
     P.group = n_heads / n_kv;
     P.block_size = block_size;
     P.window = window;
+    P.chunk = window > 0 ? 0 : chunk;
     P.small_only = skip_small ? 1 : 0;
     P.two_tiles = (n_tiles_wide > 0 && (long long)n_tiles_wide * n_kv >= sm_count()) ? 1 : 0;
     if (g_forced_rows == CHAIN_ROWS) P.two_tiles = 0;

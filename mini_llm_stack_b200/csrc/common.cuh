@@ -171,6 +171,13 @@ static __device__ __forceinline__ void angle_cos_sin(int position, double freq, 
     sincosf(r, &s, &c);
 }
 
+// The first key the query at position p sees: the last `window` tokens, or with chunks of
+// `chunk` tokens (counted from the sequence's start) its own chunk up to itself, or everything.
+// (Below zero where the window reaches past the start.)
+static __device__ __forceinline__ int first_visible(int p, int window, int chunk) {
+    return window > 0 ? p - window + 1 : (chunk > 0 ? p - p % chunk : 0);
+}
+
 // Streaming multiprocessors of the current device (148 on a B200), asked once.
 static inline int sm_count() {
     static const int n = [] {

@@ -1,7 +1,8 @@
 // Routed experts: choose, sort, multiply expert by expert, add up.
 //
 // mls_route_topk: scores s = sigmoid(z), or softmax(z) over all outputs, of float32 router
-//   logits z [T, E]; for every token the `top` largest scores (plus a per-output correction
+//   logits z [T, E], or (mode 2) the logits plus a bias themselves, whose softmax over the chosen
+//   ones gives the weights; for every token the `top` largest scores (plus a per-output correction
 //   that enters the choice only; the lowest index wins a tie) with the scores themselves as
 //   weights (optionally divided by their sum + renorm_eps).  With n_groups > 1 the outputs form
 //   n_groups equal groups of neighbours; a group's score is the sum of its two largest choice
@@ -15,6 +16,7 @@
 //   a = weight[slot] * h[token]
 //   (input scaling: the weight multiplies what enters the expert) or a = h[token]
 //   (output scaling, applied by the down product instead).
+// mls_expert_relu2: y[p, :] = relu(Wu[e] a)^2, experts without a gate.
 // mls_expert_down: per_slot[slot, :] = Wd[e] y[p, :] (times the weight with output
 //   scaling), float32.
 // mls_expert_combine: delta[t] = sum_j per_slot[t * top + j] + shared[t], j ascending; with a
@@ -33,7 +35,7 @@ constexpr int BM = 32, BN = 64, BK = 32, TM = 2, TN = 4;   // 256 threads
 constexpr int MAX_GROUPS = 256;
 
 __global__ void route_topk_kernel(const float* __restrict__ logits, int logit_stride, int n_tokens,
-                                  int n_experts, int top, int renorm, int softmax,
+                                  int n_experts, int top, int renorm, int mode,
                                   const float* __restrict__ correction, float renorm_eps,
                                   int n_groups, int keep_groups,
                                   int* __restrict__ idx, float* __restrict__ weight) {
@@ -45,6 +47,7 @@ __global__ void route_topk_kernel(const float* __restrict__ logits, int logit_st
     const int t = blockIdx.x * (blockDim.x >> 5) + warp;
     if (t >= n_tokens) return;
     const float* z = logits + (size_t)t * logit_stride;
+    const bool softmax = mode == 1, by_logit = mode == 2;     // (else sigmoid)
     // softmax over all outputs: the largest logit and the sum of exponentials, both in the
     // order of the lanes' strides, so a token's scores do not depend on its batch
     float z_max = 0.f, inv_sum = 1.f;
@@ -56,14 +59,19 @@ __global__ void route_topk_kernel(const float* __restrict__ logits, int logit_st
         for (int e = lane; e < n_experts; e += 32) sum += expf(z[e] - z_max);
         inv_sum = 1.0f / warp_sum(sum);
     }
+    // (in mode 2 the correction is a bias of the logits: part of the score)
+    auto score = [&](int e) {
+        if (by_logit) return correction ? z[e] + correction[e] : z[e];
+        return softmax ? expf(z[e] - z_max) * inv_sum : 1.0f / (1.0f + expf(-z[e]));
+    };
     const int group_size = n_groups > 1 ? n_experts / n_groups : n_experts;
     if (n_groups > 1) {
         // a group's score: the sum of its two largest choice scores (one, if it has one member)
         for (int g = lane; g < n_groups; g += 32) {
             float a = -INFINITY, b = -INFINITY;
             for (int e = g * group_size; e < (g + 1) * group_size; ++e) {
-                const float s = softmax ? expf(z[e] - z_max) * inv_sum : 1.0f / (1.0f + expf(-z[e]));
-                const float c = correction ? s + correction[e] : s;
+                const float s = score(e);
+                const float c = (correction && !by_logit) ? s + correction[e] : s;
                 if (c > a) { b = a; a = c; } else if (c > b) { b = c; }
             }
             group_score[warp][g] = group_size > 1 ? a + b : a;
@@ -88,8 +96,8 @@ __global__ void route_topk_kernel(const float* __restrict__ logits, int logit_st
                 taken = before >= keep_groups;
             }
             for (int p = 0; p < j; ++p) taken |= idx[(size_t)t * top + p] == e;
-            const float s = softmax ? expf(z[e] - z_max) * inv_sum : 1.0f / (1.0f + expf(-z[e]));
-            const float c = correction ? s + correction[e] : s;      // the choice's score
+            const float s = score(e);
+            const float c = (correction && !by_logit) ? s + correction[e] : s;      // the choice's score
             if (!taken && (c > best || (c == best && e < arg))) {
                 best = c;
                 best_s = s;
@@ -117,6 +125,17 @@ __global__ void route_topk_kernel(const float* __restrict__ logits, int logit_st
         }
         total += best_s;
         __syncwarp();
+    }
+    if (by_logit) {
+        // the first chosen logit is the largest
+        if (lane == 0) {
+            float* w = weight + (size_t)t * top;
+            const float most = w[0];
+            float sum = 0.f;
+            for (int j = 0; j < top; ++j) sum += expf(w[j] - most);
+            for (int j = 0; j < top; ++j) w[j] = expf(w[j] - most) / sum;
+        }
+        return;
     }
     if (renorm && lane == 0)
         for (int j = 0; j < top; ++j) weight[(size_t)t * top + j] /= total + renorm_eps;
@@ -221,17 +240,22 @@ __device__ __forceinline__ float gated_unit(float g, float u, float alpha, float
     return (g / (1.0f + expf(-g))) * u;
 }
 
-// GLU: A row = h[slot / top] (* weight[slot] if scale), W = [gate rows | up rows] of
+// What a product does: the experts' down projection, or an up projection with a unit on its sums.
+enum { DOWN = 0, GATED = 1, RELU2 = 2 };
+
+// GATED: A row = h[slot / top] (* weight[slot] if scale), W = [gate rows | up rows] of
 // expert e ([2F, K]), out y[p, n] = silu(gate) * up in T.
-// !GLU: A row = y[p], W = Wd[e] ([N, K]), out per_slot[slot, n] float32 (* weight[slot]
+// RELU2: the same A row, W = Wu[e] ([F, K]), y[p, n] = relu(up)^2.
+// DOWN: A row = y[p], W = Wd[e] ([N, K]), out per_slot[slot, n] float32 (* weight[slot]
 // if scale).  A thread owns rows ty*TM.. and the columns tx, tx + 16, tx + 32, tx + 48.
-template <typename T, bool GLU>
+template <typename T, int UNIT>
 __global__ void __launch_bounds__(256)
 expert_gemm_kernel(const T* __restrict__ A, const T* __restrict__ W, void* __restrict__ out,
                    const int* __restrict__ order, const int* __restrict__ offsets,
                    const int* __restrict__ tile_expert, const int* __restrict__ tile_row0,
                    const float* __restrict__ weight, int top, int scale, int N, int K,
                    float alpha, float limit) {
+    constexpr bool GLU = UNIT == GATED, UP = UNIT != DOWN;
     chain_release();
     chain_wait();
     const int e = tile_expert[blockIdx.y];
@@ -261,7 +285,7 @@ expert_gemm_kernel(const T* __restrict__ A, const T* __restrict__ W, void* __res
         fill_tile<T, BM, 1>(As, k0, K, vec_ok, [&](int r, float& sc) -> const T* {
             const int slot = slot_s[r];
             if (slot < 0) return nullptr;
-            if (GLU) {
+            if (UP) {
                 if (scale) sc = weight[slot];
                 return A + (size_t)(slot / top) * K;
             }
@@ -307,6 +331,9 @@ expert_gemm_kernel(const T* __restrict__ A, const T* __restrict__ W, void* __res
             if (GLU) {
                 Elem<T>::store((T*)out + (size_t)(p0 + r) * N + n,
                                gated_unit(acc[i][j], acu[i][j], alpha, limit));
+            } else if (UP) {
+                const float u = fmaxf(acc[i][j], 0.f);
+                Elem<T>::store((T*)out + (size_t)(p0 + r) * N + n, u * u);
             } else {
                 ((float*)out)[(size_t)slot * N + n] = scale ? acc[i][j] * weight[slot] : acc[i][j];
             }
@@ -336,7 +363,7 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], 
 // against one load of every weight tile; rows that are not there are zeros.
 // RT = 1 (few rows an expert: decoding) keeps one entry a CTA, so that as many CTAs as
 // possible stream weights.
-template <bool GLU, int RT>
+template <int UNIT, int RT>
 __global__ void __launch_bounds__(256)
 expert_mma_kernel(const __nv_bfloat16* __restrict__ A, const __nv_bfloat16* __restrict__ W,
                   void* __restrict__ out, const int* __restrict__ order,
@@ -344,6 +371,7 @@ expert_mma_kernel(const __nv_bfloat16* __restrict__ A, const __nv_bfloat16* __re
                   const int* __restrict__ tile_row0, int max_tiles,
                   const float* __restrict__ weight, int top, int scale, int N, int K,
                   float alpha, float limit) {
+    constexpr bool GLU = UNIT == GATED, UP = UNIT != DOWN;
     chain_release();
     chain_wait();
     constexpr int MROWS = RT * BM;
@@ -392,7 +420,7 @@ expert_mma_kernel(const __nv_bfloat16* __restrict__ A, const __nv_bfloat16* __re
             a_src[h2] = nullptr;
             a_scale[h2] = 1.f;
             if (slot >= 0) {
-                if (GLU) {
+                if (UP) {
                     a_src[h2] = A + (size_t)(slot / top) * K;
                     if (scale) a_scale[h2] = weight[slot];
                 } else {
@@ -409,7 +437,7 @@ expert_mma_kernel(const __nv_bfloat16* __restrict__ A, const __nv_bfloat16* __re
             for (int h2 = 0; h2 < LOADS; ++h2) {
                 if (lrow + 64 * h2 >= MROWS) continue;
                 uint4 v = (a_src[h2] && k_ok) ? *reinterpret_cast<const uint4*>(a_src[h2] + k0 + lk) : zero;
-                if (GLU && scale && a_src[h2]) {
+                if (UP && scale && a_src[h2]) {
                     __nv_bfloat162* p2 = reinterpret_cast<__nv_bfloat162*>(&v);
 #pragma unroll
                     for (int x = 0; x < 4; ++x) {
@@ -472,6 +500,9 @@ expert_mma_kernel(const __nv_bfloat16* __restrict__ A, const __nv_bfloat16* __re
                         if (GLU)
                             ((__nv_bfloat16*)out)[(size_t)(p0 + r) * N + n] = __float2bfloat16_rn(
                                 gated_unit(v, acu[mf][nf][2 * half + x], alpha, limit));
+                        else if (UP)
+                            ((__nv_bfloat16*)out)[(size_t)(p0 + r) * N + n] =
+                                __float2bfloat16_rn(fmaxf(v, 0.f) * fmaxf(v, 0.f));
                         else
                             ((float*)out)[(size_t)slot * N + n] = scale ? v * weight[slot] : v;
                     }
@@ -517,7 +548,7 @@ __global__ void expert_combine_kernel(const float* __restrict__ per_slot, int to
 MLS_API int mls_expert_tile_rows() { return BM; }
 
 MLS_API int mls_route_topk(const float* logits, int logit_stride, int n_tokens, int n_experts,
-                           int top, int renorm, int softmax, const float* correction,
+                           int top, int renorm, int mode, const float* correction,
                            float renorm_eps, int n_groups, int keep_groups, int* idx,
                            float* weight, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
@@ -526,7 +557,7 @@ MLS_API int mls_route_topk(const float* logits, int logit_stride, int n_tokens, 
                          keep_groups > n_groups || top > keep_groups * (n_experts / n_groups)))
         return MLS_ERR_UNSUPPORTED;
     MLS_LAUNCH((route_topk_kernel), dim3((n_tokens + 3) / 4), dim3(128), 0, stream, logits,
-               logit_stride, n_tokens, n_experts, top, renorm, softmax, correction, renorm_eps,
+               logit_stride, n_tokens, n_experts, top, renorm, mode, correction, renorm_eps,
                n_groups, keep_groups, idx, weight);
     return launch_status();
 }
@@ -541,55 +572,56 @@ MLS_API int mls_route_sort(const int* idx, int n_slots, int n_experts, int n_rea
     return launch_status();
 }
 
+// One of the experts' products over the sorted slots: N outputs of K inputs an expert.
+template <int UNIT>
+static int expert_product(const void* A, const void* W, void* out, int dtype, const int* order,
+                          const int* offsets, const int* tile_expert, const int* tile_row0,
+                          int max_tiles, const float* weight, int top, int scale, int N, int K,
+                          int many_rows, float alpha, float limit, cudaStream_t stream) {
+    if (max_tiles <= 0) return 0;
+    dim3 grid((N + BN - 1) / BN, max_tiles);
+    if (takes_mma(dtype, A, W, K) && many_rows)
+        MLS_LAUNCH((expert_mma_kernel<UNIT, 4>), dim3(grid.x, (max_tiles + 3) / 4), dim3(256), 0,
+                   stream, (const __nv_bfloat16*)A, (const __nv_bfloat16*)W, out, order, offsets,
+                   tile_expert, tile_row0, max_tiles, weight, top, scale, N, K, alpha, limit);
+    else if (takes_mma(dtype, A, W, K))
+        MLS_LAUNCH((expert_mma_kernel<UNIT, 1>), dim3(grid), dim3(256), 0, stream,
+                   (const __nv_bfloat16*)A, (const __nv_bfloat16*)W, out, order, offsets,
+                   tile_expert, tile_row0, max_tiles, weight, top, scale, N, K, alpha, limit);
+    else if (dtype == MLS_BF16)
+        MLS_LAUNCH((expert_gemm_kernel<__nv_bfloat16, UNIT>), dim3(grid), dim3(256), 0, stream,
+                   (const __nv_bfloat16*)A, (const __nv_bfloat16*)W, out, order, offsets,
+                   tile_expert, tile_row0, weight, top, scale, N, K, alpha, limit);
+    else
+        MLS_LAUNCH((expert_gemm_kernel<float, UNIT>), dim3(grid), dim3(256), 0, stream,
+                   (const float*)A, (const float*)W, out, order, offsets, tile_expert, tile_row0,
+                   weight, top, scale, N, K, alpha, limit);
+    return launch_status();
+}
+
 MLS_API int mls_expert_glu(const void* h, const void* w_gate_up, void* y, int dtype,
                            const int* order, const int* offsets, const int* tile_expert,
                            const int* tile_row0, int max_tiles, const float* weight, int top,
                            int scale_in, int F, int K, int many_rows, float alpha, float limit,
                            cudaStream_t stream) {
-    if (max_tiles <= 0) return 0;
-    dim3 grid((F + BN - 1) / BN, max_tiles);
-    if (takes_mma(dtype, h, w_gate_up, K) && many_rows)
-        MLS_LAUNCH((expert_mma_kernel<true, 4>), dim3(grid.x, (max_tiles + 3) / 4), dim3(256), 0,
-                   stream, (const __nv_bfloat16*)h, (const __nv_bfloat16*)w_gate_up, y, order, offsets,
-                   tile_expert, tile_row0, max_tiles, weight, top, scale_in, F, K, alpha, limit);
-    else if (takes_mma(dtype, h, w_gate_up, K))
-        MLS_LAUNCH((expert_mma_kernel<true, 1>), dim3(grid), dim3(256), 0, stream,
-                   (const __nv_bfloat16*)h, (const __nv_bfloat16*)w_gate_up, y, order, offsets,
-                   tile_expert, tile_row0, max_tiles, weight, top, scale_in, F, K, alpha, limit);
-    else if (dtype == MLS_BF16)
-        MLS_LAUNCH((expert_gemm_kernel<__nv_bfloat16, true>), dim3(grid), dim3(256), 0, stream,
-                   (const __nv_bfloat16*)h, (const __nv_bfloat16*)w_gate_up, y, order, offsets,
-                   tile_expert, tile_row0, weight, top, scale_in, F, K, alpha, limit);
-    else
-        MLS_LAUNCH((expert_gemm_kernel<float, true>), dim3(grid), dim3(256), 0, stream,
-                   (const float*)h, (const float*)w_gate_up, y, order, offsets, tile_expert,
-                   tile_row0, weight, top, scale_in, F, K, alpha, limit);
-    return launch_status();
+    return expert_product<GATED>(h, w_gate_up, y, dtype, order, offsets, tile_expert, tile_row0,
+                                 max_tiles, weight, top, scale_in, F, K, many_rows, alpha, limit, stream);
+}
+
+MLS_API int mls_expert_relu2(const void* h, const void* w_up, void* y, int dtype, const int* order,
+                             const int* offsets, const int* tile_expert, const int* tile_row0,
+                             int max_tiles, const float* weight, int top, int scale_in, int F, int K,
+                             int many_rows, cudaStream_t stream) {
+    return expert_product<RELU2>(h, w_up, y, dtype, order, offsets, tile_expert, tile_row0, max_tiles,
+                                 weight, top, scale_in, F, K, many_rows, 0.f, 0.f, stream);
 }
 
 MLS_API int mls_expert_down(const void* y, const void* w_down, float* per_slot, int dtype,
                             const int* order, const int* offsets, const int* tile_expert,
                             const int* tile_row0, int max_tiles, const float* weight, int top,
                             int scale_out, int D, int F, int many_rows, cudaStream_t stream) {
-    if (max_tiles <= 0) return 0;
-    dim3 grid((D + BN - 1) / BN, max_tiles);
-    if (takes_mma(dtype, y, w_down, F) && many_rows)
-        MLS_LAUNCH((expert_mma_kernel<false, 4>), dim3(grid.x, (max_tiles + 3) / 4), dim3(256), 0,
-                   stream, (const __nv_bfloat16*)y, (const __nv_bfloat16*)w_down, (void*)per_slot,
-                   order, offsets, tile_expert, tile_row0, max_tiles, weight, top, scale_out, D, F, 0.f, 0.f);
-    else if (takes_mma(dtype, y, w_down, F))
-        MLS_LAUNCH((expert_mma_kernel<false, 1>), dim3(grid), dim3(256), 0, stream,
-                   (const __nv_bfloat16*)y, (const __nv_bfloat16*)w_down, (void*)per_slot, order,
-                   offsets, tile_expert, tile_row0, max_tiles, weight, top, scale_out, D, F, 0.f, 0.f);
-    else if (dtype == MLS_BF16)
-        MLS_LAUNCH((expert_gemm_kernel<__nv_bfloat16, false>), dim3(grid), dim3(256), 0, stream,
-                   (const __nv_bfloat16*)y, (const __nv_bfloat16*)w_down, (void*)per_slot, order,
-                   offsets, tile_expert, tile_row0, weight, top, scale_out, D, F, 0.f, 0.f);
-    else
-        MLS_LAUNCH((expert_gemm_kernel<float, false>), dim3(grid), dim3(256), 0, stream,
-                   (const float*)y, (const float*)w_down, (void*)per_slot, order, offsets,
-                   tile_expert, tile_row0, weight, top, scale_out, D, F, 0.f, 0.f);
-    return launch_status();
+    return expert_product<DOWN>(y, w_down, per_slot, dtype, order, offsets, tile_expert, tile_row0,
+                                max_tiles, weight, top, scale_out, D, F, many_rows, 0.f, 0.f, stream);
 }
 
 MLS_API int mls_expert_combine(const float* per_slot, int top, const void* shared,

@@ -14,10 +14,30 @@
 // f for the values) are zeros, which changes no score and leaves zeros in the outputs' extra
 // entries.  The rest of a page that a request enters in this step is cleared.
 //
-// One block a token, one warp a head at a time; sums of squares in float32 in lane-stride
+// (mls_head_prep_store).  One block a token, one warp a head at a time; sums of squares in float32 in lane-stride
 // order and five shuffles, so a token's values depend on nothing else in the batch.
+//
+// mls_head_conv_rope_store: the same for attention with rotation, from contiguous columns
+// [q heads | k heads | v heads] of the float32 projection row.  A head of q and k may consist of
+// several maps (of e entries each, one after the other).  For every channel, then every map:
+//
+//   u <- u + b ;  y_t = sum_j w[j] u_(t - taps + 1 + j), zeros before the sequence's start  (optional)
+//   q, k <- y / sqrt(mean(y^2) + eps) * w_q (w_k)              per map, optional
+//   entry i < dims/2 of a map turns with entry i + dims/2 by position * freq[i]; cosine and sine
+//   are multiplied by `amplitude`                                                           optional
+//
+// A cached key row is a head's maps side by side, a query row holds one map in its place and
+// zeros elsewhere: with maps M > 1 head h's map m is a query head of its own (row h * M + m),
+// and its score against the cached row is that of its own map's key.  The convolution's last
+// taps - 1 inputs of every request are a tail [taps - 1, channels] (float32, oldest first) in its
+// state slot; mls_tail_update moves it on behind this kernel or, in a step of one token a request,
+// this kernel does itself.  A warp a map (or value head) and run of tokens.
+//
+// mls_head_difference: what becomes of two maps' outputs a head, a warp a (token, head):
+//   o = a1 - lambda a2 ;  o <- o / sqrt(mean(o^2) + eps) * mul ;  o <- o * sigmoid(gate)
 #include "common.cuh"
 #include "page_tail.cuh"
+#include "row_pack.cuh"
 
 namespace {
 constexpr int HP_THREADS = 128;      // a block of a prompt's token
@@ -100,6 +120,257 @@ head_prep_kernel(const float* __restrict__ proj, int proj_width, int q_col, int 
         clear_page_tail<T>(rest, slot, block_size, n_pages, n_kv, hd, k_pool, v_pool);
     }
 }
+
+constexpr int HC_WARPS = 8, HC_RUN = 8, HC_TAPS = 8;
+
+struct HeadConvArgs {
+    const float* proj;                 // [T, proj_width], q | k | v from column col on
+    int proj_width, col;
+    const float* bias;                 // [channels] or nullptr
+    const float* conv;                 // [taps][channels], taps > 0
+    int taps, move_tail;
+    float* tail;                       // [slots][taps - 1][channels], tail_stride apart
+    long long tail_stride;
+    const float *w_q, *w_k;            // [e] or nullptr
+    float eps;
+    const double* freq;                // [rot / 2]
+    int rot;
+    float amplitude;
+    const int *state_slot, *cu_q, *req_of_token, *positions, *slot_map;
+    int q_width, block_size, n_pages, n_tokens, n_heads, n_kv, maps, e, f, hd, writes, run;
+    int* status;
+};
+
+template <int V>
+__device__ __forceinline__ Pack<V> load_floats(const float* p) {
+    Pack<V> r;
+    if constexpr (V == 4) {
+        const float4 x = *reinterpret_cast<const float4*>(p);
+        r.v[0] = x.x; r.v[1] = x.y; r.v[2] = x.z; r.v[3] = x.w;
+    } else if constexpr (V == 2) {
+        const float2 x = *reinterpret_cast<const float2*>(p);
+        r.v[0] = x.x; r.v[1] = x.y;
+    } else {
+        r.v[0] = *p;
+    }
+    return r;
+}
+template <int V>
+__device__ __forceinline__ void store_floats(float* p, const Pack<V>& r) {
+    if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(r.v[0], r.v[1], r.v[2], r.v[3]);
+    else if constexpr (V == 2) *reinterpret_cast<float2*>(p) = make_float2(r.v[0], r.v[1]);
+    else *p = r.v[0];
+}
+template <int V>
+__device__ __forceinline__ void store_elems(float* p, const Pack<V>& r) { store_floats<V>(p, r); }
+template <int V>
+__device__ __forceinline__ void store_elems(__nv_bfloat16* p, const Pack<V>& r) {
+    if constexpr (V == 4)
+        *reinterpret_cast<uint2*>(p) = pack_bf16x4(make_float4(r.v[0], r.v[1], r.v[2], r.v[3]));
+    else if constexpr (V == 2)
+        *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(r.v[0], r.v[1]);
+    else
+        *p = __float2bfloat16_rn(r.v[0]);
+}
+
+// V: neighbouring entries a lane takes at a time (the model's sizes decide).
+template <typename T, int V>
+__global__ void __launch_bounds__(HC_WARPS * 32)
+head_conv_rope_kernel(const HeadConvArgs a, T* __restrict__ q_out, T* __restrict__ k_pool,
+                      T* __restrict__ v_pool) {
+    chain_release();
+    extern __shared__ __align__(16) float hc_smem[];
+    __shared__ int slot_s[HC_RUN], rest_s[HC_RUN], at_s[HC_RUN], state_s[HC_RUN];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int t0 = blockIdx.x * a.run, n_run = min(a.run, a.n_tokens - t0);
+    const int half = a.rot / 2, widest = max(a.e, a.f);
+    float* angles = hc_smem;                                     // [run][cos | sin]
+    float* stage = hc_smem + (((size_t)a.run * a.rot + 3) & ~(size_t)3) +
+                   (size_t)warp * ((widest + 3) & ~3);           // this warp's head
+    // the step's index arrays are its input: no kernel of the step writes them
+    if (threadIdx.x < n_run) {
+        const int t = t0 + threadIdx.x, r = a.req_of_token[t];
+        int slot = -1, rest = 0;
+        if (a.writes) {
+            slot = a.slot_map[t];
+            if (slot < 0 || slot >= a.n_pages * a.block_size) {
+                if (blockIdx.y == 0 && a.status) atomicOr(a.status, MLS_STATUS_BAD_SLOT);
+                slot = -1;
+            } else {
+                rest = page_tail_to_clear(a.slot_map, t, a.n_tokens, slot, a.block_size);
+            }
+        }
+        slot_s[threadIdx.x] = slot;
+        rest_s[threadIdx.x] = rest;
+        at_s[threadIdx.x] = t - a.cu_q[r];
+        state_s[threadIdx.x] = a.taps > 1 ? a.state_slot[r] : 0;
+    }
+    for (int u = threadIdx.x; u < n_run * half; u += blockDim.x) {
+        const int tok = u / half, i = u - tok * half;
+        float c, s;
+        angle_cos_sin(a.positions[t0 + tok], a.freq[i], c, s);
+        angles[tok * a.rot + i] = c * a.amplitude;
+        angles[tok * a.rot + half + i] = s * a.amplitude;
+    }
+    __syncthreads();
+    chain_wait();
+    const int nq = a.n_heads * a.maps, nk = a.n_kv * a.maps;
+    const int units = nq + (a.writes ? nk + a.n_kv : 0);
+    const int channels = (nq + nk) * a.e + a.n_kv * a.f, n_tail = a.taps - 1;
+    const int u = blockIdx.y * HC_WARPS + warp;
+    if (u < units) {
+        const int kind = u < nq ? 0 : (u < nq + nk ? 1 : 2);
+        const int unit = kind == 0 ? u : (kind == 1 ? u - nq : u - nq - nk);
+        const int width = kind == 2 ? a.f : a.e;
+        const int ch0 = kind == 2 ? (nq + nk) * a.e + unit * a.f : u * a.e;    // first channel
+        const float* w = kind == 0 ? a.w_q : kind == 1 ? a.w_k : nullptr;
+        const int head = kind == 2 ? unit : unit / a.maps, map = kind == 2 ? 0 : unit % a.maps;
+        const int inside = map * a.e;                            // where the map lies in its row
+        const int rot = kind == 2 ? 0 : a.rot;
+        // the entries of the row this warp writes: a query row is its own; a key row's maps share
+        // one, the last of them fills it up
+        const int c_lo = kind == 1 ? inside : 0;
+        const int c_hi = (kind == 1 && map + 1 < a.maps) ? inside + a.e : a.hd;
+        for (int tok = 0; tok < n_run; ++tok) {
+            const int t = t0 + tok, i_t = at_s[tok];
+            float* tail = n_tail > 0 ? a.tail + (size_t)state_s[tok] * a.tail_stride : nullptr;
+            float ss = 0.f;
+            for (int c = lane * V; c < width; c += 32 * V) {
+                const int ch = ch0 + c;
+                const float* src = a.proj + (size_t)t * a.proj_width + a.col + ch;
+                Pack<V> bias;
+#pragma unroll
+                for (int x = 0; x < V; ++x) bias.v[x] = 0.f;
+                if (a.bias) bias = load_floats<V>(a.bias + ch);
+                Pack<V> y;
+                if (a.taps <= 0) {
+                    y = load_floats<V>(src);
+#pragma unroll
+                    for (int x = 0; x < V; ++x) y.v[x] += bias.v[x];
+                } else {
+#pragma unroll
+                    for (int x = 0; x < V; ++x) y.v[x] = 0.f;
+                    for (int j0 = 0; j0 < a.taps; j0 += HC_TAPS) {
+                        Pack<V> in[HC_TAPS];
+#pragma unroll
+                        for (int j = 0; j < HC_TAPS; ++j) {
+                            const int back = n_tail - (j0 + j);      // tokens before this one
+                            if (j0 + j < a.taps)
+                                in[j] = back <= i_t
+                                    ? load_floats<V>(src - (size_t)back * a.proj_width)
+                                    : load_floats<V>(tail + (size_t)(n_tail + i_t - back) * channels + ch);
+                        }
+#pragma unroll
+                        for (int j = 0; j < HC_TAPS; ++j) {
+                            if (j0 + j < a.taps) {
+                                if (n_tail - (j0 + j) <= i_t) {
+#pragma unroll
+                                    for (int x = 0; x < V; ++x) in[j].v[x] += bias.v[x];
+                                }
+                                const Pack<V> cw = load_floats<V>(a.conv + (size_t)(j0 + j) * channels + ch);
+#pragma unroll
+                                for (int x = 0; x < V; ++x) y.v[x] = fmaf(cw.v[x], in[j].v[x], y.v[x]);
+                                // (row j - 1 was read by this lane one tap ago)
+                                if (a.move_tail && j0 + j >= 1)
+                                    store_floats<V>(tail + (size_t)(j0 + j - 1) * channels + ch, in[j]);
+                            }
+                        }
+                    }
+                }
+                if (w) {
+                    const Pack<V> wv = load_floats<V>(w + c);
+#pragma unroll
+                    for (int x = 0; x < V; ++x) {
+                        ss = fmaf(y.v[x], y.v[x], ss);
+                        y.v[x] *= wv.v[x];
+                    }
+                }
+                store_floats<V>(stage + c, y);
+            }
+            const float inv = w ? 1.0f / sqrtf(warp_sum(ss) / (float)width + a.eps) : 1.f;
+            __syncwarp();
+            T* dst;
+            if (kind == 0) {
+                dst = q_out + (size_t)t * a.q_width + (size_t)unit * a.hd;
+            } else {
+                const int slot = slot_s[tok];
+                if (slot < 0) continue;                          // (the same for the whole warp)
+                const int page = slot / a.block_size, off = slot - page * a.block_size;
+                dst = (kind == 1 ? k_pool : v_pool) +
+                      (((size_t)head * a.n_pages + page) * a.block_size + off) * a.hd;
+            }
+            const float* cs = angles + tok * a.rot;
+            for (int c = c_lo + lane * V; c < c_hi; c += 32 * V) {
+                const int rel = c - inside;
+                Pack<V> y;
+#pragma unroll
+                for (int x = 0; x < V; ++x) {
+                    const int i = rel + x;
+                    float val = 0.f;
+                    if (i >= 0 && i < width) {
+                        val = stage[i] * inv;
+                        if (i < half && rot > 0) {
+                            const float mate = stage[i + half] * inv;
+                            val = __fsub_rn(__fmul_rn(val, cs[i]), __fmul_rn(mate, cs[half + i]));
+                        } else if (i < rot) {
+                            const float mate = stage[i - half] * inv;
+                            val = __fadd_rn(__fmul_rn(val, cs[i - half]), __fmul_rn(mate, cs[i]));
+                        }
+                    }
+                    y.v[x] = val;
+                }
+                store_elems<V>(dst + c, y);
+            }
+            __syncwarp();                                        // the stage is filled again
+        }
+    }
+    if (a.writes && blockIdx.y == 0)
+        for (int tok = 0; tok < n_run; ++tok)
+            if (slot_s[tok] >= 0)
+                clear_page_tail<T>(rest_s[tok], slot_s[tok], a.block_size, a.n_pages, a.n_kv, a.hd,
+                                   k_pool, v_pool);
+}
+
+// o [T, 2 H * hd]: head h's two maps at rows 2h and 2h + 1; out [T, H * f].
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+head_difference_kernel(const T* __restrict__ o, int hd, float lambda, float mul, float eps,
+                       const float* __restrict__ gate, int gate_row, int gate_col,
+                       T* __restrict__ out, int n_tokens, int n_heads, int f) {
+    chain_release();
+    chain_wait();
+    const int lane = threadIdx.x & 31;
+    const long long unit = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+    if (unit >= (long long)n_tokens * n_heads) return;
+    const int t = (int)(unit / n_heads), h = (int)(unit - (long long)t * n_heads);
+    constexpr int DT = sizeof(T) == 2 ? MLS_BF16 : MLS_F32;
+    const size_t first = ((size_t)t * n_heads + h) * 2 * hd;
+    auto difference = [&](int c) {
+        const Pack<V> a1 = load_pack<V>(o, first + c, DT), a2 = load_pack<V>(o, first + hd + c, DT);
+        Pack<V> r;
+#pragma unroll
+        for (int x = 0; x < V; ++x) r.v[x] = fmaf(-lambda, a2.v[x], a1.v[x]);
+        return r;
+    };
+    float ss = 0.f;
+    for (int c = lane * V; c < f; c += 32 * V) {
+        const Pack<V> d = difference(c);
+#pragma unroll
+        for (int x = 0; x < V; ++x) ss = fmaf(d.v[x], d.v[x], ss);
+    }
+    const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)f + eps);
+    for (int c = lane * V; c < f; c += 32 * V) {
+        Pack<V> d = difference(c);
+        Pack<V> z;
+        if (gate) z = load_pack<V>(gate, (size_t)t * gate_row + gate_col + (size_t)h * f + c, MLS_F32);
+#pragma unroll
+        for (int x = 0; x < V; ++x) {
+            d.v[x] = d.v[x] * inv * mul;
+            if (gate) d.v[x] = d.v[x] / (1.0f + expf(-z.v[x]));
+        }
+        store_pack<V>(out, ((size_t)t * n_heads + h) * f + c, DT, d);
+    }
+}
 }  // namespace
 
 MLS_API int mls_head_prep_store(const float* proj, int proj_width, int q_col, int k_col, int v_col,
@@ -130,5 +401,86 @@ MLS_API int mls_head_prep_store(const float* proj, int proj_width, int q_col, in
                    temp_every, v_scale, v_first, v_mode, v_lambda, positions, slot_map, (float*)q_out, q_width,
                    (float*)k_pool, (float*)v_pool, block_size, n_pages, n_tokens, n_heads, n_kv,
                    e, f, hd, writes, status);
+    return launch_status();
+}
+
+MLS_API int mls_head_conv_rope_store(
+        const float* proj, int proj_width, int col, const float* bias, const float* conv, int taps,
+        int move_tail, float* tail, long long tail_stride, const float* w_q, const float* w_k,
+        float eps, const double* freq, int rot, float amplitude, const int* state_slot,
+        const int* cu_q, const int* req_of_token, const int* positions, const int* slot_map,
+        void* q_out, int q_width, int dtype, void* k_pool, void* v_pool, int block_size, int n_pages,
+        int n_tokens, int n_heads, int n_kv, int maps, int e, int f, int hd, int writes, int* status,
+        cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (e <= 0 || f <= 0 || maps < 1 || hd < maps * e || hd < f || n_heads <= 0 || n_kv <= 0 ||
+        taps < 0 || (taps > 0 && !conv) || (taps > 1 && !tail) || rot < 0 || (rot & 1) || rot > e ||
+        (rot > 0 && !freq) || (w_q == nullptr) != (w_k == nullptr) || (move_tail && taps <= 1))
+        return MLS_ERR_UNSUPPORTED;
+    HeadConvArgs a;
+    a.proj = proj; a.proj_width = proj_width; a.col = col; a.bias = bias; a.conv = conv; a.taps = taps;
+    a.move_tail = move_tail; a.tail = tail; a.tail_stride = tail_stride; a.w_q = w_q; a.w_k = w_k;
+    a.eps = eps; a.freq = freq; a.rot = rot; a.amplitude = amplitude; a.state_slot = state_slot;
+    a.cu_q = cu_q; a.req_of_token = req_of_token; a.positions = positions; a.slot_map = slot_map;
+    a.q_width = q_width; a.block_size = block_size; a.n_pages = n_pages; a.n_tokens = n_tokens;
+    a.n_heads = n_heads; a.n_kv = n_kv; a.maps = maps; a.e = e; a.f = f; a.hd = hd; a.writes = writes;
+    a.status = status;
+    const int units = n_heads * maps + (writes ? n_kv * maps + n_kv : 0);
+    const int grid_y = (units + HC_WARPS - 1) / HC_WARPS;
+    // runs of tokens as long as every SM still has several blocks
+    a.run = HC_RUN;
+    while (a.run > 1 && (long long)((n_tokens + a.run - 1) / a.run) * grid_y < 4LL * sm_count())
+        a.run >>= 1;
+    // entries a lane takes at a time: all lanes busy, and every row at an aligned place
+    const int widest = e > f ? e : f;
+    auto takes = [&](int v) {
+        uintptr_t bits = 0;
+        for (const void* p : {(const void*)proj, (const void*)bias, (const void*)conv,
+                              (const void*)tail, (const void*)w_q, (const void*)w_k})
+            bits |= reinterpret_cast<uintptr_t>(p);
+        return e % v == 0 && f % v == 0 && proj_width % v == 0 && col % v == 0 && q_width % v == 0 &&
+               bits % (4 * v) == 0 && (taps <= 1 || tail_stride % v == 0);
+    };
+    const int v = (widest > 64 && takes(4)) ? 4 : (widest > 32 && takes(2)) ? 2 : 1;
+    const size_t smem = ((((size_t)a.run * rot + 3) & ~(size_t)3) +
+                         (size_t)HC_WARPS * ((widest + 3) & ~3)) * sizeof(float);
+    if (smem > 48 * 1024) return MLS_ERR_UNSUPPORTED;
+    const dim3 grid((n_tokens + a.run - 1) / a.run, grid_y);
+#define HC_GO(T, V)                                                                              \
+    MLS_LAUNCH((head_conv_rope_kernel<T, V>), grid, dim3(HC_WARPS * 32), smem, stream, a,         \
+               (T*)q_out, (T*)k_pool, (T*)v_pool)
+    if (dtype == MLS_BF16) {
+        if (v == 4) HC_GO(__nv_bfloat16, 4);
+        else if (v == 2) HC_GO(__nv_bfloat16, 2);
+        else HC_GO(__nv_bfloat16, 1);
+    } else {
+        if (v == 4) HC_GO(float, 4);
+        else if (v == 2) HC_GO(float, 2);
+        else HC_GO(float, 1);
+    }
+#undef HC_GO
+    return launch_status();
+}
+
+MLS_API int mls_head_difference(const void* o, int dtype, int hd, float lambda, float mul, float eps,
+                                const float* gate, int gate_row, int gate_col, void* out,
+                                int n_tokens, int n_heads, int f, cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (f <= 0 || hd < f || n_heads <= 0) return MLS_ERR_UNSUPPORTED;
+    const int blocks = (int)(((long long)n_tokens * n_heads + 7) / 8);
+    const bool by4 = f % 4 == 0 && hd % 4 == 0 && gate_row % 4 == 0 && gate_col % 4 == 0 &&
+                     (reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(out) |
+                      reinterpret_cast<uintptr_t>(gate)) % 16 == 0;
+#define HD_GO(T, V)                                                                               \
+    MLS_LAUNCH((head_difference_kernel<T, V>), dim3(blocks), dim3(256), 0, stream, (const T*)o, hd, \
+               lambda, mul, eps, gate, gate_row, gate_col, (T*)out, n_tokens, n_heads, f)
+    if (dtype == MLS_BF16) {
+        if (by4) HD_GO(__nv_bfloat16, 4);
+        else HD_GO(__nv_bfloat16, 1);
+    } else {
+        if (by4) HD_GO(float, 4);
+        else HD_GO(float, 1);
+    }
+#undef HD_GO
     return launch_status();
 }

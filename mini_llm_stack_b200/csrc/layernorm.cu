@@ -1,4 +1,4 @@
-// Layer norm with a weight and no bias, fused with the pending residual additions.
+// Layer norm with a weight and no bias (before a sublayer), fused with the pending residual additions.
 //
 //   v = x[row] + delta[row] + more_rows[row] + more_vec        (each addend optional)
 //   h = (v - mean(v)) / sqrt(mean((v - mean(v))^2) + eps) * w
@@ -17,8 +17,19 @@
 // d alone (one block of LN_THREADS threads a row), so a row's result does not depend
 // on the batch it is in.
 //
+// mls_add_post_layernorm is the other arrangement, a norm behind a sublayer:
+//
+//   y = the sublayer's result at row t (a tensor, or the sum of K-parts) + y_bias      (optional)
+//   y = (y - mean(y)) / sqrt(mean((y - mean(y))^2) + eps) * w1 + b1
+//   v = x[t] + y                                    (x may be absent: v = y)
+//   h = v, or a second such norm of v with w2, b2   (h may be absent)
+//
+// without `rows` for every row t, x[t] = v; with rows only those are read and x stays.  The row
+// stays in registers; which thread holds which entries depends on the row's width alone.
+//
 // mls_residual_add only settles more_rows / more_vec into x, for a norm of another kind.
 #include "common.cuh"
+#include "row_pack.cuh"
 
 namespace {
 constexpr int LN_THREADS = 256;
@@ -103,7 +114,185 @@ __global__ void settle_concat_kernel(float* __restrict__ x, const void* __restri
         store_from_float(out, t * 2 * d + d + c, out_dtype, other[i]);
     }
 }
+
+struct PostNormArgs {
+    float* x;
+    const void* y;                     // [parts][T, d] or nullptr: no sublayer's result
+    int y_dtype, y_parts;
+    long long y_stride;
+    const float *y_bias, *w1, *b1, *w2, *b2;      // [d]; y_bias and (w2, b2) may be absent
+    float eps;
+    void* h;
+    int h_dtype;
+    float* y_out;
+    const int* rows;
+    int d;
+};
+
+// Sum over the block with one barrier; `scratch` belongs to this sum alone.  Every thread adds
+// the warps' sums in their order.
+__device__ __forceinline__ float row_sum(float v, float* scratch /* >= 32 floats */) {
+    v = warp_sum(v);
+    if ((threadIdx.x & 31) == 0) scratch[threadIdx.x >> 5] = v;
+    __syncthreads();
+    float s = 0.f;
+    const int n = (int)(blockDim.x >> 5);
+    for (int i = 0; i < n; ++i) s += scratch[i];
+    return s;
+}
+
+// Layer norm of a row held as packs; the vectors are held already (HELD) or read where needed.
+template <int N, int VEC, bool HELD>
+__device__ __forceinline__ void norm_packs(Pack<N> (&v)[VEC], const Pack<N> (&w)[HELD ? VEC : 1],
+                                           const Pack<N> (&b)[HELD ? VEC : 1],
+                                           const float* __restrict__ pw,
+                                           const float* __restrict__ pb, int d, float eps,
+                                           float* scratch /* >= 64 floats */) {
+    float s = 0.f, q = 0.f;
+#pragma unroll
+    for (int k = 0; k < VEC; ++k)
+        if (((int)threadIdx.x + k * (int)blockDim.x) * N < d)
+#pragma unroll
+            for (int e = 0; e < N; ++e) s += v[k].v[e];
+    const float mean = row_sum(s, scratch) / (float)d;
+#pragma unroll
+    for (int k = 0; k < VEC; ++k)
+        if (((int)threadIdx.x + k * (int)blockDim.x) * N < d)
+#pragma unroll
+            for (int e = 0; e < N; ++e) {
+                v[k].v[e] -= mean;
+                q = fmaf(v[k].v[e], v[k].v[e], q);
+            }
+    const float inv = 1.0f / sqrtf(row_sum(q, scratch + 32) / (float)d + eps);
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) {
+        const int c = ((int)threadIdx.x + k * (int)blockDim.x) * N;
+        if (c < d) {
+            const Pack<N> wk = HELD ? w[HELD ? k : 0] : load_pack<N>(pw, c, MLS_F32);
+            const Pack<N> bk = HELD ? b[HELD ? k : 0] : load_pack<N>(pb, c, MLS_F32);
+#pragma unroll
+            for (int e = 0; e < N; ++e) v[k].v[e] = fmaf(v[k].v[e] * inv, wk.v[e], bk.v[e]);
+        }
+    }
+}
+
+// N: entries a thread takes at a time (4 where every row starts at a 16-byte place), VEC: such
+// groups a thread holds, threads * N * VEC >= d.  FEW: few rows; K-parts are possible and the
+// norm's vectors are read ahead of the wait on the kernel before.
+template <int N, int VEC, int MAX_THREADS, bool FEW>
+__global__ void __launch_bounds__(MAX_THREADS, (FEW || MAX_THREADS > 256) ? 1 : VEC <= 2 ? 4 : VEC <= 4 ? 3 : 1)
+add_post_layernorm_kernel(const PostNormArgs a) {
+    chain_release();
+    __shared__ float scratch[4][32];
+    const int i = blockIdx.x, d = a.d;
+    const int t = a.rows ? a.rows[i] : i;
+    const size_t at = (size_t)t * d;
+    constexpr bool HELD = FEW && MAX_THREADS <= 256;
+    Pack<N> y[VEC], x[VEC], w[HELD ? VEC : 1], b[HELD ? VEC : 1], none[1];
+    if constexpr (HELD) {
+        if (a.y) {
+#pragma unroll
+            for (int k = 0; k < VEC; ++k) {
+                const int c = ((int)threadIdx.x + k * (int)blockDim.x) * N;
+                if (c < d) {
+                    w[k] = load_pack<N>(a.w1, c, MLS_F32);
+                    b[k] = load_pack<N>(a.b1, c, MLS_F32);
+                }
+            }
+        }
+    }
+    chain_wait();
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) {
+        const int c = ((int)threadIdx.x + k * (int)blockDim.x) * N;
+        if (c < d) {
+            if (a.y) {
+                y[k] = load_parts<N>(a.y, at + c, a.y_dtype, FEW ? a.y_parts : 1, (size_t)a.y_stride);
+                if (a.y_bias) {
+                    const Pack<N> bias = load_pack<N>(a.y_bias, c, MLS_F32);
+#pragma unroll
+                    for (int e = 0; e < N; ++e) y[k].v[e] += bias.v[e];
+                }
+            }
+            if (a.x) x[k] = load_pack<N>(a.x, at + c, MLS_F32);
+        }
+    }
+    if (a.y) norm_packs<N, VEC, HELD>(y, w, b, a.w1, a.b1, d, a.eps, scratch[0]);
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) {
+        const int c = ((int)threadIdx.x + k * (int)blockDim.x) * N;
+        if (c < d) {
+            if (a.y_out) store_pack<N>(a.y_out, (size_t)i * d + c, MLS_F32, y[k]);
+            if (!a.x) {
+                x[k] = y[k];
+            } else if (a.y) {
+#pragma unroll
+                for (int e = 0; e < N; ++e) x[k].v[e] += y[k].v[e];
+                if (!a.rows) store_pack<N>(a.x, at + c, MLS_F32, x[k]);
+            }
+        }
+    }
+    if (!a.h) return;
+    if (a.w2) norm_packs<N, VEC, false>(x, none, none, a.w2, a.b2, d, a.eps, scratch[2]);
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) {
+        const int c = ((int)threadIdx.x + k * (int)blockDim.x) * N;
+        if (c < d) store_pack<N>(a.h, (size_t)i * d + c, a.h_dtype, x[k]);
+    }
+}
 }  // namespace
+
+MLS_API int mls_add_post_layernorm(float* x, const void* y, int y_dtype, int y_parts,
+                                   long long y_stride, const float* y_bias, const float* w1,
+                                   const float* b1, const float* w2, const float* b2, float eps,
+                                   void* h, int h_dtype, float* y_out, const int* rows, int n_out,
+                                   int d, cudaStream_t stream) {
+    if (n_out <= 0 || d <= 0) return 0;
+    if ((y && (!w1 || !b1)) || (!x && !y) || (w2 && !b2) || y_parts < 1 || (y_out && !y) ||
+        (y_parts > 1 && y_dtype != MLS_F32))
+        return MLS_ERR_UNSUPPORTED;
+    PostNormArgs a;
+    a.x = x; a.y = y; a.y_dtype = y_dtype; a.y_parts = y_parts; a.y_stride = y_stride;
+    a.y_bias = y_bias; a.w1 = w1; a.b1 = b1; a.w2 = w2; a.b2 = b2; a.eps = eps; a.h = h;
+    a.h_dtype = h_dtype; a.y_out = y_out; a.rows = rows; a.d = d;
+    // four entries a thread where every row and vector starts at a 16-byte place (buffers do:
+    // this depends on the model's sizes)
+    uintptr_t bits = 0;
+    for (const void* p : {(const void*)x, y, (const void*)y_bias, (const void*)w1, (const void*)b1,
+                          (const void*)w2, (const void*)b2, (const void*)h, (const void*)y_out})
+        bits |= reinterpret_cast<uintptr_t>(p);
+    const bool by4 = d % 4 == 0 && bits % 16 == 0 && (y_parts == 1 || y_stride % 4 == 0);
+    const int groups = by4 ? d / 4 : d;
+    // few groups: a group a thread, up to 256 threads; then up to four groups a thread; then
+    // more threads
+    int threads = 32;
+    while (threads < 256 && threads < groups) threads <<= 1;
+    while (threads < 1024 && threads * 4 < groups) threads <<= 1;
+    const int vec = (groups + threads - 1) / threads;
+    const bool few = y_parts > 1 || n_out <= 2 * sm_count();
+#define PN_RUN(N, V, M, F) \
+    MLS_LAUNCH((add_post_layernorm_kernel<N, V, M, F>), dim3(n_out), dim3(threads), 0, stream, a)
+#define PN_GO(N, V)                                  \
+    do {                                             \
+        if (threads > 256) PN_RUN(N, V, 1024, true); \
+        else if (few) PN_RUN(N, V, 256, true);       \
+        else PN_RUN(N, V, 256, false);               \
+    } while (0)
+    if (by4) {
+        if (vec <= 1) PN_GO(4, 1);
+        else if (vec <= 2) PN_GO(4, 2);
+        else if (vec <= 4) PN_GO(4, 4);
+        else return MLS_ERR_UNSUPPORTED;
+    } else {
+        if (vec <= 1) PN_GO(1, 1);
+        else if (vec <= 4) PN_GO(1, 4);
+        else if (vec <= 16) PN_GO(1, 16);
+        else return MLS_ERR_UNSUPPORTED;
+    }
+#undef PN_GO
+#undef PN_RUN
+    return launch_status();
+}
 
 MLS_API int mls_settle_concat(float* x, const void* delta, int delta_dtype, int delta_parts,
                               long long part_stride, const float* other, void* out,

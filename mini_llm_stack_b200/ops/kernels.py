@@ -134,7 +134,7 @@ class Ops:
                                   _LL, _I, _P, _I, _LL, _P, _P])
         self._attention_simt = _decl(core, "mls_attention_simt",
                                      [_P, _P, _I, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I,
-                                      _I, _F, _I, _F, _LL, _P, _P, _I, _LL, _P])
+                                      _I, _F, _I, _F, _LL, _P, _P, _I, _LL, _I, _P])
         self._swiglu = _decl(core, "mls_swiglu", [_P, _P, _I, _I, _I, _P])
         self._clamped_glu = _decl(core, "mls_clamped_glu", [_P, _P, _I, _I, _I, _F, _F, _P])
         self._unary_act = _decl(core, "mls_unary_act", [_P, _I, _P, _I, _LL, _I, _P, _I, _I, _P])
@@ -529,10 +529,10 @@ class Ops:
             lib = self._load("attention", {"MLS_HEAD_DIM": int(hd)})
             fn = _decl(lib, "mls_attention_mma",
                        [_P, _P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _F, _I, _I, _I,
-                        _P, _P, _LL, _P, _I, _P, _P, _I, _LL, _P])
+                        _P, _P, _LL, _P, _I, _P, _P, _I, _LL, _I, _P])
             tc = _decl(lib, "mls_attention_tc",
                        [_P, _P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _F, _I, _F, _I, _I, _I, _LL,
-                        _P, _P, _LL, _P, _I, _P])
+                        _P, _P, _LL, _P, _I, _I, _P])
             fused = _decl(lib, "mls_attention_decode_fused",
                           [_P, _I, _LL, _P, _P, _P, _I, _P, _I, _P, _P, _P, _P, _I, _P, _P, _I, _I,
                            _I, _I, _F, _I, _I, _P, _P, _LL, _P, _P])
@@ -584,8 +584,11 @@ class Ops:
 
     def paged_attention(self, qkv, out, cache, step, n_heads: int, n_kv: int, hd: int,
                         scale: float, window: int, plan=None, softcap: float = 0.0,
-                        sink=None, slopes=None, keep_first: int = 0, simt: bool = False) -> None:
-        """Attention of the step's tokens over the pages.  ``slopes`` (float32 [n_heads]): the
+                        sink=None, slopes=None, keep_first: int = 0, simt: bool = False,
+                        chunk: int = 0) -> None:
+        """Attention of the step's tokens over the pages.  ``window`` w > 0: a query sees the last
+        w tokens; ``chunk`` c > 0 (without a window): its own chunk of c tokens, counted from the
+        sequence's start, up to itself.  ``slopes`` (float32 [n_heads]): the
         score of head h loses ``slopes[h] * (position - key's position)``.  ``keep_first``: a
         window does not hide the sequence's first so many keys.  ``out`` may be a block of
         columns of a wider buffer.  Of the tensor-core kernels the tcgen05 kernel (prompts) and
@@ -602,6 +605,7 @@ class Ops:
         _need(cache.k_pool.dtype == qkv.dtype, "attention: cache and activations differ")
         _need(slopes is None or (slopes.dtype == torch.float32 and slopes.shape == (n_heads,)
                                  and slopes.is_contiguous()), "attention: slopes are float32 [heads]")
+        _need(not (window and chunk), "attention: a window or chunks, not both")
         keep_first = int(keep_first or 0) if window else 0
         plain = slopes is None and keep_first == 0 and out.stride(0) % 8 == 0
         _need(plain or not (softcap and slopes is not None),
@@ -626,7 +630,7 @@ class Ops:
                           step.n_requests, n_heads, n_kv, g.block_size, float(scale), int(window),
                           float(softcap), n_tiles_tc, plan.n_tiles_tc_wide, n_small, cache.k_pool.shape[1],
                           _ptr(self.status), _ptr(sink), out.stride(0), _ptr(slopes), keep_first,
-                          self._stream()), "attention_tc")
+                          int(chunk), self._stream()), "attention_tc")
                 n_tiles = 0
                 if not n_small:
                     return
@@ -646,7 +650,7 @@ class Ops:
                       float(softcap), n_tiles, n_small, n_split, _ptr(part_o), _ptr(part_lse),
                       cache.k_pool.shape[1], _ptr(self.status),
                       0 if (self.attention_impl == "no_tma" or not plain) else 1, _ptr(sink),
-                      _ptr(slopes), keep_first, out.stride(0), self._stream()),
+                      _ptr(slopes), keep_first, out.stride(0), int(chunk), self._stream()),
                    "attention_mma")
             return
         self.launches += 1
@@ -654,7 +658,7 @@ class Ops:
             _ptr(qkv), _ptr(out), _code(qkv.dtype), _ptr(cache.k_pool), _ptr(cache.v_pool),
             _ptr(g.block_table), g.max_blocks, _ptr(step.positions), _ptr(step.req_of_token),
             t, n_heads, n_kv, hd, g.block_size, float(scale), int(window), float(softcap),
-            cache.k_pool.shape[1], _ptr(sink), _ptr(slopes), keep_first, out.stride(0),
+            cache.k_pool.shape[1], _ptr(sink), _ptr(slopes), keep_first, out.stride(0), int(chunk),
             self._stream()), "attention_simt")
 
     def _split_launches(self, n_split: int, tma: bool, n_ctas: int) -> int:
@@ -753,6 +757,9 @@ class Ops:
             fns = {"add_layernorm": _decl(lib, "mls_add_layernorm",
                                           [_P, _P, _I, _I, _LL, _P, _P, _I, _P, _I, _F, _P, _I,
                                            _I, _I, _P, _P]),
+                   "add_post_layernorm": _decl(lib, "mls_add_post_layernorm",
+                                               [_P, _P, _I, _I, _LL, _P, _P, _P, _P, _P, _F, _P, _I,
+                                                _P, _P, _I, _I, _P]),
                    "residual_add": _decl(lib, "mls_residual_add", [_P, _P, _P, _I, _I, _I, _P]),
                    "settle_concat": _decl(lib, "mls_settle_concat",
                                           [_P, _P, _I, _I, _LL, _P, _P, _I, _I, _I, _P])}
@@ -787,6 +794,8 @@ class Ops:
                    "glu": _decl(lib, "mls_expert_glu",
                                 [_P, _P, _P, _I, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _F, _F,
                                  _P]),
+                   "relu2": _decl(lib, "mls_expert_relu2",
+                                  [_P, _P, _P, _I, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _P]),
                    "down": _decl(lib, "mls_expert_down",
                                  [_P, _P, _P, _I, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _P]),
                    "combine": _decl(lib, "mls_expert_combine",
@@ -803,7 +812,13 @@ class Ops:
         elif name == "headprep":
             fns = {"prep": _decl(lib, "mls_head_prep_store",
                                  [_P, _I, _I, _I, _I, _P, _P, _P, _P, _P, _F, _F, _I, _F, _P, _I, _F,
-                                  _P, _P, _P, _I, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P])}
+                                  _P, _P, _P, _I, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P]),
+                   "conv_rope": _decl(lib, "mls_head_conv_rope_store",
+                                      [_P, _I, _I, _P, _P, _I, _I, _P, _LL, _P, _P, _F, _P, _I, _F, _P,
+                                       _P, _P, _P, _P, _P, _I, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I,
+                                       _I, _I, _I, _P, _P]),
+                   "difference": _decl(lib, "mls_head_difference",
+                                       [_P, _I, _I, _F, _F, _F, _P, _I, _I, _P, _I, _I, _I, _P])}
         elif name == "side":
             fns = {"settle_cast": _decl(lib, "mls_settle_cast",
                                         [_P, _P, _I, _I, _LL, _P, _I, _I, _I, _P]),
@@ -874,6 +889,40 @@ class Ops:
             self._stream()), "add_layernorm")
         if isinstance(delta, SplitParts):
             delta.release()
+
+    def add_post_layernorm(self, x, y, post, eps: float, h, bias=None, norm=None, rows=None,
+                           n_rows: int = 0, y_out=None) -> None:
+        """A layer norm behind a sublayer, in the pass that adds its result to the stream: ``y``
+        (a tensor, ``SplitParts`` or None: nothing to add) plus ``bias``, normed with ``post = (w,
+        b)``; ``x += y``; ``h`` is the stream in ``h``'s type or, with ``norm = (w, b)``, such a
+        norm of it.  The vectors are float32.  With ``rows`` only those rows are read and ``x``
+        stays as it is.  ``x`` None and ``h`` None with ``y_out`` (float32): only the normed ``y``
+        is written."""
+        src = x if x is not None else y_out
+        t, d = src.shape
+        n_out = t if rows is None else n_rows
+        _need(x is None or (x.dtype == torch.float32 and x.is_contiguous()),
+              "add_post_layernorm: x must be float32")
+        _need(h is None or (h.shape == (n_out, d) and h.is_contiguous()),
+              "add_post_layernorm: bad output")
+        _need(y_out is None or (y_out.shape == (n_out, d) and y_out.dtype == torch.float32
+                                and y_out.is_contiguous()), "add_post_layernorm: bad result")
+        for v in (*(post or ()), *(norm or ()), bias):
+            _need(v is None or (v.dtype == torch.float32 and v.shape == (d,) and v.is_contiguous()),
+                  "add_post_layernorm: vectors are float32 [d]")
+        _need(y is None or post is not None, "add_post_layernorm: a result needs its norm")
+        _need(rows is None or (rows.dtype == torch.int32 and rows.numel() >= n_rows),
+              "add_post_layernorm: bad row indices")
+        yp, ycode, parts, stride = self._delta_args(y, t, d, "add_post_layernorm")
+        w1, b1 = post if post else (None, None)
+        w2, b2 = norm if norm else (None, None)
+        self.launches += 1
+        _check(self._part_lib("layernorm")["add_post_layernorm"](
+            _ptr(x), yp, ycode, parts, stride, _ptr(bias), _ptr(w1), _ptr(b1), _ptr(w2), _ptr(b2),
+            float(eps), _ptr(h), _code(h.dtype) if h is not None else 0, _ptr(y_out), _ptr(rows),
+            n_out, d, self._stream()), "add_post_layernorm")
+        if isinstance(y, SplitParts):
+            y.release()
 
     def residual_add(self, x, more_rows=None, more_vec=None) -> None:
         """``x += more_rows + more_vec`` on the float32 residual stream."""
@@ -994,12 +1043,13 @@ class Ops:
 
     def route(self, logits, top: int, renorm: bool, work: dict, softmax: bool = False,
               correction=None, renorm_eps: float = 0.0, n_real=None, groups=None,
-              n_outputs=None) -> None:
+              n_outputs=None, by_logit: bool = False) -> None:
         """Choose and sort: from float32 router ``logits [T, E]`` the ``top`` outputs a token
         with the largest score (sigmoid, or ``softmax`` over all outputs) plus ``correction``
         (float32 [E], in the choice only), the scores themselves as weights (``renorm``:
         divided by their sum + ``renorm_eps``), then the (token, choice) slots ordered by
-        expert.  Outputs from ``n_real`` on stand for experts without weights and get no
+        expert.  ``by_logit``: the outputs with the largest ``logits + correction`` are chosen and
+        a softmax over those gives the weights.  Outputs from ``n_real`` on stand for experts without weights and get no
         tiles.  ``groups = (count, keep)``: the outputs form ``count`` equal groups of
         neighbours, and only those of the ``keep`` groups whose two largest choice scores have
         the largest sum can be chosen.  ``n_outputs``: the first so many columns of a wider
@@ -1017,7 +1067,7 @@ class Ops:
         fns = self._part_lib("experts")
         self.launches += 2
         _check(fns["topk"](_ptr(logits), row, t, n_experts, top, 1 if renorm else 0,
-                           1 if softmax else 0, _ptr(correction), float(renorm_eps), n_groups, keep,
+                           2 if by_logit else 1 if softmax else 0, _ptr(correction), float(renorm_eps), n_groups, keep,
                            _ptr(work["idx"]), _ptr(work["weight"]), self._stream()), "route_topk")
         _check(fns["sort"](_ptr(work["idx"]), t * top, n_experts,
                            n_experts if n_real is None else int(n_real), _ptr(work["order"]),
@@ -1052,6 +1102,19 @@ class Ops:
             work["max_tiles"], _ptr(work["weight"]), top, 1 if scale_in else 0, f2 // 2, k,
             self._many_rows(y.shape[0], n_experts), float(alpha), float(limit), self._stream()),
             "expert_glu")
+
+    def expert_relu_squared(self, h, w_up, y, work: dict, top: int, scale_in: bool) -> None:
+        """``y[p] = relu(Wu[e] a)^2`` for the sorted slots; ``w_up [E, F, K]``."""
+        n_experts, f, k = w_up.shape
+        _need(h.dtype == w_up.dtype == y.dtype and h.is_contiguous() and y.is_contiguous()
+              and w_up.is_contiguous() and h.shape[1] == k and y.shape[1] == f,
+              "expert_relu_squared: operands")
+        self.launches += 1
+        _check(self._part_lib("experts")["relu2"](
+            _ptr(h), _ptr(w_up), _ptr(y), _code(h.dtype), _ptr(work["order"]),
+            _ptr(work["offsets"]), _ptr(work["tile_expert"]), _ptr(work["tile_row0"]),
+            work["max_tiles"], _ptr(work["weight"]), top, 1 if scale_in else 0, f, k,
+            self._many_rows(y.shape[0], n_experts), self._stream()), "expert_relu_squared")
 
     def expert_down(self, y, w_down, per_slot, work: dict, top: int, scale_out: bool) -> None:
         """``per_slot[slot] = Wd[e] y[p]`` (float32); ``w_down [E, D, F]``."""
@@ -1405,6 +1468,76 @@ class Ops:
             _ptr(step.positions), _ptr(g.slot_map), _ptr(q_out), q_out.shape[1], _code(pool.dtype),
             _ptr(pool), _ptr(cache.v_pool), g.block_size, pool.shape[1], t, n_heads, n_kv, e, f,
             hd, 1 if cache.writes else 0, _ptr(self.status), self._stream()), "head_prep_store")
+
+    def head_conv_rope_store(self, proj, col: int, bias, conv, taps: int, tail, norms, eps: float,
+                             freq, rot_dims: int, amplitude: float, q_out, cache, step,
+                             n_heads: int, n_kv: int, e: int, f: int, hd: int, maps: int = 1,
+                             move_tail: bool = False) -> None:
+        """From the float32 projection ``proj [T, W]`` with ``[q heads | k heads | v heads]`` from
+        column ``col`` on (``n_heads`` and ``n_kv`` heads of ``maps`` maps of ``e`` entries, values
+        of ``f``): add ``bias`` (float32 [channels] or None), convolve every channel over time
+        (``conv`` float32 [taps, channels]; inputs before the step from ``tail [slots, (taps - 1) *
+        channels]``; ``taps`` 0: no convolution), RMS-normalise every map of q and k with ``norms =
+        (w_q, w_k)`` (float32 [e], or None), turn entry i < rot_dims / 2 with entry i + rot_dims / 2
+        by position * ``freq[i]`` (float64), cosine and sine times ``amplitude``.  Map m of head h
+        goes to row ``h * maps + m`` of ``q_out`` (``hd`` entries each, zeros but in the map's
+        place), the maps of a key side by side and the values into the pages at the step's slots,
+        padded with zeros to ``hd``.  ``tail_update`` moves the tail on afterwards or, in a step of
+        one token a request, this kernel itself (``move_tail``)."""
+        g = step.groups[cache.group]
+        t = step.n_tokens
+        pool = cache.k_pool
+        c = (n_heads + n_kv) * maps * e + n_kv * f
+        _need(proj.dtype == torch.float32 and proj.is_contiguous() and proj.shape[0] == t
+              and 0 <= col and col + c <= proj.shape[1], "head_conv_rope_store: bad projection")
+        _need(pool.is_contiguous() and cache.v_pool.is_contiguous() and pool.shape[0] == n_kv
+              and pool.shape[3] == hd and hd >= max(maps * e, f) and q_out.dtype == pool.dtype
+              and q_out.is_contiguous() and q_out.shape[0] >= t
+              and q_out.shape[1] >= n_heads * maps * hd, "head_conv_rope_store: bad pool or output")
+        vecs = [v for v in (bias, conv, *(norms or ())) if v is not None]
+        _need(all(v.dtype == torch.float32 and v.is_contiguous() for v in vecs),
+              "head_conv_rope_store: float32 vectors")
+        _need(bias is None or bias.shape == (c,), "head_conv_rope_store: bad bias")
+        _need(taps == 0 or conv.shape == (taps, c), "head_conv_rope_store: bad taps")
+        _need(taps <= 1 or (tail.dtype == torch.float32 and tail.stride(1) == 1
+                            and tail.shape[1] == (taps - 1) * c), "head_conv_rope_store: bad tail")
+        w_q, w_k = norms if norms else (None, None)
+        _need(w_q is None or (w_q.shape == (e,) and w_k.shape == (e,)),
+              "head_conv_rope_store: bad norms")
+        _need(rot_dims == 0 or (rot_dims <= e and freq.dtype == torch.float64
+                                and freq.numel() == rot_dims // 2),
+              "head_conv_rope_store: bad frequencies")
+        _need(not move_tail or step.max_q_len == 1, "head_conv_rope_store: the tail moves in the "
+              "kernel only in steps of single tokens")
+        self.launches += 1
+        _check(self._part_lib("headprep")["conv_rope"](
+            _ptr(proj), proj.shape[1], col, _ptr(bias), _ptr(conv) if taps else None, taps,
+            1 if (move_tail and taps > 1) else 0, _ptr(tail) if taps > 1 else None,
+            tail.stride(0) if taps > 1 else 0, _ptr(w_q), _ptr(w_k), float(eps),
+            _ptr(freq) if rot_dims else None, rot_dims, float(amplitude), _ptr(step.state_slot),
+            _ptr(step.cu_q), _ptr(step.req_of_token), _ptr(step.positions), _ptr(g.slot_map),
+            _ptr(q_out), q_out.shape[1], _code(pool.dtype), _ptr(pool), _ptr(cache.v_pool),
+            g.block_size, pool.shape[1], t, n_heads, n_kv, maps, e, f, hd,
+            1 if cache.writes else 0, _ptr(self.status), self._stream()), "head_conv_rope_store")
+
+    def head_difference(self, o, hd: int, lam: float, mul: float, eps: float, gate, gate_col: int,
+                        out, n_heads: int, f: int) -> None:
+        """Two maps' outputs a head (rows ``2h`` and ``2h + 1`` of ``o [T, 2 H * hd]``, the first
+        ``f`` entries each) become ``a1 - lam * a2``, divided by its root mean square, times ``mul``
+        and, with ``gate`` (float32 rows), times ``sigmoid(gate[t, gate_col + h * f + c])``; ``out
+        [T, H * f]``."""
+        t = o.shape[0]
+        _need(o.shape == (t, 2 * n_heads * hd) and o.is_contiguous() and hd >= f
+              and out.shape == (t, n_heads * f) and out.is_contiguous() and out.dtype == o.dtype,
+              "head_difference: operands")
+        _need(gate is None or (gate.dtype == torch.float32 and gate.is_contiguous()
+                               and gate.shape[0] == t and gate.shape[1] >= gate_col + n_heads * f),
+              "head_difference: bad gate")
+        self.launches += 1
+        _check(self._part_lib("headprep")["difference"](
+            _ptr(o), _code(o.dtype), hd, float(lam), float(mul), float(eps), _ptr(gate),
+            gate.shape[1] if gate is not None else 0, gate_col, _ptr(out), t, n_heads, f,
+            self._stream()), "head_difference")
 
     def settle_cast(self, x, delta, out) -> None:
         """``x += delta`` (a tensor, ``SplitParts`` or None); ``out = x`` in ``out``'s type."""

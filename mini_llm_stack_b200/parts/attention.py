@@ -12,12 +12,14 @@ window w additionally hides keys ``j <= p - w`` from the query at position p.
 
 from __future__ import annotations
 
+import math
 import os
 from dataclasses import dataclass
 
 import torch
 
-from .base import CacheHandle, Mixer, PagedKV, StepContext, TensorSpec, stack_rows
+from .base import (CacheHandle, FixedState, Mixer, PagedKV, PagedWithState, StepContext,
+                   TensorSpec, stack_rows)
 
 
 @dataclass(frozen=True)
@@ -66,18 +68,19 @@ def context_splits(tiles: list, n_kv: int, slots: int = 296, cluster_splits: int
 
 
 def plan_paged_attention(step: StepContext, facts: dict, n_heads: int, n_kv_heads: int,
-                         head_dim: int):
+                         head_dim: int, span=None):
     """A step's ``AttentionPlan`` for heads of this shape (None where the kernel in use
     needs none), shared through ``step.attn_tiles`` by the mixers of the same shape.
 
     Requests whose (token, head) rows of one kv head fit ``small_rows`` go to the
     context-split kernel, their context cut so that all SMs have work; the others
-    are cut into tiles of rows."""
+    are cut into tiles of rows.  ``span``: a token reads at most so many keys (a window or a
+    chunk): the cut is planned for the tiles there are."""
     f = facts
     if not f["tensor_cores"]:
         return None
     group = n_heads // n_kv_heads
-    key = ("gqa", group, n_kv_heads, head_dim)
+    key = ("gqa", group, n_kv_heads, head_dim, span)
     plan = step.attn_tiles.get(key)
     if plan is None:
         small = [q * group <= f["small_rows"] for q in step.q_lens]
@@ -86,10 +89,11 @@ def plan_paged_attention(step: StepContext, facts: dict, n_heads: int, n_kv_head
         n_split = 1
         if n_small:
             keys = f.get("split_keys", 64)
-            tiles = [-(-c // keys) for c, s in zip(step.ctx_lens, small) if s]
+            most = (span + 15 + keys - 2) // keys + 1 if span else 1 << 30
+            tiles = [min(most, -(-c // keys)) for c, s in zip(step.ctx_lens, small) if s]
             n_split = context_splits(tiles, n_kv_heads, f["split_slots"],
                                      f.get("cluster_splits", 0),
-                                     longest=-(-step.max_ctx_len // keys),
+                                     longest=min(most, -(-step.max_ctx_len // keys)),
                                      cluster_slots=f.get("cluster_slots", 0))
         plan = AttentionPlan(
             n_tiles=sum(-(-r // f["tile_rows"]) for r in big),
@@ -393,3 +397,194 @@ class UnrotatedAttention(Mixer):
 
     def rider(self):
         return self._rider_rows, self.rider_col
+
+
+class RotatedAttention(Mixer):
+    """Grouped-query attention whose queries and keys are normed per head and rotated, behind an
+    optional short convolution on queries, keys and values.
+
+    With H query heads and G key/value heads, queries and keys of size e and values of size f
+    (query head h reads head ``h // (H/G)``), per token:
+
+        u = W h (+ b)                             for q, k and v        (``qkv_bias``)
+        y_t = sum_j w_j u_(t - taps + 1 + j)      every channel, zeros before the start  (``taps``)
+        q_h, k_g <- rms_norm(.) * w_q, w_k        weights [e] for all heads  (``head_norm``)
+        the first ``position.dims`` entries of q_h and k_g turn     (``PartialRotary``, halves)
+        score_ij = (q_i . k_j) * scale;  j visible to i iff j <= i and
+            i - j < window                        (``window``)
+            floor(i / chunk) = floor(j / chunk)   (``chunk``)
+        softmax, with ``sink`` plus one term exp(sink_h) without key or value
+        out = W_o concat_h(o)
+
+    Keys and values live in the paged cache, every head padded with zeros to the kernels' head
+    size; the convolution's last ``taps - 1`` inputs of every request in its state slot (the
+    mixer's cache is then a ``PagedWithState``).  Everything between the projection and the
+    cache is one kernel (``Ops.head_conv_rope_store``)."""
+
+    decode_capturable = prompt_capturable = True   # forward only launches kernels on the current stream
+    maps = 1                                       # attentions a head, over the same values
+    has_gate = False
+
+    def __init__(self, d_model: int, n_heads: int, n_kv_heads: int, head_dim: int, v_dim: int,
+                 scale: float, eps: float, position=None, taps: int = 0, window=None, chunk=None,
+                 qkv_bias: bool = True, head_norm: bool = True, sink: bool = False):
+        if n_heads % n_kv_heads:
+            raise ValueError("n_heads must be a multiple of n_kv_heads")
+        if window and chunk:
+            raise ValueError("a window or chunks, not both")
+        if position is not None and (position.pairing != "half" or position.dims > head_dim):
+            raise ValueError("this mixer's kernel turns the first dims entries by halves")
+        self.d_model, self.n_heads, self.n_kv_heads = int(d_model), int(n_heads), int(n_kv_heads)
+        self.head_dim, self.v_dim = int(head_dim), int(v_dim)
+        self.scale, self.eps = float(scale), float(eps)
+        self.position, self.taps = position, int(taps or 0)
+        self.window = int(window) if window else None
+        self.chunk = int(chunk) if chunk else None
+        self.qkv_bias, self.head_norm, self.has_sink = bool(qkv_bias), bool(head_norm), bool(sink)
+        self.q_heads = self.n_heads * self.maps              # rows of queries the kernels see
+        self.sizes = (self.q_heads * self.head_dim, self.n_kv_heads * self.maps * self.head_dim,
+                      self.n_kv_heads * self.v_dim)          # channels of q, k and v
+        self.channels = sum(self.sizes)
+        self.pad_dim = -(-max(self.maps * self.head_dim, self.v_dim) // 16) * 16
+
+    def tensor_specs(self) -> dict:
+        out = {}
+        for n, rows in zip("qkv", self.sizes):
+            out[n] = TensorSpec((rows, self.d_model))
+            if self.qkv_bias:
+                out[f"{n}.b"] = TensorSpec((rows,), kind="vector", init="zeros")
+            if self.taps:
+                out[f"{n}.conv"] = TensorSpec((rows, self.taps))
+        if self.head_norm:
+            for n in "qk":
+                out[f"{n}.norm"] = TensorSpec((self.head_dim,), kind="vector", init="ones")
+        if self.has_sink:
+            out["sink"] = TensorSpec((self.n_heads,), kind="vector", init="zeros")
+        if self.has_gate:
+            out["g"] = TensorSpec((self.n_heads * self.v_dim, self.d_model))
+        out["o"] = TensorSpec((self.d_model, self.n_heads * self.v_dim))
+        return out
+
+    def cache_spec(self):
+        paged = PagedKV(self.n_kv_heads, self.pad_dim, self.window, chunk=self.chunk)
+        if self.taps > 1:
+            return PagedWithState(paged, FixedState(((self.taps - 1) * self.channels,),
+                                                    torch.float32))
+        return paged
+
+    def bind(self, tensors: dict, runtime) -> None:
+        self.runtime = runtime
+        ops, f32 = runtime.ops, torch.float32
+        # one projection for everything that reads the mixer's input: [q | k | v | gate]
+        self.w_in = ops.prepare_weight(stack_rows(
+            [tensors[n] for n in ("q", "k", "v", *(("g",) if self.has_gate else ()))]))
+        self.bias = (torch.cat([tensors[f"{n}.b"].to(f32) for n in "qkv"]).contiguous()
+                     if self.qkv_bias else None)
+        # the taps of all channels side by side: [taps, channels]
+        self.conv = (torch.cat([tensors[f"{n}.conv"].to(f32) for n in "qkv"]).t().contiguous()
+                     if self.taps else None)
+        self.norms = (tuple(tensors[f"{n}.norm"].to(f32).contiguous() for n in "qk")
+                      if self.head_norm else None)
+        self.sink = tensors["sink"].to(f32).contiguous() if self.has_sink else None
+        if self.position is not None:
+            self.position.bind({}, runtime)
+        self.bind_output(tensors)
+        ops.require_part("headprep")
+        if self.taps > 1:
+            ops.require_part("shortconv")            # the tail's move lives there
+        self._tensor_cores = ops.attention_tensor_cores(self.pad_dim)
+        if self._tensor_cores:
+            ops.require_attention(self.pad_dim, self.q_heads, self.n_kv_heads)
+        self._facts = ops.attention_facts(self.pad_dim)
+
+    def bind_output(self, tensors: dict) -> None:
+        w = tensors["o"]
+        if self.pad_dim != self.v_dim:
+            # zero columns where the heads' outputs are padded
+            padded = w.new_zeros((self.d_model, self.n_heads, self.pad_dim))
+            padded[:, :, :self.v_dim] = w.view(self.d_model, self.n_heads, self.v_dim)
+            w = padded.view(self.d_model, self.n_heads * self.pad_dim)
+        self.w_o = self.runtime.ops.prepare_weight(w)
+
+    def plan(self, step: StepContext):
+        if not self._tensor_cores:
+            return None
+        return plan_paged_attention(step, self._facts, self.q_heads, self.n_kv_heads, self.pad_dim,
+                                    span=self.window or self.chunk)
+
+    def decode_graph_key(self, step: StepContext) -> tuple:
+        plan = self.plan(step)
+        if plan is None:
+            return ()
+        return ("gqa", self.n_kv_heads, self.q_heads // self.n_kv_heads, self.pad_dim,
+                self.window or self.chunk, plan.n_split)
+
+    def forward(self, h, step: StepContext, cache: CacheHandle):
+        rt, ops = self.runtime, self.runtime.ops
+        t, hd, pos = step.n_tokens, self.pad_dim, self.position
+        proj = rt.buffer("attn_proj", (t, self.w_in.shape[0]), torch.float32)
+        ops.linear(h, self.w_in, proj)
+        # the attention kernels read a row of [q heads | k heads | v heads]; only q is there
+        q_row = rt.buffer("qkv", (t, (self.q_heads + 2 * self.n_kv_heads) * hd), rt.act_dtype)
+        single = step.max_q_len == 1
+        ops.head_conv_rope_store(proj, 0, self.bias, self.conv, self.taps, cache.state, self.norms,
+                                 self.eps, pos.freq if pos else None, pos.dims if pos else 0,
+                                 pos.amplitude if pos else 1.0, q_row, cache, step, self.n_heads,
+                                 self.n_kv_heads, self.head_dim, self.v_dim, hd, maps=self.maps,
+                                 move_tail=single and cache.writes)
+        if self.taps > 1 and cache.writes and not single:
+            ops.tail_update(proj, 0, self.channels, self.bias, cache.state, self.taps - 1, step)
+        o = rt.buffer("attn_out", (t, self.q_heads * hd), rt.act_dtype)
+        ops.paged_attention(q_row, o, cache, step, self.q_heads, self.n_kv_heads, hd, self.scale,
+                            self.window or 0, plan=self.plan(step), sink=self.sink,
+                            simt=not self._tensor_cores, chunk=self.chunk or 0)
+        o = self.finish_heads(o, proj)
+        delta = rt.buffer("delta", (t, self.d_model), rt.act_dtype)
+        return ops.linear_parts(o, self.w_o, delta)
+
+    def finish_heads(self, o, proj):
+        """The heads' outputs as the output projection reads them."""
+        return o
+
+
+class DifferentialAttention(RotatedAttention):
+    """Two attentions a head over the same values, the second taken from the first, and an output
+    gate; without a sink.  q and k have two maps of size e a head, side by side; with a1, a2 the
+    two maps' outputs,
+
+        lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff
+        o = a1 - lambda a2;  o <- o / sqrt(mean(o^2) + eps) * (1 - diff)        per head
+        out = W_o (concat_h(o) * sigmoid(W_g h))
+
+    The cache holds a head's two keys as one row and its values once: a map's query is a query
+    head of its own that is zero in the other map's place, so both maps are one pass over the
+    same pages."""
+
+    maps = 2
+    has_gate = True
+
+    def __init__(self, d_model: int, n_heads: int, n_kv_heads: int, head_dim: int, v_dim: int,
+                 scale: float, eps: float, diff: float, **options):
+        super().__init__(d_model, n_heads, n_kv_heads, head_dim, v_dim, scale, eps, **options)
+        if self.has_sink:
+            raise ValueError("differential attention has no sink")
+        self.diff = float(diff)
+
+    def tensor_specs(self) -> dict:
+        out = super().tensor_specs()
+        for n in ("lq1", "lk1", "lq2", "lk2"):
+            out[n] = TensorSpec((self.head_dim,), kind="vector", init="zeros")
+        return out
+
+    def bind_output(self, tensors: dict) -> None:
+        self.w_o = self.runtime.ops.prepare_weight(tensors["o"])
+        lq1, lk1, lq2, lk2 = (tensors[n].double() for n in ("lq1", "lk1", "lq2", "lk2"))
+        # one number for the layer, read once, at load time
+        self.lam = (math.exp(float(lq1 @ lk1)) - math.exp(float(lq2 @ lk2))) + self.diff
+
+    def finish_heads(self, o, proj):
+        rt = self.runtime
+        out = rt.buffer("attn_difference", (o.shape[0], self.n_heads * self.v_dim), rt.act_dtype)
+        rt.ops.head_difference(o, self.pad_dim, self.lam, 1.0 - self.diff, self.eps, proj,
+                               self.channels, out, self.n_heads, self.v_dim)
+        return out

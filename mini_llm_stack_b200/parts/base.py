@@ -53,7 +53,8 @@ class TensorSpec:
 # ----------------------------------------------------------------------------
 @dataclass(frozen=True)
 class PagedKV:
-    """Keys and values of every token (or of the last ``window`` tokens).
+    """Keys and values of every token (or of the last ``window`` tokens, or of the current
+    ``chunk``: the sequence in chunks of so many tokens, counted from its start).
 
     ``shared_kv``: one pool serves as keys and as values (a mixer that attends over a
     single cached vector a token, such as a latent); the handle's ``k_pool`` and
@@ -64,6 +65,21 @@ class PagedKV:
     window: Optional[int] = None
     shared_kv: bool = False
     keep_first: int = 0
+    chunk: Optional[int] = None
+
+    def first_key(self, position: int) -> int:
+        """The first token that the token at ``position``, or any later one, still reads (beside
+        the kept first ones)."""
+        if self.window is not None:
+            return max(0, position - self.window + 1)
+        if self.chunk is not None:
+            return position - position % self.chunk
+        return 0
+
+    @property
+    def span(self) -> Optional[int]:
+        """The most tokens a token reads (beside the kept first ones); None: all before it."""
+        return self.window if self.window is not None else self.chunk
 
 
 @dataclass(frozen=True)

@@ -1,5 +1,6 @@
 """The arrangement of a layer's parts: the pre-norm residual block, the block with a norm before
-and behind every sublayer, and that block with a gate on every sublayer's result.
+and behind every sublayer, that block with a gate on every sublayer's result, and the block with
+norms behind the sublayers only.
 
 Reference (train/model.py:200-217): ``x = x + mixer(norm_a(x))``;
 ``x = x + feed_forward(norm_b(x))``.  The block owns the order and the names
@@ -11,6 +12,7 @@ from __future__ import annotations
 import torch
 
 from .base import CacheHandle, Part, ResidualStream, StepContext, TensorSpec
+from .norm import StreamRows
 
 
 def join_name(prefix: str, name: str) -> str:
@@ -214,3 +216,36 @@ class GatedSandwichBlock(SandwichBlock):
         h = self.ffn_norm.forward(stream)
         gate = self._gate(1, h)
         stream.push(self.ffn_post.gated(self.ffn.forward(h, step), gate, self.gate_b[1]))
+
+
+class PostNormBlock(PreNormBlock):
+    """Norms behind the sublayers only: ``x <- x + post1(mixer(x))``; ``x <- x + post2(ffn(x))``.
+    The sublayers read the stream itself (``StreamRows``), and that read is the pass in which the
+    sublayer before is normed and added: as many kernels as a pre-norm block has.  The norms are of
+    a kind that can wait on the stream (``norm.behind(delta, bias)``, e.g. ``LayerNorm``).
+
+    ``names``: prefixes of (mixer, its norm, ffn, its norm)."""
+
+    def __init__(self, mixer, mixer_post, ffn, ffn_post, d_model: int,
+                 names=("mix", "norm1", "mlp", "norm2")):
+        self.mixer, self.mixer_post, self.ffn, self.ffn_post = mixer, mixer_post, ffn, ffn_post
+        self.rows = StreamRows(d_model)
+        self.names = tuple(names)
+
+    def _named_parts(self):
+        parts = (self.mixer, self.mixer_post, self.ffn, self.ffn_post)
+        return [(n, p) for n, p in zip(self.names, parts) if p is not None]
+
+    def bind(self, tensors: dict, runtime) -> None:
+        super().bind(tensors, runtime)
+        self.rows.bind({}, runtime)
+
+    @staticmethod
+    def _push(stream: ResidualStream, post, out) -> None:
+        out, bias = out if isinstance(out, tuple) else (out, None)
+        stream.push(post.behind(out, bias))
+
+    def forward(self, stream: ResidualStream, step: StepContext, cache: CacheHandle) -> None:
+        self._push(stream, self.mixer_post, self.mixer.forward(self.rows.forward(stream), step, cache))
+        if self.ffn is not None:
+            self._push(stream, self.ffn_post, self.ffn.forward(self.rows.forward(stream), step))

@@ -39,6 +39,8 @@ class ConvKeyAttention(Mixer):
         self.softcap, self.window = float(softcap or 0.0), window
         if position is not None and position.pairing != "interleaved":
             raise ValueError("this mixer's kernel rotates neighbouring entries")
+        if position is not None:
+            position.require_unit_amplitude()
         self.channels = (self.n_heads + self.n_kv_heads) * self.head_dim
 
     def tensor_specs(self) -> dict:

@@ -161,11 +161,12 @@ class SquaredReluFeedForward(FeedForward):
 
 
 class RoutedExperts(FeedForward):
-    """A mixture of small SwiGLU experts behind a float32 router.
+    """A mixture of small experts (SwiGLU, clamped or ungated) behind a float32 router.
 
     Router logits ``z = W_r h`` and scores ``s = sigmoid(z)`` or, with ``score="softmax"``,
     ``softmax(z)`` over all router outputs, in float32; a token takes its ``top`` outputs
-    with the largest scores (lowest index on a tie; with ``correction`` the vector
+    with the largest scores (``score="logit"``: with the largest logits, weighed by a softmax over
+    the chosen logits; lowest index on a tie; with ``correction`` the vector
     ``correction`` [outputs] is added for the choice only) and weighs them by the scores
     themselves (``renormalise``: divided by their sum + ``renorm_eps``).  ``weigh`` says
     where a weight multiplies: "input" (the expert sees ``w * h``) or "output".  The last
@@ -176,7 +177,9 @@ class RoutedExperts(FeedForward):
     ``count`` equal groups of neighbours, a group's score is the sum of its two largest choice
     scores, and only outputs of the ``keep`` best groups can be chosen.  ``limit`` > 0: the
     experts are clamped units, ``g' * sigmoid(alpha g') * (u' + 1)`` with ``g' = min(g, limit)``
-    and ``u' = clamp(u, -limit, limit)``, instead of ``silu(g) * u``.  Tensors: ``router``
+    and ``u' = clamp(u, -limit, limit)``, instead of ``silu(g) * u``; ``unit="relu_squared"``:
+    they have no gate, ``W_down relu(W_up h)^2``.  ``router_bias``: a bias of the logits (float32
+    ``router.b``).  Tensors: ``router``
     [E + identity, d] and ``e<i>.gate / up / down`` for each of the E experts; the shared
     part's under ``shared``."""
 
@@ -185,11 +188,16 @@ class RoutedExperts(FeedForward):
     def __init__(self, d_model: int, n_experts: int, top: int, expert_size: int, shared=None,
                  weigh: str = "input", renormalise: bool = False, score: str = "sigmoid",
                  correction: bool = False, identity: int = 0, renorm_eps: float = 0.0,
-                 groups=None, limit: float = 0.0, alpha: float = 1.0, shared_gate: bool = False):
+                 groups=None, limit: float = 0.0, alpha: float = 1.0, shared_gate: bool = False,
+                 unit: str = "gated", router_bias: bool = False):
         if weigh not in ("input", "output"):
             raise ValueError(f"weigh must be 'input' or 'output', not {weigh!r}")
-        if score not in ("sigmoid", "softmax"):
-            raise ValueError(f"score must be 'sigmoid' or 'softmax', not {score!r}")
+        if score not in ("sigmoid", "softmax", "logit"):
+            raise ValueError(f"score must be 'sigmoid', 'softmax' or 'logit', not {score!r}")
+        if unit not in ("gated", "relu_squared"):
+            raise ValueError(f"unit must be 'gated' or 'relu_squared', not {unit!r}")
+        if router_bias and (score != "logit" or correction):
+            raise ValueError("a bias of the logits goes with score='logit' and no correction")
         if not 0 < int(top) <= int(n_experts) + int(identity):
             raise ValueError("top must lie in 1..n_experts + identity")
         if identity and weigh != "output":
@@ -209,6 +217,7 @@ class RoutedExperts(FeedForward):
             if self.top > keep * (self.n_outputs // count):
                 raise ValueError("the kept groups hold fewer outputs than a token takes")
         self.limit, self.alpha = float(limit), float(alpha)
+        self.unit, self.router_bias = unit, bool(router_bias)
         self.shared_gate = bool(shared_gate)
         if self.shared_gate and shared is None:
             raise ValueError("a gate on the shared expert needs a shared expert")
@@ -218,8 +227,11 @@ class RoutedExperts(FeedForward):
         out = {"router": TensorSpec((self.n_outputs, d))}
         if self.has_correction:
             out["correction"] = TensorSpec((self.n_outputs,), kind="vector", init="zeros")
+        if self.router_bias:
+            out["router.b"] = TensorSpec((self.n_outputs,), kind="vector", init="zeros")
         for i in range(self.n_experts):
-            out[f"e{i}.gate"] = TensorSpec((f, d))
+            if self.unit == "gated":
+                out[f"e{i}.gate"] = TensorSpec((f, d))
             out[f"e{i}.up"] = TensorSpec((f, d))
             out[f"e{i}.down"] = TensorSpec((d, f))
         if self.shared is not None:
@@ -237,8 +249,13 @@ class RoutedExperts(FeedForward):
             self.w_router = torch.cat([self.w_router, tensors["shared.sg"].float()], 0).contiguous()
         if self.has_correction:
             self.correction = tensors["correction"].float().contiguous()
-        self.w_gate_up = torch.stack([torch.cat([tensors[f"e{i}.gate"], tensors[f"e{i}.up"]], 0)
-                                      for i in range(n)]).contiguous()
+        if self.router_bias:
+            self.correction = tensors["router.b"].float().contiguous()
+        if self.unit == "gated":
+            self.w_gate_up = torch.stack([torch.cat([tensors[f"e{i}.gate"], tensors[f"e{i}.up"]], 0)
+                                          for i in range(n)]).contiguous()
+        else:
+            self.w_up = torch.stack([tensors[f"e{i}.up"] for i in range(n)]).contiguous()
         self.w_down = torch.stack([tensors[f"e{i}.down"] for i in range(n)]).contiguous()
         if self.shared is not None:
             self.shared.bind({k[len("shared."):]: v for k, v in tensors.items()
@@ -266,12 +283,15 @@ class RoutedExperts(FeedForward):
         work = self._work(t)
         ops.route(logits, self.top, self.renormalise, work, softmax=self.score == "softmax",
                   correction=self.correction, renorm_eps=self.renorm_eps, n_real=self.n_experts,
-                  groups=self.groups, n_outputs=self.n_outputs)
+                  groups=self.groups, n_outputs=self.n_outputs, by_logit=self.score == "logit")
         n_slots = t * self.top
         y = rt.buffer("expert_act", (n_slots, self.expert_size), rt.act_dtype)
         per_slot = rt.buffer("expert_out", (n_slots, self.d_model), torch.float32)
-        ops.expert_glu(h, self.w_gate_up, y, work, self.top, self.weigh == "input",
-                       alpha=self.alpha, limit=self.limit)
+        if self.unit == "gated":
+            ops.expert_glu(h, self.w_gate_up, y, work, self.top, self.weigh == "input",
+                           alpha=self.alpha, limit=self.limit)
+        else:
+            ops.expert_relu_squared(h, self.w_up, y, work, self.top, self.weigh == "input")
         ops.expert_down(y, self.w_down, per_slot, work, self.top, self.weigh == "output")
         shared = None
         if self.shared is not None:

@@ -147,6 +147,8 @@ class RotaryLatentAttention(Mixer):
         self.cache_window = cache_window if own_cache else None
         if position is not None and position.dims > self.rot_dim:
             raise ValueError("the rotated part turns its first dims entries, dims <= rot_dim")
+        if position is not None:
+            position.require_unit_amplitude()
         if own_cache and window is not None and cache_window is not None and cache_window < window:
             raise ValueError("the cache keeps fewer tokens than the window sees")
         width = self.kv_rank + self.rot_dim

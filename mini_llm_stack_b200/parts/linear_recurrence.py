@@ -126,6 +126,8 @@ class RetentionMixer(Mixer):
             raise ValueError("retention needs one decay a head")
         if position is not None and position.pairing != "half":
             raise ValueError("this mixer's kernel rotates entry i with i + dims/2")
+        if position is not None:
+            position.require_unit_amplitude()
         self.position = position
 
     def tensor_specs(self) -> dict:

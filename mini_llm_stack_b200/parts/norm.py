@@ -1,6 +1,7 @@
 """Norms: RMS norm with a learned weight (a vector or one number; also behind a sublayer, with a
-gate on the sublayer's result), layer norm with a weight and no bias, and the norm without
-statistics (a scaled tanh with a weight and a bias).
+gate on the sublayer's result), layer norm with a weight and maybe a bias (also behind a
+sublayer), the norm without statistics (a scaled tanh with a weight and a bias), and, for layers
+that read the stream itself, none.
 
 Reference formula (train/model.py:29-33): ``xf = x.float()``;
 ``y = xf * rsqrt(mean(xf**2, -1) + eps)``; ``out = (y * w.float()).to(x.dtype)``.
@@ -114,28 +115,123 @@ class RMSNorm(Norm):
         return h
 
 
-class LayerNorm(Norm):
-    """``(x - mean) / sqrt(var + eps) * w`` with the biased variance and no bias, in
-    float32 with one rounding.  Adds the stream's pending delta and its other waiting
-    addends (``ResidualStream.push_more``) in the same pass.  ``tensor_name`` is the
-    local name of the weight ("" = the part's own prefix)."""
+class NormedDelta:
+    """A sublayer's output that is still to be layer-normed (plus ``bias``, a vector for every row,
+    first) before it joins the residual stream.  ``settle_normed`` does it in the pass in which it
+    adds the delta; any other consumer gets the values through ``resolve()`` (one kernel of its
+    own, float32)."""
+
+    def __init__(self, delta, norm: "LayerNorm", bias=None):
+        self.delta, self.norm, self.bias = delta, norm, bias
+
+    @property
+    def shape(self):
+        return self.delta.shape
+
+    def release(self) -> None:
+        if hasattr(self.delta, "release"):
+            self.delta.release()
+
+    def resolve(self):
+        rt = self.norm.runtime
+        out = rt.buffer("normed_delta", tuple(self.delta.shape), torch.float32)
+        rt.ops.add_post_layernorm(None, self.delta, self.norm.vectors, self.norm.eps, None,
+                                  bias=self.bias, y_out=out)
+        return out
+
+    def float(self):
+        return self.resolve()
+
+
+def settle_normed(rt, stream: ResidualStream, h, norm=None, rows=None, n_rows: int = 0) -> None:
+    """Add what waits on the stream and leave the stream's rows (all, or ``rows``) in ``h``: as they
+    are, or through ``norm``, a ``LayerNorm`` with a bias.  One kernel where a ``NormedDelta`` of
+    the same eps waits, or nothing."""
+    more_rows, more_vec = stream.take_more()
+    delta = stream.take_pending()
+    eps = norm.eps if norm is not None else None
+    if isinstance(delta, NormedDelta) and (eps is None or eps == delta.norm.eps):
+        y, post, bias, eps = delta.delta, delta.norm.vectors, delta.bias, delta.norm.eps
+    else:
+        if delta is not None:
+            rt.ops.residual_add(stream.x, delta.float())
+        y = post = bias = None
+    if more_rows is not None or more_vec is not None:
+        rt.ops.residual_add(stream.x, more_rows, more_vec)
+    rt.ops.add_post_layernorm(stream.x, y, post, eps or 0.0, h, bias=bias,
+                              norm=norm.vectors if norm is not None else None, rows=rows,
+                              n_rows=n_rows)
+
+
+class StreamRows(Norm):
+    """In the place of a norm before a sublayer that reads the residual stream itself: adds what
+    waits on the stream and gives its rows in the activations' type."""
 
     decode_capturable = prompt_capturable = True
 
-    def __init__(self, dim: int, eps: float, tensor_name: str = "weight"):
-        self.dim, self.eps, self.tensor_name = int(dim), float(eps), tensor_name
-        self.weight = None
-
-    def tensor_specs(self) -> dict:
-        return {self.tensor_name: TensorSpec((self.dim,), kind="vector", init="ones")}
+    def __init__(self, dim: int):
+        self.dim = int(dim)
 
     def bind(self, tensors: dict, runtime) -> None:
         self.runtime = runtime
-        self.weight = tensors[self.tensor_name].contiguous()
         runtime.ops.require_part("layernorm")
 
     def forward(self, stream: ResidualStream, rows=None, n_rows: int = 0):
         rt = self.runtime
+        n, name = (stream.x.shape[0], "normed") if rows is None else (n_rows, "normed_rows")
+        h = rt.buffer(name, (n, self.dim), rt.act_dtype)
+        settle_normed(rt, stream, h, rows=rows, n_rows=n_rows)
+        return h
+
+
+class LayerNorm(Norm):
+    """``(x - mean) / sqrt(var + eps) * w (+ b)`` with the biased variance, in
+    float32 with one rounding.  Adds the stream's pending delta and its other waiting
+    addends (``ResidualStream.push_more``) in the same pass.  ``tensor_name`` is the
+    local name of the weight ("" = the part's own prefix); with ``bias`` the tensor ``b`` lies
+    beside it.
+
+    Behind a sublayer (a norm with a bias only) it does not run by itself: ``behind(delta,
+    bias)`` wraps the sublayer's output, and what adds that to the stream norms it."""
+
+    decode_capturable = prompt_capturable = True
+
+    def __init__(self, dim: int, eps: float, tensor_name: str = "weight", bias: bool = False):
+        self.dim, self.eps, self.tensor_name = int(dim), float(eps), tensor_name
+        self.has_bias = bool(bias)
+        self.weight = self.vectors = None
+
+    def _bias_name(self) -> str:
+        return f"{self.tensor_name}.b" if self.tensor_name else "b"
+
+    def tensor_specs(self) -> dict:
+        out = {self.tensor_name: TensorSpec((self.dim,), kind="vector", init="ones")}
+        if self.has_bias:
+            out[self._bias_name()] = TensorSpec((self.dim,), kind="vector", init="zeros")
+        return out
+
+    def bind(self, tensors: dict, runtime) -> None:
+        self.runtime = runtime
+        self.weight = tensors[self.tensor_name].contiguous()
+        if self.has_bias:
+            self.vectors = (self.weight.float().contiguous(),
+                            tensors[self._bias_name()].float().contiguous())
+        runtime.ops.require_part("layernorm")
+
+    def behind(self, delta, bias=None) -> NormedDelta:
+        """``delta`` (a tensor or ``SplitParts``; ``bias`` a vector added to every row first) as
+        what this norm makes of it, for ``ResidualStream.push``."""
+        if not self.has_bias:
+            raise RuntimeError("a layer norm behind a sublayer has a weight and a bias")
+        return NormedDelta(delta, self, None if bias is None else bias.float().contiguous())
+
+    def forward(self, stream: ResidualStream, rows=None, n_rows: int = 0):
+        rt = self.runtime
+        if self.has_bias:
+            n, name = (stream.x.shape[0], "normed") if rows is None else (n_rows, "normed_rows")
+            h = rt.buffer(name, (n, self.dim), rt.act_dtype)
+            settle_normed(rt, stream, h, norm=self, rows=rows, n_rows=n_rows)
+            return h
         more_rows, more_vec = stream.take_more()
         delta = stream.take_pending()
         if rows is None:

@@ -15,6 +15,9 @@ same float32 values; the rotation itself runs in float32 and rounds once.
 
 from __future__ import annotations
 
+import math
+from dataclasses import dataclass
+
 import torch
 
 from .base import CacheHandle, PositionEncoding, StepContext
@@ -72,33 +75,92 @@ class RotaryPosition(PositionEncoding):
             self.head_dim, self.max_positions, cache.writes, parts=parts)
 
 
+@dataclass(frozen=True)
+class BandScaling:
+    """Frequencies by wavelength (Llama 3.1): with l = 2 pi / f, f stays where
+    l < original / high, becomes f / factor where l > original / low, and between the two, with
+    s = (original / l - low) / (high - low), (1 - s) f / factor + s f."""
+    factor: float
+    low: float
+    high: float
+    original: float
+    amplitude = 1.0
+
+    def apply(self, freq, base: float):
+        wavelength = 2.0 * math.pi / freq
+        s = (self.original / wavelength - self.low) / (self.high - self.low)
+        mixed = (1.0 - s) * freq / self.factor + s * freq
+        out = torch.where(wavelength > self.original / self.low, freq / self.factor, mixed)
+        return torch.where(wavelength < self.original / self.high, freq, out)
+
+
+@dataclass(frozen=True)
+class YarnScaling:
+    """Frequencies by the number of the pair (YaRN): a pair that turns more than ``fast`` times over
+    ``original`` positions keeps its frequency, one that turns fewer than ``slow`` times gets
+    f / factor, those between a mixture linear in the pair's number; cosine and sine are
+    multiplied by 0.1 ln(factor) + 1."""
+    factor: float
+    original: float
+    fast: float
+    slow: float
+
+    @property
+    def amplitude(self) -> float:
+        return 0.1 * math.log(self.factor) + 1.0
+
+    def apply(self, freq, base: float):
+        dims = 2 * freq.numel()
+
+        def pair_of(turns):
+            return dims * math.log(self.original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+
+        lo = max(math.floor(pair_of(self.fast)), 0)
+        hi = min(math.ceil(pair_of(self.slow)), dims - 1)
+        i = torch.arange(freq.numel(), dtype=torch.float64)
+        ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+        return freq / self.factor * ramp + freq * (1.0 - ramp)
+
+
 class PartialRotary(PositionEncoding):
     """Rotation of the first ``dims`` entries of every head; the rest pass unchanged.
 
     The pair number i (0 <= i < dims/2) at position p turns by the angle
     ``p * base^(-2i/dims) / factor`` (``factor``: linear scaling of the frequencies):
     ``(u, v) -> (u cos - v sin, v cos + u sin)``.  ``pairing`` says which entries form
-    pair i: "interleaved" (2i, 2i + 1) or "half" (i, i + dims/2).  There is no table
+    pair i: "interleaved" (2i, 2i + 1) or "half" (i, i + dims/2).  ``scaling`` (``BandScaling``,
+    ``YarnScaling``) changes the frequencies and may ask that cosine and sine be multiplied by
+    its ``amplitude`` (only some kernels do: the others' mixers refuse it).  There is no table
     and so no bound on the positions: the kernels that rotate form the angle in float64
     from the position and this part's float64 frequencies, and round its cosine and
     sine once to float32."""
 
     decode_capturable = prompt_capturable = True
 
-    def __init__(self, dims: int, base: float, factor: float = 1.0, pairing: str = "half"):
+    def __init__(self, dims: int, base: float, factor: float = 1.0, pairing: str = "half",
+                 scaling=None):
         if pairing not in ("interleaved", "half"):
             raise ValueError(f"pairing must be 'interleaved' or 'half', not {pairing!r}")
         if dims < 0 or dims % 2:
             raise ValueError("the rotated entries of a head come in pairs")
         self.dims, self.base, self.factor = int(dims), float(base), float(factor)
-        self.pairing = pairing
+        self.pairing, self.scaling = pairing, scaling
+        self.amplitude = scaling.amplitude if scaling is not None else 1.0
         self.freq = None
 
     def frequencies(self):
-        """``base^(-2i/dims) / factor`` for i < dims/2, float64 on the host."""
+        """``base^(-2i/dims) / factor``, scaled, for i < dims/2, float64 on the host."""
         i = torch.arange(self.dims // 2, dtype=torch.float64)
-        return torch.pow(torch.tensor(self.base, dtype=torch.float64),
+        freq = torch.pow(torch.tensor(self.base, dtype=torch.float64),
                          -2.0 * i / max(self.dims, 1)) / self.factor
+        if self.scaling is not None and self.dims:
+            freq = self.scaling.apply(freq, self.base)
+        return freq
+
+    def require_unit_amplitude(self) -> None:
+        """For a mixer whose kernel does not multiply cosine and sine."""
+        if self.amplitude != 1.0:
+            raise ValueError("this mixer's kernel does not scale the rotation's cosine and sine")
 
     def bind(self, tensors: dict, runtime) -> None:
         self.runtime = runtime

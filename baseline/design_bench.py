@@ -1,4 +1,4 @@
-"""``bench.py --design zededra | logulix | zefenex | movazen | nekedra``: prefill and decode
+"""``bench.py --design zededra | logulix | zefenex | movazen | nekedra | sevazen``: prefill and decode
 throughput of the design's layers at sizes that resemble a real model's, beside the dense
 Llama-style decoder at equal size.
 
@@ -152,19 +152,52 @@ def nekedra_config(s: dict, kind: str, layers: int, vocab: int = 32000) -> dict:
             "layers": stack}
 
 
+def sevazen_config(s: dict, kind: str, layers: int, vocab: int = 32000) -> dict:
+    """Layers of Sevazen's mixers: windowed attention with the dense decoder's heads (a window of
+    1,024, four taps, sinks, full rotation with scaled frequencies), differential attention with as
+    many heads of two maps of half the head size over the same cache bytes (chunks of 1,100 tokens:
+    a token decoded at 2,048 sees 948 before it), with the ungated feed-forward or with routed
+    ungated experts and a gated shared one; ``turns_moe`` alternates the two."""
+    kv = max(1, s["kv_rank"] // (2 * s["dim"]), s["heads"] // 16)
+    heads, dim = s["heads"], s["dim"]
+    attention = {"type": "attention",
+                 "mixer": {"conv": 4, "dim": dim, "heads": heads, "kv_heads": kv, "vdim": dim,
+                           "scale": dim ** -0.5, "mask": {"size": 1024},
+                           "rot": {"base": 500000.0, "dims": dim,
+                                   "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0,
+                                               "original": 8192}}}}
+    pair = {"type": "attention_2",
+            "mixer": {"diff": 0.4, "dim": dim // 2, "heads": heads, "kv_heads": kv, "vdim": dim,
+                      "scale": (dim // 2) ** -0.5, "mask": {"size": 1100},
+                      "rot": {"base": 10000.0, "dims": dim // 2,
+                              "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0,
+                                          "slow": 1.0}}}}
+    dense = {"ff": s["ff"], "kind": "dense"}
+    moe = {"expert": {"ff": s["eff"]}, "kind": "moe",
+           "router": {"experts": s["experts"], "top": s["top"]}, "shared": {"ff": s["shared"]}}
+    mlp = moe if kind.endswith("moe") else dense
+    turns = {"attention": [attention], "differential": [pair], "turns": [attention, pair]}[
+        kind.split("_")[0]]
+    return {"architecture": "Sevazen", "vocab": vocab, "width": s["width"], "norm": {"eps": 1e-5},
+            "layers": [dict(turns[i % len(turns)], mlp=mlp) for i in range(layers)]}
+
+
 DESIGNS = {
     "zededra": (zededra_config, ("latent_dense", "latent_moe", "mlstm_dense")),
     "logulix": (logulix_config, ("attention_dense", "wkv_dense", "retention_dense")),
     "zefenex": (zefenex_config, ("latent_dense", "latent_moe", "shared_cache_dense")),
     "movazen": (movazen_config, ("attention_moe", "parallel_moe", "mixers_only")),
     "nekedra": (nekedra_config, ("delta_dense", "latent_dense", "attention_dense", "turns_dense")),
+    "sevazen": (sevazen_config, ("attention_dense", "differential_dense", "attention_moe",
+                                 "turns_moe")),
 }
 # rows of another design measured beside a design's own: the closest existing layers
 BESIDE = {"zefenex": (("zededra", "latent_dense"), ("zededra", "latent_moe")),
           "movazen": (("zefenex", "latent_moe"), ("logulix", "attention_dense"),
                       ("logulix", "retention_dense")),
           "nekedra": (("logulix", "retention_dense"), ("zefenex", "latent_dense"),
-                      ("logulix", "attention_dense"))}
+                      ("logulix", "attention_dense")),
+          "sevazen": (("logulix", "attention_dense"), ("movazen", "attention_moe"))}
 
 
 def llama_config(s: dict, layers: int, vocab: int = 32000) -> dict:
@@ -185,7 +218,8 @@ _LEAVES = ("embed", "add_rmsnorm", "gather_add_rmsnorm", "add_layernorm", "resid
            "decay_lowrank", "relu_squared", "scale_", "settle_concat", "add_tanh_norm",
            "latent_rope_prep", "sigmoid_gate", "softcap_", "head_prep_store", "settle_cast",
            "gelu_gate_rows", "rms_scale", "scan_finish_row", "add_gated_norm", "delta_prep",
-           "delta_scan", "delta_step")
+           "delta_scan", "delta_step", "add_post_layernorm", "head_conv_rope_store",
+           "head_difference", "expert_relu_squared")
 _PRODUCTS = ("linear", "linear_parts", "linear_swiglu", "linear_clamped_glu",
              "linear_relu_squared")
 

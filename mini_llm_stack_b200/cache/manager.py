@@ -333,13 +333,15 @@ class CacheManager:
                                  f"but the tables name {held}")
 
     # -------------------------------------------------------------- step arrays
-    def step_arrays(self, entries: list) -> dict:
+    def step_arrays(self, entries: list, width: int | None = None) -> dict:
         """Per paged group, the block-table rows and slot map of a step.
 
         ``entries`` is ``[(owner, n_tokens)]`` in batch order; pages for the
         tokens must have been reserved.  Returns ``{gid: (block_table [R,
-        max_blocks] int32, slot_map [T] int32)}`` as numpy arrays.
+        max_blocks] int32, slot_map [T] int32)}`` as numpy arrays.  ``width``: only so many
+        entries of every block-table row (no request of the step holds more pages).
         """
+        width = self.max_blocks if width is None else min(width, self.max_blocks)
         out = {}
         bs = self.block_size
         recs = [self._records[o] for o, _ in entries]
@@ -352,11 +354,11 @@ class CacheManager:
                 pages = g.table[rows_a, pos // bs]
                 if pages.size and pages.min() < 0:
                     raise CacheError("no page reserved for a token of this step")
-                out[g.gid] = (g.table[rows_a],
+                out[g.gid] = (g.table[rows_a, :width],
                               (pages.astype(np.int64) * bs + pos % bs).astype(np.int32))
             return out
         for g in self.paged:
-            table = g.table[rows]
+            table = g.table[rows, :width]
             slot_parts = []
             for (owner, n), row in zip(entries, rows):
                 rec = self._records[owner]

@@ -31,7 +31,8 @@
 // and its score against the cached row is that of its own map's key.  The convolution's last
 // taps - 1 inputs of every request are a tail [taps - 1, channels] (float32, oldest first) in its
 // state slot; mls_tail_update moves it on behind this kernel or, in a step of one token a request,
-// this kernel does itself.  A warp a map (or value head) and run of tokens.
+// this kernel does itself.  A warp a map (or value head) and run of tokens.  Which of two kernels
+// and how many entries a lane takes depends on the model's sizes alone.
 //
 // mls_head_difference: what becomes of two maps' outputs a head, a warp a (token, head):
 //   o = a1 - lambda a2 ;  o <- o / sqrt(mean(o^2) + eps) * mul ;  o <- o * sigmoid(gate)
@@ -173,21 +174,16 @@ __device__ __forceinline__ void store_elems(__nv_bfloat16* p, const Pack<V>& r) 
         *p = __float2bfloat16_rn(r.v[0]);
 }
 
-// V: neighbouring entries a lane takes at a time (the model's sizes decide).
-template <typename T, int V>
-__global__ void __launch_bounds__(HC_WARPS * 32)
-head_conv_rope_kernel(const HeadConvArgs a, T* __restrict__ q_out, T* __restrict__ k_pool,
-                      T* __restrict__ v_pool) {
-    chain_release();
-    extern __shared__ __align__(16) float hc_smem[];
-    __shared__ int slot_s[HC_RUN], rest_s[HC_RUN], at_s[HC_RUN], state_s[HC_RUN];
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int t0 = blockIdx.x * a.run, n_run = min(a.run, a.n_tokens - t0);
-    const int half = a.rot / 2, widest = max(a.e, a.f);
-    float* angles = hc_smem;                                     // [run][cos | sin]
-    float* stage = hc_smem + (((size_t)a.run * a.rot + 3) & ~(size_t)3) +
-                   (size_t)warp * ((widest + 3) & ~3);           // this warp's head
-    // the step's index arrays are its input: no kernel of the step writes them
+// What the kernels below look up once for a run of tokens: each token's cache slot (-1: none), the
+// slots behind it to clear, its place among its request's tokens of this step and its request's
+// state slot; and the angles' cosines and sines.  All of it is the step's own input, which no kernel
+// of the step writes.
+struct RunTokens {
+    int slot[HC_RUN], rest[HC_RUN], at[HC_RUN], state[HC_RUN];
+};
+__device__ __forceinline__ void look_up_run(const HeadConvArgs& a, int t0, int n_run, RunTokens& R,
+                                            float* angles) {
+    const int half = a.rot / 2;
     if (threadIdx.x < n_run) {
         const int t = t0 + threadIdx.x, r = a.req_of_token[t];
         int slot = -1, rest = 0;
@@ -200,10 +196,10 @@ head_conv_rope_kernel(const HeadConvArgs a, T* __restrict__ q_out, T* __restrict
                 rest = page_tail_to_clear(a.slot_map, t, a.n_tokens, slot, a.block_size);
             }
         }
-        slot_s[threadIdx.x] = slot;
-        rest_s[threadIdx.x] = rest;
-        at_s[threadIdx.x] = t - a.cu_q[r];
-        state_s[threadIdx.x] = a.taps > 1 ? a.state_slot[r] : 0;
+        R.slot[threadIdx.x] = slot;
+        R.rest[threadIdx.x] = rest;
+        R.at[threadIdx.x] = t - a.cu_q[r];
+        R.state[threadIdx.x] = a.taps > 1 ? a.state_slot[r] : 0;
     }
     for (int u = threadIdx.x; u < n_run * half; u += blockDim.x) {
         const int tok = u / half, i = u - tok * half;
@@ -213,6 +209,32 @@ head_conv_rope_kernel(const HeadConvArgs a, T* __restrict__ q_out, T* __restrict
         angles[tok * a.rot + half + i] = s * a.amplitude;
     }
     __syncthreads();
+}
+template <typename T>
+__device__ __forceinline__ void clear_run_tails(const HeadConvArgs& a, int n_run, const RunTokens& R,
+                                                T* k_pool, T* v_pool) {
+    if (!a.writes || blockIdx.y != 0) return;
+    for (int tok = 0; tok < n_run; ++tok)
+        if (R.slot[tok] >= 0)
+            clear_page_tail<T>(R.rest[tok], R.slot[tok], a.block_size, a.n_pages, a.n_kv, a.hd, k_pool,
+                               v_pool);
+}
+
+// V: neighbouring entries a lane takes at a time (the model's sizes decide).
+template <typename T, int V>
+__global__ void __launch_bounds__(HC_WARPS * 32)
+head_conv_rope_kernel(const HeadConvArgs a, T* __restrict__ q_out, T* __restrict__ k_pool,
+                      T* __restrict__ v_pool) {
+    chain_release();
+    extern __shared__ __align__(16) float hc_smem[];
+    __shared__ RunTokens R;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int t0 = blockIdx.x * a.run, n_run = min(a.run, a.n_tokens - t0);
+    const int half = a.rot / 2, widest = max(a.e, a.f);
+    float* angles = hc_smem;                                     // [run][cos | sin]
+    float* stage = hc_smem + (((size_t)a.run * a.rot + 3) & ~(size_t)3) +
+                   (size_t)warp * ((widest + 3) & ~3);           // this warp's head
+    look_up_run(a, t0, n_run, R, angles);
     chain_wait();
     const int nq = a.n_heads * a.maps, nk = a.n_kv * a.maps;
     const int units = nq + (a.writes ? nk + a.n_kv : 0);
@@ -232,8 +254,8 @@ head_conv_rope_kernel(const HeadConvArgs a, T* __restrict__ q_out, T* __restrict
         const int c_lo = kind == 1 ? inside : 0;
         const int c_hi = (kind == 1 && map + 1 < a.maps) ? inside + a.e : a.hd;
         for (int tok = 0; tok < n_run; ++tok) {
-            const int t = t0 + tok, i_t = at_s[tok];
-            float* tail = n_tail > 0 ? a.tail + (size_t)state_s[tok] * a.tail_stride : nullptr;
+            const int t = t0 + tok, i_t = R.at[tok];
+            float* tail = n_tail > 0 ? a.tail + (size_t)R.state[tok] * a.tail_stride : nullptr;
             float ss = 0.f;
             for (int c = lane * V; c < width; c += 32 * V) {
                 const int ch = ch0 + c;
@@ -293,7 +315,7 @@ head_conv_rope_kernel(const HeadConvArgs a, T* __restrict__ q_out, T* __restrict
             if (kind == 0) {
                 dst = q_out + (size_t)t * a.q_width + (size_t)unit * a.hd;
             } else {
-                const int slot = slot_s[tok];
+                const int slot = R.slot[tok];
                 if (slot < 0) continue;                          // (the same for the whole warp)
                 const int page = slot / a.block_size, off = slot - page * a.block_size;
                 dst = (kind == 1 ? k_pool : v_pool) +
@@ -324,11 +346,154 @@ head_conv_rope_kernel(const HeadConvArgs a, T* __restrict__ q_out, T* __restrict
             __syncwarp();                                        // the stage is filled again
         }
     }
-    if (a.writes && blockIdx.y == 0)
-        for (int tok = 0; tok < n_run; ++tok)
-            if (slot_s[tok] >= 0)
-                clear_page_tail<T>(rest_s[tok], slot_s[tok], a.block_size, a.n_pages, a.n_kv, a.hd,
-                                   k_pool, v_pool);
+    clear_run_tails<T>(a, n_run, R, k_pool, v_pool);
+}
+
+// The same with a lane's entries in registers: a lane takes V entries and the V that turn with
+// them (past the rotated ones: the V behind them), so a map or value head of up to 64 V entries
+// needs at most a warp, a smaller one a power of two of lanes, and a warp works on as many tokens
+// of the run at a time as fit it.  TAPS: 0, or the most taps (weights, biases and norm weights are
+// then read once a run).
+template <typename T, int V, int TAPS>
+__global__ void __launch_bounds__(HC_WARPS * 32, V == 4 ? 2 : 3)
+head_conv_rope_lanes_kernel(const HeadConvArgs a, T* __restrict__ q_out, T* __restrict__ k_pool,
+                            T* __restrict__ v_pool) {
+    chain_release();
+    extern __shared__ __align__(16) float hc_smem[];
+    __shared__ RunTokens R;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int t0 = blockIdx.x * a.run, n_run = min(a.run, a.n_tokens - t0);
+    const int half = a.rot / 2;
+    float* angles = hc_smem;
+    look_up_run(a, t0, n_run, R, angles);
+    const int nq = a.n_heads * a.maps, nk = a.n_kv * a.maps;
+    const int units = nq + (a.writes ? nk + a.n_kv : 0);
+    const int channels = (nq + nk) * a.e + a.n_kv * a.f, n_tail = a.taps - 1;
+    const int u = blockIdx.y * HC_WARPS + warp;
+    const bool there = u < units;
+    const int kind = u < nq ? 0 : (u < nq + nk ? 1 : 2);
+    const int unit = kind == 0 ? u : (kind == 1 ? u - nq : u - nq - nk);
+    const int width = kind == 2 ? a.f : a.e;
+    const int ch0 = kind == 2 ? (nq + nk) * a.e + unit * a.f : u * a.e;
+    const float* w = kind == 0 ? a.w_q : kind == 1 ? a.w_k : nullptr;
+    const int head = kind == 2 ? unit : unit / a.maps, map = kind == 2 ? 0 : unit % a.maps;
+    const int inside = map * a.e, rot = kind == 2 ? 0 : a.rot;
+    const int turning = rot / (2 * V);                           // lanes whose entries turn
+    const int items = turning + ((width - rot) / V + 1) / 2;
+    int lanes = 1;
+    while (lanes < items) lanes <<= 1;                           // (at most 32: the host's choice)
+    const int at_once = 32 / lanes, mine = lane & (lanes - 1), group = lane / lanes;
+    const bool turns = mine < turning;
+    const int ca = turns ? mine * V : rot + (mine - turning) * 2 * V;      // this lane's entries
+    const int cb = turns ? ca + half : ca + V;
+    const bool has_a = there && mine < items, has_b = has_a && cb < width;
+    // the rest of the row that this warp fills with zeros
+    const int z_lo = kind == 2 ? width : (kind == 1 ? (map + 1 < a.maps ? a.hd : a.maps * a.e) : 0);
+
+    Pack<V> bias[2], cw[2][TAPS > 0 ? TAPS : 1], wv[2];
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+        const int c = x ? cb : ca;
+        const bool has = x ? has_b : has_a;
+#pragma unroll
+        for (int k = 0; k < V; ++k) {
+            bias[x].v[k] = 0.f;
+            wv[x].v[k] = 1.f;
+        }
+        if (has && a.bias) bias[x] = load_floats<V>(a.bias + ch0 + c);
+        if (has && w) wv[x] = load_floats<V>(w + c);
+        if constexpr (TAPS > 0) {
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j)
+                if (has && j < a.taps)
+                    cw[x][j] = load_floats<V>(a.conv + (size_t)j * channels + ch0 + c);
+        }
+    }
+    chain_wait();
+    for (int tok0 = 0; tok0 < n_run; tok0 += at_once) {
+        const int tok = tok0 + group, t = t0 + tok;
+        const bool live = tok < n_run;
+        Pack<V> y[2];
+        float ss = 0.f;
+        const int i_t = live ? R.at[tok] : 0;
+        float* tail = (live && n_tail > 0) ? a.tail + (size_t)R.state[tok] * a.tail_stride : nullptr;
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+#pragma unroll
+            for (int k = 0; k < V; ++k) y[x].v[k] = 0.f;
+            if (!live || !(x ? has_b : has_a)) continue;
+            const int ch = ch0 + (x ? cb : ca);
+            const float* src = a.proj + (size_t)t * a.proj_width + a.col + ch;
+            if constexpr (TAPS == 0) {
+                y[x] = load_floats<V>(src);
+#pragma unroll
+                for (int k = 0; k < V; ++k) y[x].v[k] += bias[x].v[k];
+            } else {
+                Pack<V> in[TAPS];
+#pragma unroll
+                for (int j = 0; j < TAPS; ++j) {
+                    const int back = n_tail - j;                 // tokens before this one
+                    if (j < a.taps)
+                        in[j] = back <= i_t
+                            ? load_floats<V>(src - (size_t)back * a.proj_width)
+                            : load_floats<V>(tail + (size_t)(n_tail + i_t - back) * channels + ch);
+                }
+#pragma unroll
+                for (int j = 0; j < TAPS; ++j) {
+                    if (j < a.taps) {
+                        if (n_tail - j <= i_t) {
+#pragma unroll
+                            for (int k = 0; k < V; ++k) in[j].v[k] += bias[x].v[k];
+                        }
+#pragma unroll
+                        for (int k = 0; k < V; ++k)
+                            y[x].v[k] = fmaf(cw[x][j].v[k], in[j].v[k], y[x].v[k]);
+                        if (a.move_tail && j >= 1)
+                            store_floats<V>(tail + (size_t)(j - 1) * channels + ch, in[j]);
+                    }
+                }
+            }
+#pragma unroll
+            for (int k = 0; k < V; ++k) ss = fmaf(y[x].v[k], y[x].v[k], ss);
+        }
+        if (w) {
+            for (int o = lanes >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+            const float inv = 1.0f / sqrtf(ss / (float)width + a.eps);
+#pragma unroll
+            for (int x = 0; x < 2; ++x)
+#pragma unroll
+                for (int k = 0; k < V; ++k) y[x].v[k] = y[x].v[k] * inv * wv[x].v[k];
+        }
+        if (!live || !there) continue;
+        if (turns) {
+            const Pack<V> c = load_floats<V>(angles + tok * a.rot + ca);
+            const Pack<V> s = load_floats<V>(angles + tok * a.rot + half + ca);
+#pragma unroll
+            for (int k = 0; k < V; ++k) {
+                const float p = y[0].v[k], q = y[1].v[k];
+                y[0].v[k] = __fsub_rn(__fmul_rn(p, c.v[k]), __fmul_rn(q, s.v[k]));
+                y[1].v[k] = __fadd_rn(__fmul_rn(q, c.v[k]), __fmul_rn(p, s.v[k]));
+            }
+        }
+        T* dst;
+        if (kind == 0) {
+            dst = q_out + (size_t)t * a.q_width + (size_t)unit * a.hd;
+        } else {
+            const int slot = R.slot[tok];
+            if (slot < 0) continue;
+            const int page = slot / a.block_size, off = slot - page * a.block_size;
+            dst = (kind == 1 ? k_pool : v_pool) +
+                  (((size_t)head * a.n_pages + page) * a.block_size + off) * a.hd;
+        }
+        if (has_a) store_elems<V>(dst + inside + ca, y[0]);
+        if (has_b) store_elems<V>(dst + inside + cb, y[1]);
+        Pack<V> zero;
+#pragma unroll
+        for (int k = 0; k < V; ++k) zero.v[k] = 0.f;
+        for (int z = z_lo + mine * V; z < a.hd; z += lanes * V)
+            if (kind != 0 || z < inside || z >= inside + a.e) store_elems<V>(dst + z, zero);
+    }
+    clear_run_tails<T>(a, n_run, R, k_pool, v_pool);
 }
 
 // o [T, 2 H * hd]: head h's two maps at rows 2h and 2h + 1; out [T, H * f].
@@ -441,24 +606,35 @@ MLS_API int mls_head_conv_rope_store(
         return e % v == 0 && f % v == 0 && proj_width % v == 0 && col % v == 0 && q_width % v == 0 &&
                bits % (4 * v) == 0 && (taps <= 1 || tail_stride % v == 0);
     };
-    const int v = (widest > 64 && takes(4)) ? 4 : (widest > 32 && takes(2)) ? 2 : 1;
+    // with the entries in registers where a map (a value head) fits a warp and the taps their array
+    int v = takes(4) && rot % 8 == 0 ? 4 : takes(2) && rot % 4 == 0 ? 2 : 1;
+    auto items = [&](int width, int turned) { return turned / (2 * v) + ((width - turned) / v + 1) / 2; };
+    const bool lanes = taps <= 4 && items(e, rot) <= 32 && items(f, 0) <= 32;
+    if (!lanes) v = (widest > 64 && takes(4)) ? 4 : (widest > 32 && takes(2)) ? 2 : 1;
     const size_t smem = ((((size_t)a.run * rot + 3) & ~(size_t)3) +
-                         (size_t)HC_WARPS * ((widest + 3) & ~3)) * sizeof(float);
+                         (lanes ? 0 : (size_t)HC_WARPS * ((widest + 3) & ~3))) * sizeof(float);
     if (smem > 48 * 1024) return MLS_ERR_UNSUPPORTED;
     const dim3 grid((n_tokens + a.run - 1) / a.run, grid_y);
-#define HC_GO(T, V)                                                                              \
-    MLS_LAUNCH((head_conv_rope_kernel<T, V>), grid, dim3(HC_WARPS * 32), smem, stream, a,         \
-               (T*)q_out, (T*)k_pool, (T*)v_pool)
-    if (dtype == MLS_BF16) {
-        if (v == 4) HC_GO(__nv_bfloat16, 4);
-        else if (v == 2) HC_GO(__nv_bfloat16, 2);
-        else HC_GO(__nv_bfloat16, 1);
-    } else {
-        if (v == 4) HC_GO(float, 4);
-        else if (v == 2) HC_GO(float, 2);
-        else HC_GO(float, 1);
-    }
+#define HC_RUN_KERNEL(K)                                                                          \
+    MLS_LAUNCH(K, grid, dim3(HC_WARPS * 32), smem, stream, a, (E*)q_out, (E*)k_pool, (E*)v_pool)
+#define HC_GO(V)                                                                                  \
+    do {                                                                                          \
+        if (!lanes) HC_RUN_KERNEL((head_conv_rope_kernel<E, V>));                                 \
+        else if (taps > 0) HC_RUN_KERNEL((head_conv_rope_lanes_kernel<E, V, 4>));                 \
+        else HC_RUN_KERNEL((head_conv_rope_lanes_kernel<E, V, 0>));                               \
+    } while (0)
+#define HC_TYPE(TYPE)                                                                             \
+    do {                                                                                          \
+        using E = TYPE;                                                                           \
+        if (v == 4) HC_GO(4);                                                                     \
+        else if (v == 2) HC_GO(2);                                                                \
+        else HC_GO(1);                                                                            \
+    } while (0)
+    if (dtype == MLS_BF16) HC_TYPE(__nv_bfloat16);
+    else HC_TYPE(float);
+#undef HC_TYPE
 #undef HC_GO
+#undef HC_RUN_KERNEL
     return launch_status();
 }
 

@@ -64,6 +64,12 @@ class BatchBuilder:
         self._dev = None
         self.generation = 0           # grows when the device buffer moves
         self.last_bytes = 0           # bytes of the last step's host-to-device copy
+        self.width = min(cache.max_blocks, self.LEAST_WIDTH)      # of the block tables sent
+
+    # Entries of a block-table row that are sent at least.  A model whose sequences have no bound
+    # of their own has tables of nominal length; a step sends the part that its longest request
+    # reaches, doubled as contexts grow (so the layout of a step seldom changes).
+    LEAST_WIDTH = 2048
 
     def _staging(self, n: int):
         use_cuda = self.device.type == "cuda"
@@ -116,7 +122,9 @@ class BatchBuilder:
             rows.append(cache.row(e.owner))
         t_total, r_total = sum(q_lens), len(entries)
         n_out = sum(len(e.want) for e in entries)
-        groups = cache.step_arrays([(e.owner, len(e.tokens)) for e in entries])
+        while self.width < cache.max_blocks and self.width < cache.pages_for(max(ctx_lens)):
+            self.width = min(cache.max_blocks, 2 * self.width)
+        groups = cache.step_arrays([(e.owner, len(e.tokens)) for e in entries], self.width)
 
         # layout of the packed buffer (int32 elements)
         off = {}

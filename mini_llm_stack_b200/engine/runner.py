@@ -21,6 +21,7 @@ import torch
 from ..cache.manager import CacheError, CacheManager
 from ..config.registry import build_model, config_from_folder
 from ..ops.kernels import Runtime
+from ..parts.base import PagedKV
 from ..weights.loader import device_dtype, load_tensors, open_weights
 from ..weights.random_init import random_tensors
 from .batch import BatchBuilder
@@ -121,10 +122,10 @@ class ModelRunner:
         specs = model.cache_specs()
         # a request whose every token keeps a page can never be longer than the pool; a model
         # without positions of its own would otherwise ask for block tables of its nominal
-        # length (pages a window gives back let a request outgrow the pool)
+        # length (pages a window or a chunk gives back let a request outgrow the pool)
         max_len = cfg.max_seq_len
-        paged = [s for s in specs if hasattr(s, "window")]
-        if paged and all(s.window is None for s in paged):
+        paged = [s for s in (getattr(s, "paged", s) for s in specs) if isinstance(s, PagedKV)]
+        if any(s.span is None for s in paged):
             max_len = min(max_len, num_blocks * block_size)
         self.max_seq_len = max_len
         self.cache = CacheManager(
@@ -200,8 +201,8 @@ class ModelRunner:
         """A step replayed from a CUDA graph.
 
         A step launches the same kernels with the same arguments whenever the requests'
-        token counts, the number of wanted rows and what the parts add to the key (the
-        attention's cut of the context) are the same; only the arrays the batch builder
+        token counts, the number of wanted rows, the block tables' widths and what the parts add
+        to the key (the attention's cut of the context) are the same; only the arrays the batch builder
         has just copied to the device differ, and they lie at the same addresses.  The
         first step of a kind runs eagerly (which sizes every buffer), the second is
         captured, later ones replay.  A step with portions of prompts, whose shape may
@@ -217,7 +218,8 @@ class ModelRunner:
             self._graphs = {"moved": moved}      # a buffer moved: the old graphs are stale
         decoding = ctx.max_q_len == 1
         shape = ctx.n_requests if decoding else tuple(ctx.q_lens)
-        key = (shape, ctx.n_out, self.model.decode_graph_key(ctx))
+        widths = tuple(g.max_blocks for g in ctx.groups.values())
+        key = (shape, ctx.n_out, widths, self.model.decode_graph_key(ctx))
         entry = self._graphs.pop(key, None)      # taken out and put back: the dict's order is by use
         if not isinstance(entry, tuple):
             seen = entry or _Seen()

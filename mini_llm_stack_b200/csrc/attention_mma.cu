@@ -51,6 +51,8 @@ struct Params {
     int max_blocks, n_req, n_tokens, n_heads, n_kv, group, block_size, window, n_split;
     int chunk;                           // > 0 (and no window): a query sees its own chunk of so many
                                          // tokens, counted from the sequence's start
+    int share;                           // CTAs of the split kernel that share a kv head's group of
+                                         // query heads (its `group` is then a share of it)
     int small_only;                      // tile kernel: 1 = skip requests the split kernel takes
     int cluster_merge;                   // split TMA kernel: the splits of a request and kv head are
                                          // one cluster and merge through shared memory
@@ -165,7 +167,7 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
 }
 
 // A request goes to the split kernel when all its (token, head) rows of one kv
-// head fit one 16-row tile.
+// head, or of one share of its query heads, fit one 16-row tile.
 __device__ __forceinline__ bool is_small(int q_len, int group) { return q_len * group <= 16; }
 
 // Key tiles a context split holds: the most tiles a small request of this step can have,
@@ -240,7 +242,7 @@ __global__ void __launch_bounds__(NT) attention_tile_kernel(const Params P) {
     for (; r < P.n_req; ++r) {
         q_len = P.cu_q[r + 1] - P.cu_q[r];
         rows = q_len * P.group;
-        int tiles = (P.small_only && is_small(q_len, P.group)) ? 0 : (rows + 63) / 64;
+        int tiles = (P.small_only && is_small(q_len, P.group / P.share)) ? 0 : (rows + 63) / 64;
         if (tile < tiles) break;
         tile -= tiles;
     }
@@ -446,7 +448,7 @@ __global__ void __launch_bounds__(NT) attention_split_kernel(const Params P) {
 #pragma unroll
         for (int st = 0; st < STAGES - 1; ++st) {
             if (st < n_tiles)
-                load_kv_tile(kbuf + st * TILE_BYTES, vbuf + st * TILE_BYTES, P, table, kvh,
+                load_kv_tile(kbuf + st * TILE_BYTES, vbuf + st * TILE_BYTES, P, table, kvh / P.share,
                              tile_base(R, t_begin + st, BN), lo, hi);
             cp_async_commit();
         }
@@ -464,7 +466,7 @@ __global__ void __launch_bounds__(NT) attention_split_kernel(const Params P) {
             const int nt = t + STAGES - 1;
             if (nt < n_tiles)
                 load_kv_tile(kbuf + (nt % STAGES) * TILE_BYTES, vbuf + (nt % STAGES) * TILE_BYTES,
-                             P, table, kvh, tile_base(R, t_begin + nt, BN), lo, hi);
+                             P, table, kvh / P.share, tile_base(R, t_begin + nt, BN), lo, hi);
             cp_async_commit();
         }
         const int kbase = tile_base(R, t_begin + t, BN) + warp * 16;   // this warp's 16 keys
@@ -818,10 +820,10 @@ attention_split_tma_kernel(const Params P, const Fused F,
         const int kb_first = kbase0 + t_begin * BN;
         const int old_tiles = max(0, (pos0 - kb_first) / BN);
         const int ahead = min(min(n_tiles, TSTAGES), old_tiles);
-        produce_tiles(P, &kmap, &vmap, &kmap_wide, &vmap_wide, table, kvh, kb_first, 0, ahead, lo,
+        produce_tiles(P, &kmap, &vmap, &kmap_wide, &vmap_wide, table, kvh / P.share, kb_first, 0, ahead, lo,
                       hi, base, bar0, /*late_slot=*/-1);
         chain_wait();
-        produce_tiles(P, &kmap, &vmap, &kmap_wide, &vmap_wide, table, kvh, kb_first, ahead,
+        produce_tiles(P, &kmap, &vmap, &kmap_wide, &vmap_wide, table, kvh / P.share, kb_first, ahead,
                       n_tiles, lo, hi, base, bar0, /*late_slot=*/-1);
         if (P.cluster_merge) {           // every thread of the cluster meets at its two barriers
             cluster_sync_all();
@@ -1199,7 +1201,7 @@ attention_tile_tma_kernel(const Params P, const __grid_constant__ CUtensorMap km
     for (; r < P.n_req; ++r) {
         q_len = P.cu_q[r + 1] - P.cu_q[r];
         rows = q_len * P.group;
-        int tiles = (P.small_only && is_small(q_len, P.group)) ? 0 : (rows + 63) / 64;
+        int tiles = (P.small_only && is_small(q_len, P.group / P.share)) ? 0 : (rows + 63) / 64;
         if (tile < tiles) break;
         tile -= tiles;
     }
@@ -1448,9 +1450,9 @@ static int launch_split_tma(Params P, const Fused& F, const CUtensorMap& kmap,
         const char* v = getenv("MLS_B200_CLUSTER_MERGE");
         return !(v && v[0] == '0');
     }();
-    const dim3 grid(P.n_req, P.n_kv, P.n_split);
+    const dim3 grid(P.n_req, P.n_kv * P.share, P.n_split);
     P.cluster_merge = (allowed && P.n_split >= 2 && P.n_split <= MAX_CLUSTER &&
-                       (long long)P.n_req * P.n_kv * P.n_split <= 2LL * sm_count()) ? 1 : 0;
+                       (long long)P.n_req * P.n_kv * P.share * P.n_split <= 2LL * sm_count()) ? 1 : 0;
     if (P.cluster_merge) {
         const int rc = launch_chained_cluster(attention_split_tma_kernel, grid, dim3(TMA_THREADS),
                                               TMA_SMEM, stream, dim3(1, 1, P.n_split), P, F, kmap,
@@ -1476,6 +1478,8 @@ constexpr int SPLIT_SMEM = SPLIT_SMEM_PIPE > SPLIT_SMEM_MERGE ? SPLIT_SMEM_PIPE 
 // many tokens, counted from the sequence's start, up to itself.
 // softcap c > 0: scores become c * tanh(score / c) before the softmax.  sink (float32 [H] or
 // nullptr): exp(sink_h) joins the denominator of head h's softmax.
+// share: so many CTAs of the split kernel divide a kv head's query heads among them (groups of more
+// than 16), each reading the same keys and values.
 // n_tiles: 64-row tiles the tile kernel has to run (0: none); n_small: 1 if any
 // request goes to the split kernel.  part_o / part_lse are scratch memory of
 // n_split * T * H * (HD + 1) floats, needed when n_split > 1.
@@ -1486,9 +1490,9 @@ MLS_API int mls_attention_mma(const void* qkv, void* out, const void* k_pool, co
                               int n_small, int n_split, float* part_o, float* part_lse,
                               long long pool_pages, int* status, int use_tma,
                               const float* sink, const float* slopes, int keep_first,
-                              long long out_stride, int chunk, cudaStream_t stream) {
+                              long long out_stride, int chunk, int share, cudaStream_t stream) {
     if (n_tokens <= 0 || n_req <= 0) return 0;
-    if (n_heads % n_kv || n_split < 1 || n_split > MAX_SPLITS ||
+    if (n_heads % n_kv || share < 1 || (n_heads / n_kv) % share || n_split < 1 || n_split > MAX_SPLITS ||
         (n_split > 1 && (!part_o || !part_lse)))
         return MLS_ERR_UNSUPPORTED;
     if (out_stride <= 0) out_stride = (long long)n_heads * HD;
@@ -1526,6 +1530,7 @@ MLS_API int mls_attention_mma(const void* qkv, void* out, const void* k_pool, co
     P.window = window;
     P.chunk = window > 0 ? 0 : chunk;
     P.n_split = n_split;
+    P.share = share;
     P.small_only = n_small ? 1 : 0;
     P.cluster_merge = 0;
     P.scale_log2 = scale * LOG2E;
@@ -1574,11 +1579,13 @@ MLS_API int mls_attention_mma(const void* qkv, void* out, const void* k_pool, co
         if (rc) return rc;
     }
     if (n_small) {
+        // the split kernel's view: a share of a group each CTA, that many CTAs a kv head
+        P.group /= share;
 #if MLS_HEAD_DIM % 64 == 0
         if (tma_ok)
             return launch_split_tma(P, Fused{}, kmap, vmap, kmap_wide, vmap_wide, n_tokens, stream);
 #endif
-        MLS_LAUNCH((attention_split_kernel), dim3(n_req, n_kv, n_split), dim3(NT), SPLIT_SMEM,
+        MLS_LAUNCH((attention_split_kernel), dim3(n_req, n_kv * share, n_split), dim3(NT), SPLIT_SMEM,
                    stream, P);
         int rc = launch_status();
         if (rc) return rc;
@@ -1649,6 +1656,7 @@ MLS_API int mls_attention_decode_fused(const float* parts, int n_parts, long lon
     P.window = window;
     P.chunk = 0;
     P.n_split = n_split;
+    P.share = 1;
     P.small_only = 1;
     P.cluster_merge = 0;
     P.scale_log2 = scale * LOG2E;

@@ -71,6 +71,8 @@ struct Params {
     const int* cu_q;
     const int* ctx_len;
     int max_blocks, n_req, n_heads, n_kv, group, block_size, window, small_only;
+    int share;                           // of a group of query heads, the split kernel's CTAs take
+                                         // one part in so many each (which decides what is small)
     int chunk;                           // > 0 (and no window): a query sees its own chunk of so many
                                          // tokens, counted from the sequence's start
     int two_tiles;                       // 1: a CTA owns two row tiles; 0: one, its keys in halves
@@ -133,7 +135,7 @@ attention_tc_kernel(const Params P, const __grid_constant__ CUtensorMap kmap,
     for (; r < P.n_req; ++r) {
         q_len = P.cu_q[r + 1] - P.cu_q[r];
         rows = q_len * P.group;
-        int tiles = (P.small_only && is_small(q_len, P.group)) ? 0 : (rows + tile_rows - 1) / tile_rows;
+        int tiles = (P.small_only && is_small(q_len, P.group / P.share)) ? 0 : (rows + tile_rows - 1) / tile_rows;
         if (tile < tiles) break;
         tile -= tiles;
     }
@@ -615,10 +617,10 @@ MLS_API int mls_attention_tc(const void* qkv, void* out, const void* k_pool, con
                              float scale, int window, float softcap, int n_tiles, int n_tiles_wide,
                              int skip_small, long long pool_pages, int* status,
                              const float* sink, long long out_stride, const float* slopes,
-                             int keep_first, int chunk, cudaStream_t stream) {
+                             int keep_first, int chunk, int share, cudaStream_t stream) {
 #if MLS_HEAD_DIM == 64 || MLS_HEAD_DIM == 128
     if (n_tiles <= 0 || n_req <= 0) return 0;
-    if (n_heads % n_kv) return MLS_ERR_UNSUPPORTED;
+    if (n_heads % n_kv || share < 1) return MLS_ERR_UNSUPPORTED;
     if (!(block_size == 8 || block_size == 16 || block_size == 32 || block_size == 64))
         return MLS_ERR_UNSUPPORTED;
     static bool configured = false;
@@ -650,6 +652,7 @@ MLS_API int mls_attention_tc(const void* qkv, void* out, const void* k_pool, con
     P.block_size = block_size;
     P.window = window;
     P.chunk = window > 0 ? 0 : chunk;
+    P.share = share;
     P.small_only = skip_small ? 1 : 0;
     P.two_tiles = (n_tiles_wide > 0 && (long long)n_tiles_wide * n_kv >= sm_count()) ? 1 : 0;
     if (g_forced_rows == CHAIN_ROWS) P.two_tiles = 0;

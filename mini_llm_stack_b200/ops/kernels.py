@@ -529,10 +529,10 @@ class Ops:
             lib = self._load("attention", {"MLS_HEAD_DIM": int(hd)})
             fn = _decl(lib, "mls_attention_mma",
                        [_P, _P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _F, _I, _I, _I,
-                        _P, _P, _LL, _P, _I, _P, _P, _I, _LL, _I, _P])
+                        _P, _P, _LL, _P, _I, _P, _P, _I, _LL, _I, _I, _P])
             tc = _decl(lib, "mls_attention_tc",
                        [_P, _P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _F, _I, _F, _I, _I, _I, _LL,
-                        _P, _P, _LL, _P, _I, _I, _P])
+                        _P, _P, _LL, _P, _I, _I, _I, _P])
             fused = _decl(lib, "mls_attention_decode_fused",
                           [_P, _I, _LL, _P, _P, _P, _I, _P, _I, _P, _P, _P, _P, _I, _P, _P, _I, _I,
                            _I, _I, _F, _I, _I, _P, _P, _LL, _P, _P])
@@ -598,7 +598,8 @@ class Ops:
         ``c * tanh(score / c)`` before the softmax.  ``sink`` (float32 [n_heads]): the softmax's
         denominator of head h also holds ``exp(sink[h])``, a term without key or value.  ``plan`` (the mixer's, from
         ``attention_facts``): ``n_tiles`` / ``n_tiles_tc`` / ``n_tiles_tc_wide`` tiles of the
-        requests that are not small, ``any_small``, ``n_split`` context splits for the small ones."""
+        requests that are not small, ``any_small``, ``n_split`` context splits for the small ones,
+        ``share`` CTAs that divide a kv head's query heads among them."""
         g = step.groups[cache.group]
         t = step.n_tokens
         _need(out.shape == (t, n_heads * hd) and out.stride(1) == 1, "attention: bad out")
@@ -630,7 +631,7 @@ class Ops:
                           step.n_requests, n_heads, n_kv, g.block_size, float(scale), int(window),
                           float(softcap), n_tiles_tc, plan.n_tiles_tc_wide, n_small, cache.k_pool.shape[1],
                           _ptr(self.status), _ptr(sink), out.stride(0), _ptr(slopes), keep_first,
-                          int(chunk), self._stream()), "attention_tc")
+                          int(chunk), plan.share, self._stream()), "attention_tc")
                 n_tiles = 0
                 if not n_small:
                     return
@@ -643,14 +644,14 @@ class Ops:
             tma = (self.attention_impl != "no_tma" and plain and hd % 64 == 0
                    and g.block_size in (8, 16, 32, 64))
             self.launches += (1 if n_tiles else 0) + (n_small and self._split_launches(
-                n_split, tma, step.n_requests * n_kv * n_split))
+                n_split, tma, step.n_requests * n_kv * plan.share * n_split))
             _check(fn(_ptr(qkv), _ptr(out), _ptr(cache.k_pool), _ptr(cache.v_pool),
                       _ptr(g.block_table), g.max_blocks, _ptr(step.cu_q), _ptr(step.ctx_len),
                       step.n_requests, t, n_heads, n_kv, g.block_size, float(scale), int(window),
                       float(softcap), n_tiles, n_small, n_split, _ptr(part_o), _ptr(part_lse),
                       cache.k_pool.shape[1], _ptr(self.status),
                       0 if (self.attention_impl == "no_tma" or not plain) else 1, _ptr(sink),
-                      _ptr(slopes), keep_first, out.stride(0), int(chunk), self._stream()),
+                      _ptr(slopes), keep_first, out.stride(0), int(chunk), plan.share, self._stream()),
                    "attention_mma")
             return
         self.launches += 1

@@ -30,6 +30,7 @@ class AttentionPlan:
     n_tiles_tc_wide: int  # tiles of twice as many rows: the kernel takes these when they fill the SMs
     any_small: bool       # some request has so few rows that the context-split kernel takes it
     n_split: int          # parts the context of the small requests is cut into
+    share: int = 1        # CTAs that divide a kv head's query heads of a small request among them
 
 
 def context_splits(tiles: list, n_kv: int, slots: int = 296, cluster_splits: int = 0,
@@ -68,22 +69,26 @@ def context_splits(tiles: list, n_kv: int, slots: int = 296, cluster_splits: int
 
 
 def plan_paged_attention(step: StepContext, facts: dict, n_heads: int, n_kv_heads: int,
-                         head_dim: int, span=None):
+                         head_dim: int, span=None, share_groups: bool = False):
     """A step's ``AttentionPlan`` for heads of this shape (None where the kernel in use
     needs none), shared through ``step.attn_tiles`` by the mixers of the same shape.
 
     Requests whose (token, head) rows of one kv head fit ``small_rows`` go to the
     context-split kernel, their context cut so that all SMs have work; the others
     are cut into tiles of rows.  ``span``: a token reads at most so many keys (a window or a
-    chunk): the cut is planned for the tiles there are."""
+    chunk): the cut is planned for the tiles there are.  ``share_groups``: a group of more query
+    heads than ``small_rows`` is divided among up to four CTAs that read the same keys, so that its
+    decoded tokens are small requests too."""
     f = facts
     if not f["tensor_cores"]:
         return None
     group = n_heads // n_kv_heads
-    key = ("gqa", group, n_kv_heads, head_dim, span)
+    key = ("gqa", group, n_kv_heads, head_dim, span, share_groups)
     plan = step.attn_tiles.get(key)
     if plan is None:
-        small = [q * group <= f["small_rows"] for q in step.q_lens]
+        share = next((s for s in (1, 2, 3, 4) if group % s == 0 and group // s <= f["small_rows"]),
+                     1) if share_groups else 1
+        small = [q * (group // share) <= f["small_rows"] for q in step.q_lens]
         big = [q * group for q, s in zip(step.q_lens, small) if not s]
         n_small = sum(small)
         n_split = 1
@@ -91,7 +96,7 @@ def plan_paged_attention(step: StepContext, facts: dict, n_heads: int, n_kv_head
             keys = f.get("split_keys", 64)
             most = (span + 15 + keys - 2) // keys + 1 if span else 1 << 30
             tiles = [min(most, -(-c // keys)) for c, s in zip(step.ctx_lens, small) if s]
-            n_split = context_splits(tiles, n_kv_heads, f["split_slots"],
+            n_split = context_splits(tiles, n_kv_heads * share, f["split_slots"],
                                      f.get("cluster_splits", 0),
                                      longest=min(most, -(-step.max_ctx_len // keys)),
                                      cluster_slots=f.get("cluster_slots", 0))
@@ -99,7 +104,7 @@ def plan_paged_attention(step: StepContext, facts: dict, n_heads: int, n_kv_head
             n_tiles=sum(-(-r // f["tile_rows"]) for r in big),
             n_tiles_tc=sum(-(-r // f["tc_rows"]) for r in big),
             n_tiles_tc_wide=sum(-(-r // (2 * f["tc_rows"])) for r in big),
-            any_small=n_small > 0, n_split=n_split)
+            any_small=n_small > 0, n_split=n_split, share=share)
         step.attn_tiles[key] = plan
     return plan
 
@@ -510,7 +515,7 @@ class RotatedAttention(Mixer):
         if not self._tensor_cores:
             return None
         return plan_paged_attention(step, self._facts, self.q_heads, self.n_kv_heads, self.pad_dim,
-                                    span=self.window or self.chunk)
+                                    span=self.window or self.chunk, share_groups=True)
 
     def decode_graph_key(self, step: StepContext) -> tuple:
         plan = self.plan(step)

@@ -394,7 +394,8 @@ class SpanAttention:
         if ops.attention_tensor_cores(self.hd):
             ops.require_attention(self.hd)
         plan = plan_paged_attention(step, ops.attention_facts(self.hd), self.heads, self.kv, self.hd,
-                                    span=self.spec.span)
+                                    span=self.spec.span, share_groups=True)
+        assert plan is None or plan.share == (1 if self.heads // self.kv <= 16 else 2)
         ops.paged_attention(qkv, out, handle, step, self.heads, self.kv, self.hd, self.hd ** -0.5,
                             self.window or 0, plan=plan, chunk=self.chunk or 0,
                             sink=self.sink.cuda() if self.sink is not None else None)
@@ -469,7 +470,8 @@ def test_chunked_attention_in_float32(rts, chunk, ctxs, q_lens):
 @pytest.mark.parametrize("span", [dict(chunk=700), dict(chunk=2000), dict(window=700)])
 def test_chunks_cut_into_forced_splits(rts, monkeypatch, splits, span):
     monkeypatch.setenv("MLS_B200_SPLITS", str(splits))
-    for hd, heads, kv, sink in ((64, 8, 2, True), (128, 32, 8, False), (32, 6, 3, True)):
+    for hd, heads, kv, sink in ((64, 8, 2, True), (128, 32, 8, False), (32, 6, 3, True),
+                                (128, 64, 2, True), (64, 24, 1, False), (48, 40, 2, True)):
         SpanAttention(rts[torch.bfloat16], heads, kv, hd, 16, [3000, 70, 1025, 1, 1399, 2001],
                       [1, 1, 1, 1, 2, 1], seed=31, sink=sink, **span).check((hd, splits))
 

@@ -185,6 +185,11 @@ __device__ __forceinline__ int tiles_per_split(const int* ctx_len, int n_req, in
     return (max(most, 1) + n_split - 1) / n_split;
 }
 
+// The kv head whose keys and values the split kernel's CTA number kvh reads.
+__device__ __forceinline__ int pool_head(const Params& P, int kvh) {
+    return P.share == 1 ? kvh : kvh / P.share;
+}
+
 // Keys kbase .. kbase+63 of one kv head into shared memory; rows outside [lo, hi]
 // or on a released page are zero-filled, so nothing that is not a key of this
 // request can reach the products.
@@ -448,7 +453,7 @@ __global__ void __launch_bounds__(NT) attention_split_kernel(const Params P) {
 #pragma unroll
         for (int st = 0; st < STAGES - 1; ++st) {
             if (st < n_tiles)
-                load_kv_tile(kbuf + st * TILE_BYTES, vbuf + st * TILE_BYTES, P, table, kvh / P.share,
+                load_kv_tile(kbuf + st * TILE_BYTES, vbuf + st * TILE_BYTES, P, table, pool_head(P, kvh),
                              tile_base(R, t_begin + st, BN), lo, hi);
             cp_async_commit();
         }
@@ -466,7 +471,7 @@ __global__ void __launch_bounds__(NT) attention_split_kernel(const Params P) {
             const int nt = t + STAGES - 1;
             if (nt < n_tiles)
                 load_kv_tile(kbuf + (nt % STAGES) * TILE_BYTES, vbuf + (nt % STAGES) * TILE_BYTES,
-                             P, table, kvh / P.share, tile_base(R, t_begin + nt, BN), lo, hi);
+                             P, table, pool_head(P, kvh), tile_base(R, t_begin + nt, BN), lo, hi);
             cp_async_commit();
         }
         const int kbase = tile_base(R, t_begin + t, BN) + warp * 16;   // this warp's 16 keys
@@ -761,6 +766,9 @@ __device__ __forceinline__ void produce_tiles(const Params& P, const CUtensorMap
     }
 }
 
+// MORE: chunks, and groups of query heads shared among CTAs (an instantiation of its own, so that
+// the kernel of the models without them carries none of their arithmetic).
+template <bool MORE>
 __global__ void __launch_bounds__(TMA_THREADS)
 attention_split_tma_kernel(const Params P, const Fused F,
                            const __grid_constant__ CUtensorMap kmap,
@@ -791,12 +799,12 @@ attention_split_tma_kernel(const Params P, const Fused F,
     const int tok0 = P.cu_q[r], ctx = P.ctx_len[r];
     const int pos0 = ctx - q_len;
     const int hi = ctx - 1;
-    const int lo = max(0, first_visible(pos0, P.window, P.chunk));
+    const int lo = max(0, first_visible(pos0, P.window, MORE ? P.chunk : 0));
     const int* table = P.block_table + (size_t)r * P.max_blocks;
     const int kbase0 = (lo / BN) * BN;
     const int tiles_all = (hi - kbase0) / BN + 1;
     const int per = P.n_split == 1 ? tiles_all
-        : tiles_per_split(P.ctx_len, P.n_req, P.window > 0 ? P.window : P.chunk, BN, P.n_split);
+        : tiles_per_split(P.ctx_len, P.n_req, P.window > 0 ? P.window : (MORE ? P.chunk : 0), BN, P.n_split);
     const int t_begin = split * per, t_end = min(tiles_all, t_begin + per);
     const int n_tiles = max(0, t_end - t_begin);
     if (n_tiles == 0 && !P.cluster_merge) {           // a stretch past the request's end: the merge
@@ -820,10 +828,10 @@ attention_split_tma_kernel(const Params P, const Fused F,
         const int kb_first = kbase0 + t_begin * BN;
         const int old_tiles = max(0, (pos0 - kb_first) / BN);
         const int ahead = min(min(n_tiles, TSTAGES), old_tiles);
-        produce_tiles(P, &kmap, &vmap, &kmap_wide, &vmap_wide, table, kvh / P.share, kb_first, 0, ahead, lo,
+        produce_tiles(P, &kmap, &vmap, &kmap_wide, &vmap_wide, table, MORE ? pool_head(P, kvh) : kvh, kb_first, 0, ahead, lo,
                       hi, base, bar0, /*late_slot=*/-1);
         chain_wait();
-        produce_tiles(P, &kmap, &vmap, &kmap_wide, &vmap_wide, table, kvh / P.share, kb_first, ahead,
+        produce_tiles(P, &kmap, &vmap, &kmap_wide, &vmap_wide, table, MORE ? pool_head(P, kvh) : kvh, kb_first, ahead,
                       n_tiles, lo, hi, base, bar0, /*late_slot=*/-1);
         if (P.cluster_merge) {           // every thread of the cluster meets at its two barriers
             cluster_sync_all();
@@ -863,8 +871,8 @@ attention_split_tma_kernel(const Params P, const Fused F,
     const int rA = lane >> 2, rB = rA + 8;
     const int pA = rA < rows ? pos0 + rA / P.group : -1;
     const int pB = rB < rows ? pos0 + rB / P.group : -1;
-    const int loA = first_visible(pA, P.window, P.chunk);
-    const int loB = first_visible(pB, P.window, P.chunk);
+    const int loA = first_visible(pA, P.window, MORE ? P.chunk : 0);
+    const int loB = first_visible(pB, P.window, MORE ? P.chunk : 0);
 
     float o[HD / 8][4];
 #pragma unroll
@@ -1453,13 +1461,15 @@ static int launch_split_tma(Params P, const Fused& F, const CUtensorMap& kmap,
     const dim3 grid(P.n_req, P.n_kv * P.share, P.n_split);
     P.cluster_merge = (allowed && P.n_split >= 2 && P.n_split <= MAX_CLUSTER &&
                        (long long)P.n_req * P.n_kv * P.share * P.n_split <= 2LL * sm_count()) ? 1 : 0;
+    auto kernel = (P.chunk > 0 || P.share > 1) ? attention_split_tma_kernel<true>
+                                               : attention_split_tma_kernel<false>;
     if (P.cluster_merge) {
-        const int rc = launch_chained_cluster(attention_split_tma_kernel, grid, dim3(TMA_THREADS),
+        const int rc = launch_chained_cluster(kernel, grid, dim3(TMA_THREADS),
                                               TMA_SMEM, stream, dim3(1, 1, P.n_split), P, F, kmap,
                                               vmap, kmap_wide, vmap_wide);
         return rc ? rc : launch_status();
     }
-    MLS_LAUNCH((attention_split_tma_kernel), grid, dim3(TMA_THREADS), TMA_SMEM, stream, P, F, kmap,
+    MLS_LAUNCH(kernel, grid, dim3(TMA_THREADS), TMA_SMEM, stream, P, F, kmap,
                vmap, kmap_wide, vmap_wide);
     if (P.n_split > 1)
         MLS_LAUNCH((attention_merge_kernel), dim3(merge_tokens, P.n_heads),
@@ -1550,9 +1560,12 @@ MLS_API int mls_attention_mma(const void* qkv, void* out, const void* k_pool, co
     if (tma_ok) {
         static bool tma_configured = false;
         if (!tma_configured) {
-            cudaError_t e = cudaFuncSetAttribute(attention_split_tma_kernel,
+            cudaError_t e = cudaFuncSetAttribute(attention_split_tma_kernel<false>,
                                                  cudaFuncAttributeMaxDynamicSharedMemorySize,
                                                  TMA_SMEM);
+            if (e == cudaSuccess)
+                e = cudaFuncSetAttribute(attention_split_tma_kernel<true>,
+                                         cudaFuncAttributeMaxDynamicSharedMemorySize, TMA_SMEM);
             if (e == cudaSuccess)
                 e = cudaFuncSetAttribute(attention_tile_tma_kernel,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -1626,7 +1639,7 @@ MLS_API int mls_attention_decode_fused(const float* parts, int n_parts, long lon
         return MLS_ERR_UNSUPPORTED;
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attention_split_tma_kernel,
+        cudaError_t e = cudaFuncSetAttribute(attention_split_tma_kernel<false>,
                                              cudaFuncAttributeMaxDynamicSharedMemorySize, TMA_SMEM);
         if (e != cudaSuccess) return (int)e;
         configured = true;
@@ -1695,9 +1708,9 @@ MLS_API int mls_attention_split_ctas_per_sm(int use_tma) {
     int n = 0;
 #if MLS_HEAD_DIM % 64 == 0
     if (use_tma) {
-        if (cudaFuncSetAttribute(attention_split_tma_kernel,
+        if (cudaFuncSetAttribute(attention_split_tma_kernel<false>,
                                  cudaFuncAttributeMaxDynamicSharedMemorySize, TMA_SMEM) != cudaSuccess ||
-            cudaOccupancyMaxActiveBlocksPerMultiprocessor(&n, attention_split_tma_kernel, TMA_THREADS,
+            cudaOccupancyMaxActiveBlocksPerMultiprocessor(&n, attention_split_tma_kernel<false>, TMA_THREADS,
                                                           TMA_SMEM) != cudaSuccess)
             return 0;
         return n;

@@ -19,7 +19,8 @@
 // mls_expert_relu2: y[p, :] = relu(Wu[e] a)^2, experts without a gate.
 // mls_expert_down: per_slot[slot, :] = Wd[e] y[p, :] (times the weight with output
 //   scaling), float32.
-// mls_expert_combine: delta[t] = sum_j per_slot[t * top + j] + shared[t], j ascending; with a
+// mls_expert_combine: delta[t] = sum_j per_slot[t * top + j] + shared[t], j ascending (shared: a
+//   tensor, or the float32 K-parts of its product, shared_stride apart, added in their order); with a
 //   gate (float32, one number a token) the shared addend is multiplied by sigmoid(gate[t]).
 //
 // The products run with float32 accumulation over k ascending (bfloat16 rows of whole
@@ -519,6 +520,7 @@ static inline bool takes_mma(int dtype, const void* a, const void* w, int K) {
 template <typename T>
 __global__ void expert_combine_kernel(const float* __restrict__ per_slot, int top,
                                       const void* __restrict__ shared, int shared_dtype,
+                                      int shared_parts, size_t shared_stride,
                                       const int* __restrict__ idx, const float* __restrict__ weight,
                                       int n_real, const T* __restrict__ h,
                                       const float* __restrict__ gate, int gate_stride,
@@ -537,7 +539,9 @@ __global__ void expert_combine_kernel(const float* __restrict__ per_slot, int to
                 s += per_slot[(t * top + j) * d + c];
         }
         if (shared) {
-            const float v = load_as_float(shared, i, shared_dtype);
+            float v = load_as_float(shared, i, shared_dtype);
+#pragma unroll 4
+            for (int k = 1; k < shared_parts; ++k) v += ((const float*)shared)[i + k * shared_stride];
             s += gate ? v / (1.0f + expf(-gate[t * gate_stride])) : v;
         }
         Elem<T>::store(delta + i, s);
@@ -625,20 +629,24 @@ MLS_API int mls_expert_down(const void* y, const void* w_down, float* per_slot, 
 }
 
 MLS_API int mls_expert_combine(const float* per_slot, int top, const void* shared,
-                               int shared_dtype, const int* idx, const float* weight, int n_real,
+                               int shared_dtype, int shared_parts, long long shared_stride,
+                               const int* idx, const float* weight, int n_real,
                                const void* h, const float* gate, int gate_stride, void* delta,
                                int dtype, int n_tokens, int d, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
+    if (shared_parts > 1 && shared_dtype != MLS_F32) return MLS_ERR_UNSUPPORTED;
     const size_t n = (size_t)n_tokens * d;
     const size_t want = (n + 255) / 256;
     const int blocks = (int)(want < (size_t)(8 * sm_count()) ? want : 8 * sm_count());
     if (dtype == MLS_BF16)
         MLS_LAUNCH((expert_combine_kernel<__nv_bfloat16>), dim3(blocks), dim3(256), 0, stream,
-                   per_slot, top, shared, shared_dtype, idx, weight, n_real, (const __nv_bfloat16*)h,
+                   per_slot, top, shared, shared_dtype, shared_parts, (size_t)shared_stride, idx,
+                   weight, n_real, (const __nv_bfloat16*)h,
                    gate, gate_stride, (__nv_bfloat16*)delta, n, d);
     else
         MLS_LAUNCH((expert_combine_kernel<float>), dim3(blocks), dim3(256), 0, stream, per_slot,
-                   top, shared, shared_dtype, idx, weight, n_real, (const float*)h, gate, gate_stride,
+                   top, shared, shared_dtype, shared_parts, (size_t)shared_stride, idx, weight, n_real,
+                   (const float*)h, gate, gate_stride,
                    (float*)delta, n, d);
     return launch_status();
 }

@@ -800,7 +800,8 @@ class Ops:
                    "down": _decl(lib, "mls_expert_down",
                                  [_P, _P, _P, _I, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _P]),
                    "combine": _decl(lib, "mls_expert_combine",
-                                    [_P, _I, _P, _I, _P, _P, _I, _P, _P, _I, _P, _I, _I, _I, _P])}
+                                    [_P, _I, _P, _I, _I, _LL, _P, _P, _I, _P, _P, _I, _P, _I, _I, _I,
+                                     _P])}
         elif name == "shortconv":
             fns = {"qk": _decl(lib, "mls_qk_conv_norm_rope_store",
                                [_P, _I, _LL, _P, _P, _I, _P, _P, _I, _F, _P, _LL, _I, _P, _P, _P, _P,
@@ -1132,14 +1133,14 @@ class Ops:
 
     def expert_combine(self, per_slot, top: int, shared, delta, work=None, n_real=None,
                        h=None, shared_gate=None) -> None:
-        """``delta[t] = sum_j per_slot[t * top + j] + shared[t]``; with ``n_real`` a choice of
+        """``delta[t] = sum_j per_slot[t * top + j] + shared[t]`` (``shared``: a tensor,
+        ``SplitParts`` or None); with ``n_real`` a choice of
         an output from ``n_real`` on adds ``weight * h[t]`` instead (an expert that returns
         its input).  ``shared_gate``: a float32 column (one number a token, any row stride);
         the shared addend is multiplied by its sigmoid."""
         t, d = delta.shape
         _need(per_slot.shape == (t * top, d) and delta.is_contiguous(), "expert_combine: shapes")
-        _need(shared is None or (shared.shape == (t, d) and shared.is_contiguous()),
-              "expert_combine: bad shared addend")
+        sp, scode, parts, stride = self._delta_args(shared, t, d, "expert_combine: shared addend")
         idx = weight = None
         if n_real is not None:
             _need(work is not None and h is not None and h.shape == (t, d) and h.is_contiguous()
@@ -1150,10 +1151,11 @@ class Ops:
               "expert_combine: the shared addend's gate is one float32 number a token")
         self.launches += 1
         _check(self._part_lib("experts")["combine"](
-            _ptr(per_slot), top, _ptr(shared), _code(shared.dtype) if shared is not None else 0,
-            _ptr(idx), _ptr(weight), int(n_real or 0), _ptr(h), _ptr(shared_gate),
+            _ptr(per_slot), top, sp, scode, parts, stride, _ptr(idx), _ptr(weight), int(n_real or 0), _ptr(h), _ptr(shared_gate),
             shared_gate.stride(0) if shared_gate is not None else 0,
             _ptr(delta), _code(delta.dtype), t, d, self._stream()), "expert_combine")
+        if isinstance(shared, SplitParts):
+            shared.release()
 
     def add_tanh_norm(self, x, delta, norm, h, post=None, bias=None, rows=None, n_rows: int = 0,
                       y_out=None) -> None:

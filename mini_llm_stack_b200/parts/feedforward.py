@@ -295,9 +295,7 @@ class RoutedExperts(FeedForward):
         ops.expert_down(y, self.w_down, per_slot, work, self.top, self.weigh == "output")
         shared = None
         if self.shared is not None:
-            shared = self.shared.forward(h, step)
-            if not isinstance(shared, torch.Tensor):
-                shared = shared.float()              # a product left as its K-parts
+            shared = self.shared.forward(h, step)    # (maybe left as its product's K-parts)
         delta = rt.buffer("routed_delta", (t, self.d_model), rt.act_dtype)
         gate = logits[:, self.n_outputs] if self.shared_gate else None
         if self.identity:
